@@ -67,13 +67,20 @@ int b200m_rmsnorm_rows(const float* x, const int32_t* rows_idx, const void* w, f
 int b200m_add_layernorm(float* x, const void* a, const void* b, const float* b32, const void* w, void* out,
                         const int32_t* rows_idx, int rows, int cols, float eps, int is32, void* stream);
 
+/* A layer boundary of a parallel block: r = x_in + mult * y + add (y in the activation type, add fp32; each optional), x_out = r (may
+ * be x_in; required with y or add), and up to two layer norms of r, out_k = (r - mean) / sqrt(mean((r - mean)^2) + eps) * w_k + b_k
+ * (out_k NULL: skipped).  With rows_idx (int32 [rows]) nothing is added and out_k[i, :] is the norm of row rows_idx[i]. */
+int b200m_add_layernorm2(const float* x_in, float* x_out, const void* y, float mult, const float* add, const void* w1,
+                         const void* b1, void* out1, const void* w2, const void* b2, void* out2, const int32_t* rows_idx, int rows,
+                         int cols, float eps, int is32, void* stream);
+
 /* out = x / sqrt(mean(x^2) + eps) * w over the first `cols` elements of each (strided) row. */
 int b200m_rmsnorm(const void* x, int64_t x_stride, const void* w, void* out, int64_t out_stride, int rows, int cols,
                   float eps, int is32, void* stream);
 
 /* kind 0: x = [gate | up] (2n per row), out = gelu_tanh(gate) * up;  1: out = relu(x)^2 (n per row);  2: silu(gate) * up;
- * 3: out = gelu_tanh(x) (n per row). */
-int b200m_ff_act(const void* x, void* out, int64_t rows, int n, int kind, int is32, void* stream);
+ * 3: out = gelu_tanh(x) (n per row).  Rows of out are out_stride apart. */
+int b200m_ff_act(const void* x, void* out, int64_t out_stride, int64_t rows, int n, int kind, int is32, void* stream);
 
 /* Gated unit with clamped branches: x = [gate | up] (2n of x_stride elements per row), g = min(gate, limit), u = clamp(up, -limit, limit),
  * out = g * sigmoid(alpha * g) * (u + 1). */
@@ -126,13 +133,14 @@ int b200m_qk_norm_store(void* qkv, int64_t stride, int q_cols, int k_cols, int v
 
 /* Per token and head of x (row stride `stride`; q heads at q_off, key heads at k_off, value heads at v_off): q <- q / rms(q) *
  * q_norm_w with ONE weight vector of `dim` elements for all heads (NULL: no norm), then the pairs (2i, 2i+1), i < rope_dims / 2,
- * turned by cos_sin[position] = [cos (rope_dims/2) | sin (rope_dims/2)] (fp32; NULL: no rotation), in place; keys the same with
+ * turned by cos_sin[position] = [cos (rope_dims/2) | sin (rope_dims/2)] (fp32; NULL: no rotation; layout 1: the query and key pairs are
+ * (i, i + rope_dims / 2) instead), in place; keys the same with
  * k_norm_w into cache[slot] = [k (G * dim) | v (G * vdim)]; values divided by their root mean square per head (v_unit_norm) or
  * copied; v_cos_sin (optional, fp32 [positions, v_rope_dims]): the value pairs (2m, 2m+1), m < v_rope_dims / 2, are turned by the
  * token's position before the store.  cache NULL or slot < 0: queries only. */
 int b200m_headnorm_rope_store(void* x, int64_t stride, int q_off, int k_off, int v_off, int num_heads, int num_kv_heads, int dim,
                               int vdim, const void* q_norm_w, const void* k_norm_w, int v_unit_norm, const float* cos_sin,
-                              int rope_dims, const float* v_cos_sin, int v_rope_dims, const int64_t* positions, const int32_t* slots,
+                              int layout, int rope_dims, const float* v_cos_sin, int v_rope_dims, const int64_t* positions, const int32_t* slots,
                               void* cache, int n, float eps, int is32, void* stream);
 
 /* out[t, h, :] = rotate(acc[t, h, :], sign * position[t]) * sigmoid(gate[t, h, :]): per-head attention results turned (back) by
@@ -152,16 +160,19 @@ int b200m_head_mix_gate(const void* acc, int acc_f32, const float* mix, const vo
 
 /* Causal attention of num_heads query heads over num_kv_heads cached key/value heads (head h reads h / (num_heads /
  * num_kv_heads)): score = q . k * scale - slopes[h] * (i - j) (slopes NULL: no bias), visible keys 0 <= i - j < window
- * or j < keep_first (window <= 0: all j <= i), ordinary softmax.  all_values: every query head's weights are applied to the
+ * or j < keep_first (window <= 0: all j <= i); chunk > 0 (window 0 then): the keys j <= i of the query's own chunk, i - i % chunk <= j,
+ * or j < keep_first.  Softmax with, when sinks (fp32 [num_heads]) is given, one more term exp(sinks[h]) in the denominator that has no
+ * value.  gate (optional, activation type, row stride gate_stride; not with all_values): head h of token t times sigmoid(gate[t, h]).
+ * all_values: every query head's weights are applied to the
  * values of EVERY value head, out [total_q, num_heads, num_kv_heads, vdim] (for b200m_head_mix_gate).  flags & 2: out is fp32.  A cache row is row_elems long: key head g at g * dim, value head g at
- * v_off + g * vdim.  q [total_q, >= num_heads * dim] with row stride q_stride; out [total_q, num_heads * vdim].
+ * v_off + g * vdim.  q [total_q, >= num_heads * dim] with row stride q_stride; out [total_q, >= num_heads * vdim] with row stride out_stride.
  * bf16 with dim and vdim in {32, 64, 128} runs on the tensor cores unless flags & 1; everything else on the fp32 FMA pipe.
  * splits > 1 (bf16 tensor-core decode steps only): the visible keys of every row are shared out over `splits` CTAs whose
  * partials, fp32 [num_seqs, splits, num_heads (x num_kv_heads with all_values), vdim + 2] in `part`, a second launch merges. */
 int b200m_window_attention(const void* q, int64_t q_stride, const void* cache, int row_elems, int v_off,
                            const int32_t* block_tables, int bt_stride, int block_size, const int32_t* cu_q,
                            const int32_t* cu_k, const int32_t* ctx_lens, const float* slopes, int window, int keep_first,
-                           int all_values, void* out, int total_q, int num_seqs, int max_q, int num_heads, int num_kv_heads,
+                           int chunk, const float* sinks, const void* gate, int64_t gate_stride, int all_values, void* out, int64_t out_stride, int total_q, int num_seqs, int max_q, int num_heads, int num_kv_heads,
                            int dim, int vdim, float scale, int is32, int flags, int splits, float* part, void* stream);
 
 /* ---- selective scan ------------------------------------------------------------------------------------------------ */
@@ -206,6 +217,22 @@ int b200m_gated_delta(const void* x, int64_t stride, int q_off, int k_off, int v
                       const float* rate, const float* dt_bias, float* state, const int32_t* state_slots, const int32_t* cu_q,
                       const int32_t* cu_k, const int32_t* ctx_lens, float* out, int num_seqs, int num_heads, int num_kv_heads, int dim,
                       int vdim, float q_scale, int is32, void* stream);
+
+/* Matrix state with a decay per (head, key channel): g = exp(rate[h] * softplus(sign * (decay_in[t, h * dim + c] + decay_bias[h * dim + c]))),
+ * or decay_in itself when decay_done (after b200m_channel_decay).  x and the state as for b200m_gated_delta.
+ * write_in given (activation type, [n, num_heads] with row stride write_stride): the delta rule,
+ *     q, k as for b200m_gated_delta;  S <- diag(g) S;  u = sigmoid(write_in) (v - S^T k);  S <- S + k u^T;  out = S^T q
+ * write_in NULL: gated linear attention,  S <- diag(g) S + k v^T;  out = q_scale * S^T q.   dim <= 256. */
+int b200m_channel_state(const void* x, int64_t stride, int q_off, int k_off, int v_off, const void* write_in, int64_t write_stride,
+                        const float* decay_in, int64_t decay_stride, const float* rate, const float* decay_bias, float decay_sign,
+                        int decay_done, float* state, const int32_t* state_slots, const int32_t* cu_q, const int32_t* cu_k,
+                        const int32_t* ctx_lens, float* out, int num_seqs, int num_heads, int num_kv_heads, int dim, int vdim,
+                        float q_scale, int is32, void* stream);
+
+/* a[t, h * dim + c] <- exp(rate[h] * softplus(sign * (a[t, h * dim + c] + bias[h * dim + c]))), fp32, in place: the decays of many tokens
+ * formed once (b200m_channel_state forms them itself in each of a head's CTAs otherwise). */
+int b200m_channel_decay(float* a, int64_t stride, const float* rate, const float* bias, float sign, int n, int num_heads, int dim,
+                        void* stream);
 
 /* out[t, h, :] = out_scale * x[t, h, :] / sqrt(mean(x[t, h, :]^2) + eps) * w * act(gate[t, h, :]); x fp32 [n, num_heads, vdim];
  * w [vdim] shared by the heads (NULL: none); gate with row stride gate_stride (NULL: none); act 0 = sigmoid, 1 = silu; out with

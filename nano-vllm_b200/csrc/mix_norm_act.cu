@@ -2,6 +2,8 @@
 // weight-only layer norm, RMS norm of a projection output, and the feed-forward activations.
 #include "mix_common.cuh"
 
+#include <initializer_list>
+
 namespace {
 
 constexpr int ROW_THREADS = 256;
@@ -166,6 +168,122 @@ __global__ void __launch_bounds__(ROW_THREADS) add_layernorm_kernel(float* __res
     for (int c = threadIdx.x; c < cols; c += blockDim.x) stf(o + c, (xr[c] - mean) * rstd * ldf(w + c));
 }
 
+// A layer boundary of a parallel block whose branches read two layer norms of one stream:
+//     r = x_in + mult * y + add   (y: the summed branches, activation type; add: fp32; each optional)  ->  x_out (optional)
+//     out_k = (r - mean) / sqrt(mean((r - mean)^2) + eps) * w_k + b_k,  k = 1, 2 (each optional): one pair of statistics for both.
+// rows_idx (optional): row i of the outputs is row rows_idx[i] of the stream.  V columns per access (4: 128-bit stream accesses);
+// PER groups of V columns per thread stay in registers from the update to the outputs, wider rows re-read what was written.
+template <typename T, int V>
+__device__ __forceinline__ void load_cols(const T* p, float (&f)[V]) {
+    if constexpr (V == 1) {
+        f[0] = ldf(p);
+    } else if constexpr (sizeof(T) == 4) {
+        const float4 v = *reinterpret_cast<const float4*>(p);
+        f[0] = v.x, f[1] = v.y, f[2] = v.z, f[3] = v.w;
+    } else {
+        const uint2 v = *reinterpret_cast<const uint2*>(p);
+        f[0] = bf16lo(v.x), f[1] = bf16hi(v.x), f[2] = bf16lo(v.y), f[3] = bf16hi(v.y);
+    }
+}
+template <typename T, int V>
+__device__ __forceinline__ void store_cols(T* p, const float (&f)[V]) {
+    if constexpr (V == 1) stf(p, f[0]);
+    else if constexpr (sizeof(T) == 4) *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]);
+    else *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16x2(f[0], f[1]), pack_bf16x2(f[2], f[3]));
+}
+
+template <typename T, int V, int PER>
+__global__ void __launch_bounds__(ROW_THREADS) add_layernorm2_kernel(const float* x_in, float* x_out, const T* __restrict__ y, float mult,
+                                                                     const float* __restrict__ add, const T* __restrict__ w1,
+                                                                     const T* __restrict__ b1, T* __restrict__ out1, const T* __restrict__ w2,
+                                                                     const T* __restrict__ b2, T* __restrict__ out2,
+                                                                     const int32_t* __restrict__ rows_idx, int cols, float eps) {
+    B200_PDL_SYNC();
+    __shared__ float red[ROW_THREADS / 32];
+    const int64_t row = rows_idx ? rows_idx[blockIdx.x] : blockIdx.x, base = row * cols, obase = (int64_t)blockIdx.x * cols;
+    const int step = blockDim.x * V;
+    auto updated = [&](int c, float (&f)[V]) {
+        float a[V];
+        load_cols<float, V>(x_in + base + c, f);
+        if (y) {
+            load_cols<T, V>(y + base + c, a);
+#pragma unroll
+            for (int e = 0; e < V; ++e) f[e] = fmaf(mult, a[e], f[e]);
+        }
+        if (add) {
+            load_cols<float, V>(add + base + c, a);
+#pragma unroll
+            for (int e = 0; e < V; ++e) f[e] += a[e];
+        }
+        if (x_out) store_cols<float, V>(x_out + base + c, f);
+    };
+    const float* again = x_out ? x_out : x_in;             // beyond the registers: the same thread wrote these elements, no fence needed
+    float r[PER][V];
+    float s = 0.f;
+#pragma unroll
+    for (int k = 0; k < PER; ++k) {
+        const int c = threadIdx.x * V + k * step;
+#pragma unroll
+        for (int e = 0; e < V; ++e) r[k][e] = 0.f;
+        if (c < cols) updated(c, r[k]);
+#pragma unroll
+        for (int e = 0; e < V; ++e) s += r[k][e];
+    }
+    for (int c = threadIdx.x * V + PER * step; c < cols; c += step) {
+        float f[V];
+        updated(c, f);
+#pragma unroll
+        for (int e = 0; e < V; ++e) s += f[e];
+    }
+    if (out1 == nullptr && out2 == nullptr) return;
+    const float mean = block_sum(s, red) / (float)cols;
+    float q = 0.f;
+#pragma unroll
+    for (int k = 0; k < PER; ++k)
+        if (threadIdx.x * V + k * step < cols)
+#pragma unroll
+            for (int e = 0; e < V; ++e) {
+                r[k][e] -= mean;
+                q = fmaf(r[k][e], r[k][e], q);
+            }
+    for (int c = threadIdx.x * V + PER * step; c < cols; c += step) {
+        float f[V];
+        load_cols<float, V>(again + base + c, f);
+#pragma unroll
+        for (int e = 0; e < V; ++e) q = fmaf(f[e] - mean, f[e] - mean, q);
+    }
+    const float rstd = 1.0f / sqrtf(block_sum(q, red) / (float)cols + eps);
+    auto emit = [&](int c, const float (&f)[V]) {          // f: deviations from the mean
+        float w[V], b[V], o[V];
+        if (out1) {
+            load_cols<T, V>(w1 + c, w);
+            load_cols<T, V>(b1 + c, b);
+#pragma unroll
+            for (int e = 0; e < V; ++e) o[e] = fmaf(f[e] * rstd, w[e], b[e]);
+            store_cols<T, V>(out1 + obase + c, o);
+        }
+        if (out2) {
+            load_cols<T, V>(w2 + c, w);
+            load_cols<T, V>(b2 + c, b);
+#pragma unroll
+            for (int e = 0; e < V; ++e) o[e] = fmaf(f[e] * rstd, w[e], b[e]);
+            store_cols<T, V>(out2 + obase + c, o);
+        }
+    };
+#pragma unroll
+    for (int k = 0; k < PER; ++k) {
+        const int c = threadIdx.x * V + k * step;
+        if (c < cols) emit(c, r[k]);
+    }
+    for (int c = threadIdx.x * V + PER * step; c < cols; c += step) {
+        float f[V];
+        load_cols<float, V>(again + base + c, f);
+#pragma unroll
+        for (int e = 0; e < V; ++e) f[e] -= mean;
+        emit(c, f);
+    }
+}
+
 template <typename T>
 __global__ void __launch_bounds__(ROW_THREADS) rmsnorm_any_kernel(const T* __restrict__ x, int64_t x_stride, const T* __restrict__ w,
                                                                   T* __restrict__ out, int64_t out_stride, int cols, float eps) {
@@ -189,25 +307,27 @@ __device__ __forceinline__ float gelu_tanh_(float z) {
 // kind 0: x = [gate | up] per row, out = gelu_tanh(gate) * up;  kind 1: out = relu(x)^2 (no second half);
 // kind 2: x = [gate | up], out = silu(gate) * up;  kind 3: out = gelu_tanh(x) (no second half)
 template <typename T>
-__global__ void ff_act_kernel(const T* __restrict__ x, T* __restrict__ out, int64_t rows, int n, int kind) {
+__global__ void ff_act_kernel(const T* __restrict__ x, T* __restrict__ out, int64_t out_stride, int64_t rows, int n, int kind) {
     B200_PDL_SYNC();
     const int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x;
     if (i >= rows * n) return;
     const int64_t r = i / n;
     const int c = (int)(i - r * n);
+    T* o = out + r * out_stride + c;
     if (kind == 1) {
         const float v = fmaxf(ldf(x + i), 0.f);
-        stf(out + i, v * v);
+        stf(o, v * v);
     } else if (kind == 3) {
-        stf(out + i, gelu_tanh_(ldf(x + i)));
+        stf(o, gelu_tanh_(ldf(x + i)));
     } else {
         const float g = ldf(x + r * 2 * n + c), u = ldf(x + r * 2 * n + n + c);
-        stf(out + i, (kind == 0 ? gelu_tanh_(g) : siluf_(g)) * u);
+        stf(o, (kind == 0 ? gelu_tanh_(g) : siluf_(g)) * u);
     }
 }
 
 // bf16 rows whose halves are multiples of 8: 8 columns per thread, 128-bit accesses, one row per blockIdx.y
-__global__ void __launch_bounds__(256) ff_act_vec_kernel(const __nv_bfloat16* __restrict__ x, __nv_bfloat16* __restrict__ out, int n, int kind) {
+__global__ void __launch_bounds__(256) ff_act_vec_kernel(const __nv_bfloat16* __restrict__ x, __nv_bfloat16* __restrict__ out, int64_t out_stride, int n,
+                                                        int kind) {
     B200_PDL_SYNC();
     const int c = (blockIdx.x * 256 + threadIdx.x) << 3;
     if (c >= n) return;
@@ -228,7 +348,7 @@ __global__ void __launch_bounds__(256) ff_act_vec_kernel(const __nv_bfloat16* __
 #pragma unroll
         for (int e = 0; e < 8; ++e) o[e] = (kind == 0 ? gelu_tanh_(gt[e]) : siluf_(gt[e])) * up[e];
     }
-    *reinterpret_cast<uint4*>(out + r * n + c) = pack8(o);
+    *reinterpret_cast<uint4*>(out + r * out_stride + c) = pack8(o);
 }
 
 // Gated unit with clamped branches: x = [gate | up] per row, g = min(gate, limit), u = clamp(up, -limit, limit),
@@ -334,7 +454,7 @@ __global__ void __launch_bounds__(256) softcap_kernel(float* __restrict__ x, int
 
 }  // namespace
 
-extern "C" int b200m_abi_version(void) { return 4; }
+extern "C" int b200m_abi_version(void) { return 5; }
 
 extern "C" int b200m_ff_glu_clamped(const void* x, int64_t x_stride, void* out, int64_t rows, int n, float limit, float alpha, int is32,
                                     void* stream) {
@@ -448,6 +568,30 @@ extern "C" int b200m_add_layernorm(float* x, const void* a, const void* b, const
     return b200_launch_status(nullptr);
 }
 
+extern "C" int b200m_add_layernorm2(const float* x_in, float* x_out, const void* y, float mult, const float* add, const void* w1,
+                                    const void* b1, void* out1, const void* w2, const void* b2, void* out2, const int32_t* rows_idx,
+                                    int rows, int cols, float eps, int is32, void* stream) {
+    if (!x_in || rows < 0 || cols <= 0 || (out1 && (!w1 || !b1)) || (out2 && (!w2 || !b2))) return B200_EINVAL;
+    if ((y || add) ? (!x_out || rows_idx) : (rows_idx && x_out)) return B200_EINVAL;     // an update needs a destination and covers whole steps
+    if (rows == 0) return B200_OK;
+    cudaStream_t st = static_cast<cudaStream_t>(stream);
+    uintptr_t bits = 0;
+    for (const void* p : {static_cast<const void*>(x_in), static_cast<const void*>(x_out), y, static_cast<const void*>(add), w1, b1,
+                          static_cast<const void*>(out1), w2, b2, static_cast<const void*>(out2)})
+        bits |= reinterpret_cast<uintptr_t>(p);
+    const bool vec = cols % 4 == 0 && bits % 16 == 0;
+#define LN2_GO(V, PER)                                                                                                             \
+    B200M_DISPATCH(is32, B200_LAUNCH((add_layernorm2_kernel<T, V, PER>), rows, ROW_THREADS, 0, st, x_in, x_out, static_cast<const T*>(y), mult, add, \
+                                     static_cast<const T*>(w1), static_cast<const T*>(b1), static_cast<T*>(out1), static_cast<const T*>(w2), \
+                                     static_cast<const T*>(b2), static_cast<T*>(out2), rows_idx, cols, eps))
+    if (vec && cols <= 4 * ROW_THREADS) LN2_GO(4, 1);
+    else if (vec && cols <= 8 * ROW_THREADS) LN2_GO(4, 2);
+    else if (vec) LN2_GO(4, 4);
+    else LN2_GO(1, 4);
+#undef LN2_GO
+    return b200_launch_status(nullptr);
+}
+
 extern "C" int b200m_rmsnorm(const void* x, int64_t x_stride, const void* w, void* out, int64_t out_stride, int rows, int cols,
                              float eps, int is32, void* stream) {
     if (!x || !w || !out || rows < 0 || cols <= 0) return B200_EINVAL;
@@ -458,20 +602,20 @@ extern "C" int b200m_rmsnorm(const void* x, int64_t x_stride, const void* w, voi
     return b200_launch_status(nullptr);
 }
 
-extern "C" int b200m_ff_act(const void* x, void* out, int64_t rows, int n, int kind, int is32, void* stream) {
-    if (!x || !out || rows < 0 || n <= 0 || kind < 0 || kind > 3) return B200_EINVAL;
+extern "C" int b200m_ff_act(const void* x, void* out, int64_t out_stride, int64_t rows, int n, int kind, int is32, void* stream) {
+    if (!x || !out || rows < 0 || n <= 0 || out_stride < n || kind < 0 || kind > 3) return B200_EINVAL;
     if (rows == 0) return B200_OK;
-    if (!is32 && n % 8 == 0 && rows <= 65535 * 32 && ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(out)) & 15) == 0) {
+    if (!is32 && n % 8 == 0 && out_stride % 8 == 0 && rows <= 65535 * 32 && ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(out)) & 15) == 0) {
         for (int64_t r0 = 0; r0 < rows; r0 += 65535) {             // grid.y limit
             const int64_t nr = rows - r0 < 65535 ? rows - r0 : 65535;
             const int64_t in_row = (kind == 1 || kind == 3) ? n : 2 * (int64_t)n;
             B200_LAUNCH((ff_act_vec_kernel), dim3((n / 8 + 255) / 256, (unsigned)nr), 256, 0, static_cast<cudaStream_t>(stream),
-                        static_cast<const __nv_bfloat16*>(x) + r0 * in_row, static_cast<__nv_bfloat16*>(out) + r0 * n, n, kind);
+                        static_cast<const __nv_bfloat16*>(x) + r0 * in_row, static_cast<__nv_bfloat16*>(out) + r0 * out_stride, out_stride, n, kind);
         }
         return b200_launch_status(nullptr);
     }
     const int64_t total = rows * n;
     B200M_DISPATCH(is32, B200_LAUNCH((ff_act_kernel<T>), (unsigned)((total + 255) / 256), 256, 0, static_cast<cudaStream_t>(stream),
-                                     static_cast<const T*>(x), static_cast<T*>(out), rows, n, kind));
+                                     static_cast<const T*>(x), static_cast<T*>(out), out_stride, rows, n, kind));
     return b200_launch_status(nullptr);
 }

@@ -14,13 +14,14 @@
 //   zero keeping (product of a, end state), a serial pass over the chunk summaries that leaves every chunk's start state, and
 //   every chunk again from its start state writing the output.
 //
-// Gated delta rule (per head a matrix state S [dim, vdim]; query/key head h / (H / G)):
-//     q <- q / sqrt(|q|^2 + 1e-6) * q_scale,  k <- k / sqrt(|k|^2 + 1e-6)
-//     g = exp(rate_h softplus(a_t + dt_bias_h)),  beta = sigmoid(b_t)
-//     S <- g S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q
-//   Columns of S are independent, so a thread group of four lanes owns one column (dim / 4 state elements per lane in
-//   registers) and walks the tokens; a CTA covers 32 columns of one (sequence, head).  The decay folds into the update:
-//   d = S_old^T k;  u = beta (v - g d);  S_new = g S_old + k u.  Tokens are staged through shared memory a chunk ahead.
+// Matrix states (per head S [dim, vdim]; query/key head h / (H / G)); one kernel, three rules:
+//   gated delta rule            q <- q / sqrt(|q|^2 + 1e-6) * q_scale,  k <- k / sqrt(|k|^2 + 1e-6)
+//                               g = exp(rate_h softplus(a_t + dt_bias_h)),  beta = sigmoid(b_t)
+//                               S <- g S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q
+//   delta rule, channel decays  the same with g per (head, key channel) on the rows of S
+//   gated linear attention      S <- diag(g) S + k (q_scale q, k as they are) v^T;  o = S^T q;  g per (head, key channel)
+//   Channel decays are g = exp(rate_h softplus(sign (a + bias))): sign 1 is the softplus form; sigmoid(z)^(1 / tau) is rate
+//   -1 / tau with sign -1.  Columns of S are independent: a lane group owns one or two of them and walks the tokens.
 #include "mix_common.cuh"
 
 namespace {
@@ -105,117 +106,165 @@ __global__ void __launch_bounds__(128) diag_carry_kernel(float* __restrict__ ws,
     *st = S;
 }
 
-constexpr int GD_LANES = 4;            // lanes that share one column of the state
-constexpr int GD_COLS = 32;            // columns per CTA (128 threads)
-
-// DPL state rows per lane: lane `sub` of a column's group owns rows sub * DPL .. sub * DPL + DPL - 1 (zero beyond dim).
+// Matrix-state recurrences.  LANES lanes share COLS columns of a head's state: lane `sub` of a group owns rows sub * DPL ..
+// sub * DPL + DPL - 1 of them (zero beyond dim) in registers; a CTA covers MS_THREADS / LANES * COLS columns of one (sequence, head).
 // state: [slots, H, vdim, dim] (a column's rows are contiguous).
+//   CH    : decays come per (head, key channel) as rows of decay_in instead of one number per (token, head)
+//   DELTA : delta rule (unit-norm q and k, write strength, correction towards v); otherwise S <- g S + k v^T with q and k as they are
 // Tokens are staged through shared memory TB at a time, as fp32: the chunk after the current one is fetched into registers
 // before the current one is worked on and stored afterwards (two buffers), so the serial walk never waits for global memory.
-// A staged key or query row is four lane segments of DPL floats, each padded by four: 128-bit reads without bank conflicts.
-// After a chunk lands, 128 / TB threads per token form its unit-norm factors, write strength and decay once for the CTA.
-template <typename T, int DPL>
-__global__ void __launch_bounds__(GD_LANES * GD_COLS) gated_delta_kernel(
-    const T* __restrict__ x, int64_t stride, int q_off, int k_off, int v_off,     // per token: q, k [G, dim], v [H, vdim] (convolved, activated)
-    const float* __restrict__ ba, int64_t ba_stride,                              // per token: H write strengths, then H decay inputs (pre-activation)
-    const float* __restrict__ rate, const float* __restrict__ dt_bias,            // [H]: rate = -exp(A_log)
-    float* __restrict__ state, const int32_t* __restrict__ state_slots, const int32_t* __restrict__ cu_q,
+// A staged row is LANES segments of DPL floats, each padded by four: 128-bit reads without bank conflicts.  After a chunk
+// lands, MS_THREADS / TB threads per token form its unit-norm factors and k . q once for the CTA.  The delta rule reads out
+// before it writes, o = (g S)^T q + u (k . q), so that both column sums of a token are reduced together.
+constexpr int MS_THREADS = 128;
+
+struct DecayIn {
+    const float* in;          // pre-activations (or, with `done`, the decays themselves): CH: [n, >= H * dim], else one per head
+    int64_t stride;
+    const float* rate;        // [H]
+    const float* bias;        // CH: [H * dim], else [H]
+    float sign;               // g = exp(rate_h * softplus(sign * (in + bias)))
+    int done;
+};
+__device__ __forceinline__ float decay_of(float a, float rate, float bias, float sign) { return expf(rate * softplus_(sign * (a + bias))); }
+
+template <typename T, int DPL, int LANES, int COLS, bool CH, bool DELTA>
+__global__ void __launch_bounds__(MS_THREADS) matrix_state_kernel(
+    const T* __restrict__ x, int64_t stride, int q_off, int k_off, int v_off,     // per token: q, k [G, dim], v [H, vdim]
+    const float* __restrict__ write_in, const T* __restrict__ write_t, int64_t write_stride,      // DELTA: H write strengths (pre-activation), fp32 or T
+    DecayIn dec, float* __restrict__ state, const int32_t* __restrict__ state_slots, const int32_t* __restrict__ cu_q,
     const int32_t* __restrict__ cu_k, const int32_t* __restrict__ ctx_lens, float* __restrict__ out,      // [n, H, vdim] fp32
     int H, int G, int dim, int vdim, float q_scale) {
     B200_PDL_SYNC();
-    constexpr int NT = GD_LANES * GD_COLS;
-    constexpr int TB = DPL >= 64 ? 8 : 16;
-    constexpr int SEG = DPL + 4, ROW = GD_LANES * SEG, DP = GD_LANES * DPL;
-    constexpr int PF = (TB * DP) / NT;                     // key (and query) elements a thread fetches per chunk
-    constexpr int PV = (TB * GD_COLS) / NT;                // value elements a thread fetches per chunk
-    constexpr int TPT = NT / TB;                           // threads that share one token's factors
+    constexpr int NT = MS_THREADS, GC = NT / LANES * COLS;  // columns of the CTA
+    constexpr int DP = LANES * DPL, SEG = DPL + 4, ROW = LANES * SEG;
+    constexpr int TB = DP >= 256 ? 4 : (DP >= 128 || CH) ? 8 : 16;
+    constexpr int PF = (TB * DP + NT - 1) / NT;            // key (query, decay) elements a thread fetches per chunk
+    constexpr int PV = (TB * GC + NT - 1) / NT;            // value elements a thread fetches per chunk
+    constexpr int TPT = NT / TB < 32 ? NT / TB : 32;       // threads that share one token's factors
     __shared__ __align__(16) float ks[2][TB][ROW];
     __shared__ __align__(16) float qs[2][TB][ROW];
-    __shared__ float vs[2][TB][GD_COLS];
-    __shared__ float sc[2][TB][4];                         // key normaliser, query normaliser * scale, write strength, decay
+    __shared__ __align__(16) float gs[CH ? 2 : 1][CH ? TB : 1][CH ? ROW : 4];
+    __shared__ __align__(16) float vs[2][TB][GC];
+    __shared__ __align__(16) float sc[2][TB][4];           // key normaliser, query normaliser * scale, write strength, (k . q) of the unit keys and scaled queries
+    __shared__ float sd[2][TB];                            // decay per token (not CH)
     const int h = blockIdx.x, s = blockIdx.y, tid = threadIdx.x;
     const SeqSpan sp = seq_span(cu_q, cu_k, ctx_lens, s);
     if (sp.qlen <= 0) return;
-    const int sub = tid % GD_LANES;
-    const int col0 = blockIdx.z * GD_COLS, col = col0 + tid / GD_LANES;
-    const bool live = col < vdim;
-    const int cc = live ? col : vdim - 1;
+    const int sub = tid % LANES, grp = tid / LANES;
+    const int col0 = blockIdx.z * GC, mycol = col0 + grp * COLS;
     const int g = h / (H / G);
-    float* st = state + (((int64_t)state_slots[s] * H + h) * vdim + cc) * dim + sub * DPL;
+    float* st = state + ((int64_t)state_slots[s] * H + h) * vdim * dim + sub * DPL;      // + column * dim
     const bool has_hist = sp.klen - sp.qlen > 0;
-    const bool vec_state = dim == GD_LANES * DPL;           // whole lane segments (then 16-byte aligned too): 128-bit state accesses
-    float S[DPL];
-    if (has_hist && vec_state) {
+    const bool vec_state = dim % 4 == 0;                    // 16-byte aligned segments: 128-bit state accesses
+    float S[COLS][DPL];
 #pragma unroll
-        for (int k = 0; k < DPL / 4; ++k) {
-            const float4 f = reinterpret_cast<const float4*>(st)[k];
-            S[4 * k] = f.x, S[4 * k + 1] = f.y, S[4 * k + 2] = f.z, S[4 * k + 3] = f.w;
+    for (int c = 0; c < COLS; ++c) {
+        const bool have = has_hist && mycol + c < vdim;
+        const float* sr = st + (int64_t)(mycol + c) * dim;
+        if (vec_state) {
+#pragma unroll
+            for (int k = 0; k < DPL / 4; ++k) {
+                float4 f = make_float4(0.f, 0.f, 0.f, 0.f);
+                if (have && sub * DPL + 4 * k < dim) f = reinterpret_cast<const float4*>(sr)[k];
+                S[c][4 * k] = f.x, S[c][4 * k + 1] = f.y, S[c][4 * k + 2] = f.z, S[c][4 * k + 3] = f.w;
+            }
+        } else {
+#pragma unroll
+            for (int k = 0; k < DPL; ++k) S[c][k] = (have && sub * DPL + k < dim) ? sr[k] : 0.f;
         }
-    } else {
-#pragma unroll
-        for (int k = 0; k < DPL; ++k) S[k] = (has_hist && sub * DPL + k < dim) ? st[k] : 0.f;
     }
-    const float rt = rate[h], db = dt_bias[h];
+    const float rt = dec.done ? 0.f : dec.rate[h], db = (CH || dec.done) ? 0.f : dec.bias[h];
     const T* qp = x + q_off + (int64_t)g * dim;
     const T* kp = x + k_off + (int64_t)g * dim;
     const T* vp = x + v_off + (int64_t)h * vdim + col0;
-    float fk[PF], fq[PF], fv[PV], fb = 0.f, fa = 0.f;      // the next chunk, in flight
+    const float* gp = CH ? dec.in + (int64_t)h * dim : dec.in + h;
+    float fk[PF], fq[PF], fg[CH ? PF : 1], fv[PV], fb = 0.f, fa = 0.f;      // the next chunk, in flight
     auto fetch = [&](int i0) {
 #pragma unroll
         for (int j = 0; j < PF; ++j) {
             const int e = tid + NT * j, t = e / DP, d = e - t * DP;
-            const bool ok = i0 + t < sp.qlen && d < dim;
+            const bool ok = t < TB && i0 + t < sp.qlen && d < dim;
             const int64_t row = sp.q0 + i0 + t;
             fk[j] = ok ? ldf(kp + row * stride + d) : 0.f;
             fq[j] = ok ? ldf(qp + row * stride + d) : 0.f;
+            if constexpr (CH) fg[j] = ok ? gp[row * dec.stride + d] : 0.f;
         }
 #pragma unroll
         for (int j = 0; j < PV; ++j) {
-            const int e = tid + NT * j, t = e / GD_COLS, c = e - t * GD_COLS;
-            fv[j] = (i0 + t < sp.qlen && col0 + c < vdim) ? ldf(vp + (int64_t)(sp.q0 + i0 + t) * stride + c) : 0.f;
+            const int e = tid + NT * j, t = e / GC, c = e - t * GC;
+            fv[j] = (t < TB && i0 + t < sp.qlen && col0 + c < vdim) ? ldf(vp + (int64_t)(sp.q0 + i0 + t) * stride + c) : 0.f;
         }
         if (tid < TB && i0 + tid < sp.qlen) {
-            fb = ba[(int64_t)(sp.q0 + i0 + tid) * ba_stride + h];
-            fa = ba[(int64_t)(sp.q0 + i0 + tid) * ba_stride + H + h];
+            const int64_t row = sp.q0 + i0 + tid;
+            if constexpr (DELTA) fb = write_in ? write_in[row * write_stride + h] : ldf(write_t + row * write_stride + h);
+            if constexpr (!CH) fa = gp[row * dec.stride];
         }
     };
     auto land = [&](int buf) {                             // registers -> shared memory
 #pragma unroll
         for (int j = 0; j < PF; ++j) {
             const int e = tid + NT * j, t = e / DP, d = e - t * DP;
+            if (t >= TB) break;
             const int at = (d / DPL) * SEG + (d % DPL);
             ks[buf][t][at] = fk[j];
-            qs[buf][t][at] = fq[j];
+            qs[buf][t][at] = DELTA ? fq[j] : fq[j] * q_scale;
+            if constexpr (CH) gs[buf][t][at] = d < dim ? (dec.done ? fg[j] : decay_of(fg[j], rt, dec.bias[(int64_t)h * dim + d], dec.sign)) : 0.f;
         }
 #pragma unroll
         for (int j = 0; j < PV; ++j) {
             const int e = tid + NT * j;
-            vs[buf][e / GD_COLS][e % GD_COLS] = fv[j];
+            if (e < TB * GC) vs[buf][e / GC][e % GC] = fv[j];
         }
         if (tid < TB) {
-            sc[buf][tid][2] = sigmoidf_(fb);
-            sc[buf][tid][3] = expf(rt * softplus_(fa + db));
+            if constexpr (DELTA) sc[buf][tid][2] = sigmoidf_(fb);
+            if constexpr (!CH) sd[buf][tid] = dec.done ? fa : decay_of(fa, rt, db, dec.sign);
         }
     };
-    auto factors = [&](int buf) {                          // after a barrier: the unit-norm factors of the chunk's tokens
-        const int t = tid / TPT, j = tid % TPT;
-        float ssk = 0.f, ssq = 0.f;
-        for (int d = j; d < DP; d += TPT) {
-            const int at = (d / DPL) * SEG + (d % DPL);
-            const float a = ks[buf][t][at], b = qs[buf][t][at];
-            ssk = fmaf(a, a, ssk);
-            ssq = fmaf(b, b, ssq);
-        }
+    auto factors = [&](int buf) {                          // after a barrier: the unit-norm factors and k . q of the chunk's tokens
+        if constexpr (DELTA) {
+            const int t = tid / TPT, j = tid % TPT;
+            float ssk = 0.f, ssq = 0.f, skq = 0.f;
+            if (t < TB)
+                for (int d = j; d < DP; d += TPT) {
+                    const int at = (d / DPL) * SEG + (d % DPL);
+                    const float a = ks[buf][t][at], b = qs[buf][t][at];
+                    ssk = fmaf(a, a, ssk);
+                    ssq = fmaf(b, b, ssq);
+                    skq = fmaf(a, b, skq);
+                }
 #pragma unroll
-        for (int o = 1; o < TPT; o <<= 1) {
-            ssk += __shfl_xor_sync(0xffffffffu, ssk, o);
-            ssq += __shfl_xor_sync(0xffffffffu, ssq, o);
-        }
-        if (j == 0) {
-            sc[buf][t][0] = 1.0f / sqrtf(ssk + 1e-6f);
-            sc[buf][t][1] = q_scale / sqrtf(ssq + 1e-6f);
+            for (int o = 1; o < TPT; o <<= 1) {
+                ssk += __shfl_xor_sync(0xffffffffu, ssk, o);
+                ssq += __shfl_xor_sync(0xffffffffu, ssq, o);
+                skq += __shfl_xor_sync(0xffffffffu, skq, o);
+            }
+            if (j == 0 && t < TB) {
+                const float rk = 1.0f / sqrtf(ssk + 1e-6f), rq = q_scale / sqrtf(ssq + 1e-6f);
+                sc[buf][t][0] = rk;
+                sc[buf][t][1] = rq;
+                sc[buf][t][3] = skq * rq;                  // times u (which carries the key's normaliser): what the token's own write adds to its read-out
+            }
         }
     };
+    // Column sums over the group's lanes.  COLS = 2: the first exchange sends one column each way, after which even lanes carry
+    // column 0 and odd lanes column 1.
+    auto reduce = [&](float (&v)[COLS]) -> float {
+        if constexpr (COLS == 2) {
+            const bool odd = sub & 1;
+            float r = (odd ? v[1] : v[0]) + __shfl_xor_sync(0xffffffffu, odd ? v[0] : v[1], 1);
+#pragma unroll
+            for (int o = 2; o < LANES; o <<= 1) r += __shfl_xor_sync(0xffffffffu, r, o);
+            return r;
+        } else {
+            float r = v[0];
+#pragma unroll
+            for (int o = 1; o < LANES; o <<= 1) r += __shfl_xor_sync(0xffffffffu, r, o);
+            return r;
+        }
+    };
+    const int ocol = mycol + (COLS == 2 ? (sub & 1) : 0);  // the column whose sum this lane holds after reduce()
+    const bool writer = sub < COLS && ocol < vdim;
     fetch(0);
     land(0);
     __syncthreads();
@@ -228,39 +277,71 @@ __global__ void __launch_bounds__(GD_LANES * GD_COLS) gated_delta_kernel(
         for (int t = 0; t < nt; ++t) {
             const float4* kr = reinterpret_cast<const float4*>(&ks[buf][t][sub * SEG]);
             const float4* qr = reinterpret_cast<const float4*>(&qs[buf][t][sub * SEG]);
-            float4 kk[DPL / 4];
-            float d4[4] = {0.f, 0.f, 0.f, 0.f};
+            const float4* gr = reinterpret_cast<const float4*>(&gs[CH ? buf : 0][CH ? t : 0][CH ? sub * SEG : 0]);
+            const float gt = CH ? 0.f : sd[buf][t];
+            float v[COLS], o[COLS];
 #pragma unroll
-            for (int k = 0; k < DPL / 4; ++k) {
-                kk[k] = kr[k];
-                d4[0] = fmaf(S[4 * k], kk[k].x, d4[0]);
-                d4[1] = fmaf(S[4 * k + 1], kk[k].y, d4[1]);
-                d4[2] = fmaf(S[4 * k + 2], kk[k].z, d4[2]);
-                d4[3] = fmaf(S[4 * k + 3], kk[k].w, d4[3]);
+            for (int c = 0; c < COLS; ++c) {
+                v[c] = vs[buf][t][grp * COLS + c];
+                o[c] = 0.f;
             }
-            float dk = (d4[0] + d4[1]) + (d4[2] + d4[3]);
+            if constexpr (DELTA) {
+                float4 kk[DPL / 4];
+                float d[COLS];
 #pragma unroll
-            for (int o = 1; o < GD_LANES; o <<= 1) dk += __shfl_xor_sync(0xffffffffu, dk, o);
-            const float rk = sc[buf][t][0], rq = sc[buf][t][1], beta = sc[buf][t][2], gdec = sc[buf][t][3];
-            const float v = vs[buf][t][tid / GD_LANES];
-            const float uw = beta * (v - gdec * dk * rk) * rk;   // u times the key's normaliser: S += (k rk) u
-            float o4[4] = {0.f, 0.f, 0.f, 0.f};
+                for (int c = 0; c < COLS; ++c) d[c] = 0.f;
 #pragma unroll
-            for (int k = 0; k < DPL / 4; ++k) {
-                const float4 qq = qr[k];
-                S[4 * k] = fmaf(kk[k].x, uw, gdec * S[4 * k]);
-                S[4 * k + 1] = fmaf(kk[k].y, uw, gdec * S[4 * k + 1]);
-                S[4 * k + 2] = fmaf(kk[k].z, uw, gdec * S[4 * k + 2]);
-                S[4 * k + 3] = fmaf(kk[k].w, uw, gdec * S[4 * k + 3]);
-                o4[0] = fmaf(S[4 * k], qq.x, o4[0]);
-                o4[1] = fmaf(S[4 * k + 1], qq.y, o4[1]);
-                o4[2] = fmaf(S[4 * k + 2], qq.z, o4[2]);
-                o4[3] = fmaf(S[4 * k + 3], qq.w, o4[3]);
+                for (int k = 0; k < DPL / 4; ++k) {
+                    kk[k] = kr[k];
+                    const float4 qq = qr[k];
+                    const float4 gg = CH ? gr[k] : make_float4(gt, gt, gt, gt);
+#pragma unroll
+                    for (int c = 0; c < COLS; ++c) {
+                        S[c][4 * k] *= gg.x, S[c][4 * k + 1] *= gg.y, S[c][4 * k + 2] *= gg.z, S[c][4 * k + 3] *= gg.w;
+                        d[c] = fmaf(S[c][4 * k], kk[k].x, d[c]), o[c] = fmaf(S[c][4 * k], qq.x, o[c]);
+                        d[c] = fmaf(S[c][4 * k + 1], kk[k].y, d[c]), o[c] = fmaf(S[c][4 * k + 1], qq.y, o[c]);
+                        d[c] = fmaf(S[c][4 * k + 2], kk[k].z, d[c]), o[c] = fmaf(S[c][4 * k + 2], qq.z, o[c]);
+                        d[c] = fmaf(S[c][4 * k + 3], kk[k].w, d[c]), o[c] = fmaf(S[c][4 * k + 3], qq.w, o[c]);
+                    }
+                }
+                const float dk = reduce(d), oq = reduce(o);
+                const float4 f = *reinterpret_cast<const float4*>(sc[buf][t]);
+                const float vo = COLS == 2 ? ((sub & 1) ? v[COLS - 1] : v[0]) : v[0];
+                const float ub = f.z * (vo - dk * f.x) * f.x;             // u times the key's normaliser: S += (k rk) u
+                if (writer) out[((int64_t)(sp.q0 + i0 + t) * H + h) * vdim + ocol] = fmaf(ub, f.w, oq * f.y);
+                float u[COLS];
+                if constexpr (COLS == 2) {
+                    const float other = __shfl_xor_sync(0xffffffffu, ub, 1);
+                    u[0] = (sub & 1) ? other : ub;
+                    u[COLS - 1] = (sub & 1) ? ub : other;
+                } else {
+                    u[0] = ub;
+                }
+#pragma unroll
+                for (int k = 0; k < DPL / 4; ++k)
+#pragma unroll
+                    for (int c = 0; c < COLS; ++c) {
+                        S[c][4 * k] = fmaf(kk[k].x, u[c], S[c][4 * k]);
+                        S[c][4 * k + 1] = fmaf(kk[k].y, u[c], S[c][4 * k + 1]);
+                        S[c][4 * k + 2] = fmaf(kk[k].z, u[c], S[c][4 * k + 2]);
+                        S[c][4 * k + 3] = fmaf(kk[k].w, u[c], S[c][4 * k + 3]);
+                    }
+            } else {
+#pragma unroll
+                for (int k = 0; k < DPL / 4; ++k) {
+                    const float4 kk = kr[k], qq = qr[k];
+                    const float4 gg = CH ? gr[k] : make_float4(gt, gt, gt, gt);
+#pragma unroll
+                    for (int c = 0; c < COLS; ++c) {
+                        S[c][4 * k] = fmaf(kk.x, v[c], gg.x * S[c][4 * k]), o[c] = fmaf(S[c][4 * k], qq.x, o[c]);
+                        S[c][4 * k + 1] = fmaf(kk.y, v[c], gg.y * S[c][4 * k + 1]), o[c] = fmaf(S[c][4 * k + 1], qq.y, o[c]);
+                        S[c][4 * k + 2] = fmaf(kk.z, v[c], gg.z * S[c][4 * k + 2]), o[c] = fmaf(S[c][4 * k + 2], qq.z, o[c]);
+                        S[c][4 * k + 3] = fmaf(kk.w, v[c], gg.w * S[c][4 * k + 3]), o[c] = fmaf(S[c][4 * k + 3], qq.w, o[c]);
+                    }
+                }
+                const float oq = reduce(o);
+                if (writer) out[((int64_t)(sp.q0 + i0 + t) * H + h) * vdim + ocol] = oq;
             }
-            float oq = (o4[0] + o4[1]) + (o4[2] + o4[3]);
-#pragma unroll
-            for (int o = 1; o < GD_LANES; o <<= 1) oq += __shfl_xor_sync(0xffffffffu, oq, o);
-            if (live && sub == 0) out[((int64_t)(sp.q0 + i0 + t) * H + h) * vdim + col] = oq * rq;
         }
         if (more) {
             land(buf ^ 1);                                 // its last readers passed the barrier that closed the previous chunk
@@ -269,14 +350,54 @@ __global__ void __launch_bounds__(GD_LANES * GD_COLS) gated_delta_kernel(
             __syncthreads();
         }
     }
-    if (live && vec_state) {
 #pragma unroll
-        for (int k = 0; k < DPL / 4; ++k) reinterpret_cast<float4*>(st)[k] = make_float4(S[4 * k], S[4 * k + 1], S[4 * k + 2], S[4 * k + 3]);
-    } else if (live) {
+    for (int c = 0; c < COLS; ++c) {
+        if (mycol + c >= vdim) break;
+        float* sr = st + (int64_t)(mycol + c) * dim;
+        if (vec_state) {
 #pragma unroll
-        for (int k = 0; k < DPL; ++k)
-            if (sub * DPL + k < dim) st[k] = S[k];
+            for (int k = 0; k < DPL / 4; ++k)
+                if (sub * DPL + 4 * k < dim)
+                    reinterpret_cast<float4*>(sr)[k] = make_float4(S[c][4 * k], S[c][4 * k + 1], S[c][4 * k + 2], S[c][4 * k + 3]);
+        } else {
+#pragma unroll
+            for (int k = 0; k < DPL; ++k)
+                if (sub * DPL + k < dim) sr[k] = S[c][k];
+        }
     }
+}
+
+// Decay pre-activations of many tokens -> decays, in place: a[t, h, c] <- exp(rate[h] * softplus(sign * (a + bias[h, c]))).
+__global__ void __launch_bounds__(256) channel_decay_kernel(float* __restrict__ a, int64_t stride, const float* __restrict__ rate,
+                                                            const float* __restrict__ bias, float sign, int cols, int dim) {
+    B200_PDL_SYNC();
+    const int64_t t = blockIdx.x;
+    for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < cols; c += gridDim.y * blockDim.x) {
+        float* p = a + t * stride + c;
+        *p = decay_of(*p, rate[c / dim], bias[c], sign);
+    }
+}
+
+template <typename T, bool CH, bool DELTA>
+int launch_matrix_state(const void* x, int64_t stride, int q_off, int k_off, int v_off, const float* write_in, const void* write_t,
+                        int64_t write_stride, const DecayIn& dec, float* state, const int32_t* state_slots, const int32_t* cu_q,
+                        const int32_t* cu_k, const int32_t* ctx_lens, float* out, int num_seqs, int H, int G, int dim, int vdim,
+                        float q_scale, cudaStream_t st) {
+#define MS_GO(DPL, LANES, COLS)                                                                                                    \
+    do {                                                                                                                           \
+        constexpr int GC = MS_THREADS / LANES * COLS;                                                                              \
+        B200_LAUNCH((matrix_state_kernel<T, DPL, LANES, COLS, CH, DELTA>), dim3(H, num_seqs, (vdim + GC - 1) / GC), MS_THREADS, 0, st,  \
+                    static_cast<const T*>(x), stride, q_off, k_off, v_off, write_in, static_cast<const T*>(write_t), write_stride, dec, \
+                    state, state_slots, cu_q, cu_k, ctx_lens, out, H, G, dim, vdim, q_scale);                                       \
+        return b200_launch_status(nullptr);                                                                                        \
+    } while (0)
+    if (dim <= 16) MS_GO(4, 4, 1);
+    if (dim <= 32) MS_GO(4, 8, 2);
+    if (dim <= 64) MS_GO(8, 8, 2);
+    if (dim <= 128) MS_GO(16, 8, 2);
+    if (dim <= 256) MS_GO(32, 8, 2);
+#undef MS_GO
+    return B200_EUNSUPPORTED;
 }
 
 // out[t, h, :] = c * o / sqrt(mean(o^2) + eps) * w * act(gate[t, h, :]) for o = x[t, h, :] (fp32), one warp per (token, head).
@@ -346,22 +467,46 @@ extern "C" int b200m_gated_delta(const void* x, int64_t stride, int q_off, int k
     if (!x || !ba || !rate || !dt_bias || !state || !state_slots || !out) return B200_EINVAL;
     if ((cu_q == nullptr) != (cu_k == nullptr) || (cu_q == nullptr && ctx_lens == nullptr)) return B200_EINVAL;
     if (num_heads <= 0 || num_kv_heads <= 0 || num_heads % num_kv_heads || dim <= 0 || vdim <= 0) return B200_EINVAL;
-    if (dim > 64 * GD_LANES) return B200_EUNSUPPORTED;
     if (num_seqs <= 0) return B200_OK;
-    cudaStream_t st = static_cast<cudaStream_t>(stream);
-    dim3 grid(num_heads, num_seqs, (vdim + GD_COLS - 1) / GD_COLS);
-#define GD_GO(N)                                                                                                                   \
-    B200M_DISPATCH(is32, B200_LAUNCH((gated_delta_kernel<T, N>), grid, GD_LANES * GD_COLS, 0, st, static_cast<const T*>(x), stride, q_off, \
-                                     k_off, v_off, ba, ba_stride, rate, dt_bias, state, state_slots, cu_q, cu_k, ctx_lens, out, num_heads, \
-                                     num_kv_heads, dim, vdim, q_scale))
-    const int dpl = (dim + GD_LANES - 1) / GD_LANES;
-    if (dpl <= 4) GD_GO(4);
-    else if (dpl <= 8) GD_GO(8);
-    else if (dpl <= 16) GD_GO(16);
-    else if (dpl <= 32) GD_GO(32);
-    else GD_GO(64);
-#undef GD_GO
+    const DecayIn dec{ba + num_heads, ba_stride, rate, dt_bias, 1.0f, 0};
+    B200M_DISPATCH(is32, return (launch_matrix_state<T, false, true>(x, stride, q_off, k_off, v_off, ba, nullptr, ba_stride, dec, state,
+                                                                     state_slots, cu_q, cu_k, ctx_lens, out, num_seqs, num_heads,
+                                                                     num_kv_heads, dim, vdim, q_scale, static_cast<cudaStream_t>(stream))));
+    return B200_EUNSUPPORTED;
+}
+
+extern "C" int b200m_channel_decay(float* a, int64_t stride, const float* rate, const float* bias, float sign, int n, int num_heads,
+                                   int dim, void* stream) {
+    if (!a || !rate || !bias || n < 0 || num_heads <= 0 || dim <= 0 || stride < (int64_t)num_heads * dim) return B200_EINVAL;
+    if (n == 0) return B200_OK;
+    const int cols = num_heads * dim;
+    B200_LAUNCH((channel_decay_kernel), dim3(n, (unsigned)((cols + 1023) / 1024)), 256, 0, static_cast<cudaStream_t>(stream), a, stride, rate, bias, sign,
+                cols, dim);
     return b200_launch_status(nullptr);
+}
+
+extern "C" int b200m_channel_state(const void* x, int64_t stride, int q_off, int k_off, int v_off, const void* write_in,
+                                   int64_t write_stride, const float* decay_in, int64_t decay_stride, const float* rate,
+                                   const float* decay_bias, float decay_sign, int decay_done, float* state,
+                                   const int32_t* state_slots, const int32_t* cu_q, const int32_t* cu_k, const int32_t* ctx_lens,
+                                   float* out, int num_seqs, int num_heads, int num_kv_heads, int dim, int vdim, float q_scale,
+                                   int is32, void* stream) {
+    if (!x || !decay_in || !state || !state_slots || !out || (!decay_done && (!rate || !decay_bias))) return B200_EINVAL;
+    if ((cu_q == nullptr) != (cu_k == nullptr) || (cu_q == nullptr && ctx_lens == nullptr)) return B200_EINVAL;
+    if (num_heads <= 0 || num_kv_heads <= 0 || num_heads % num_kv_heads || dim <= 0 || vdim <= 0) return B200_EINVAL;
+    if (num_seqs <= 0) return B200_OK;
+    const DecayIn dec{decay_in, decay_stride, rate, decay_bias, decay_sign, decay_done};
+    cudaStream_t st = static_cast<cudaStream_t>(stream);
+    if (write_in) {
+        B200M_DISPATCH(is32, return (launch_matrix_state<T, true, true>(x, stride, q_off, k_off, v_off, nullptr, write_in, write_stride, dec,
+                                                                        state, state_slots, cu_q, cu_k, ctx_lens, out, num_seqs, num_heads,
+                                                                        num_kv_heads, dim, vdim, q_scale, st)));
+    } else {
+        B200M_DISPATCH(is32, return (launch_matrix_state<T, true, false>(x, stride, q_off, k_off, v_off, nullptr, nullptr, 0, dec, state,
+                                                                         state_slots, cu_q, cu_k, ctx_lens, out, num_seqs, num_heads,
+                                                                         num_kv_heads, dim, vdim, q_scale, st)));
+    }
+    return B200_EUNSUPPORTED;
 }
 
 extern "C" int b200m_head_rmsnorm_gate(const float* x, const void* w, const void* gate, int64_t gate_stride, int act, void* out,

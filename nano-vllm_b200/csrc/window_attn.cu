@@ -3,7 +3,9 @@
 // Per token the cache holds one row [k (G * dim) | v (G * vdim)] per layer that owns a key/value projection; query head h
 // reads key/value head h / (H / G).  There is no rotation: position enters through the bias and the window only.
 //     s_ij = (q_i . k_j) * scale - slope[h] * (i - j),   visible: 0 <= i - j < window or j < keep_first   (window <= 0: every j <= i)
-//     p = softmax over the visible j,   out_i = sum_j p_ij v_j
+//     or, with chunk > 0, the j <= i of i's own chunk of positions: j >= i - i % chunk
+//     p = softmax over the visible j (with sinks: one more term exp(sink[h]) in the denominator, which has no value),
+//     out_i = sum_j p_ij v_j   (with a head gate: times sigmoid(gate[i, h]))
 // The kernels read whatever the cache rows hold: a design that rotates its keys stores them rotated (headnorm_rope_store_kernel).
 // Softmax statistics and the output accumulate in fp32 in both element types.
 //
@@ -20,6 +22,22 @@ namespace {
 
 constexpr int WA_WARPS = 8;
 constexpr int WA_TILE = 32;
+
+// What decides which keys a row sees and what happens to its weights beside the scores.
+struct RowRule {
+    int window, keep_first, chunk;
+    const float* sinks;           // [H] scores of the valueless extra term, or NULL
+    const void* gate;             // activation type, element (token, head) at token * gate_stride + head, or NULL
+    int64_t gate_stride;
+    // first key (kept first tokens aside) that the row at position pos sees; never decreasing in pos
+    __device__ __forceinline__ int first_key(int pos) const {
+        return chunk > 0 ? pos - pos % chunk : window > 0 ? max(0, pos - window + 1) : 0;
+    }
+    template <typename T>
+    __device__ __forceinline__ float gate_of(int64_t token, int h) const {
+        return gate ? sigmoidf_(ldf(static_cast<const T*>(gate) + token * gate_stride + h)) : 1.0f;
+    }
+};
 
 template <typename T>
 __global__ void __launch_bounds__(256) qk_norm_store_kernel(T* __restrict__ qkv, int64_t stride, int q_cols, int k_cols, int v_cols,
@@ -109,8 +127,8 @@ __global__ void __launch_bounds__(WA_WARPS * 32) window_attn_kernel(
     const T* __restrict__ cache, int row_elems, int v_off,
     const int32_t* __restrict__ block_tables, int bt_stride, int block_size,
     const int32_t* __restrict__ cu_q, const int32_t* __restrict__ cu_k, const int32_t* __restrict__ ctx_lens,
-    const float* __restrict__ slopes, int window, int keep_first, int vsets,
-    T* __restrict__ out, float* __restrict__ out32,   // [total_q, H * vsets * vdim]
+    const float* __restrict__ slopes, RowRule rule, int vsets,
+    T* __restrict__ out, float* __restrict__ out32, int64_t out_stride,       // [total_q, >= H * vsets * vdim]
     int H, int G, int dim, int vdim, float scale) {
     B200_PDL_SYNC();
     extern __shared__ float smem[];
@@ -133,16 +151,16 @@ __global__ void __launch_bounds__(WA_WARPS * 32) window_attn_kernel(
     const int pos = first + i;
     const int i_lo = pair0 / rep, i_hi = min(sp.qlen - 1, (pair0 + WA_WARPS - 1) / rep);
     const int kmax = first + i_hi + 1;                     // keys any warp of this CTA may see: [0, nkeep) and [kmin, kmax)
-    const int kmin = window > 0 ? max(0, first + i_lo - window + 1) : 0;
-    const int nkeep = min(keep_first, kmin);
-    const int my_lo = window > 0 ? max(0, pos - window + 1) : 0;
+    const int kmin = rule.first_key(first + i_lo);
+    const int nkeep = min(rule.keep_first, kmin);
+    const int my_lo = rule.first_key(pos);
     float* myq = qs + warp * dim;
     if (active) {
         const T* qr = q + (int64_t)(sp.q0 + i) * q_stride + (int64_t)h * dim;
         for (int c = lane; c < dim; c += 32) myq[c] = ldf(qr + c) * scale;
     }
     const float slope = (active && slopes) ? slopes[h] : 0.f;
-    float m = -INFINITY, l = 0.f;
+    float m = rule.sinks ? rule.sinks[h] : -INFINITY, l = rule.sinks ? 1.f : 0.f;
     float acc[OACC];
 #pragma unroll
     for (int k = 0; k < OACC; ++k) acc[k] = 0.f;
@@ -162,7 +180,7 @@ __global__ void __launch_bounds__(WA_WARPS * 32) window_attn_kernel(
         __syncthreads();
         const int u = u0 + lane;
         const int j = u < nkeep ? u : kmin + (u - nkeep);
-        const bool valid = active && lane < rows && j <= pos && (j >= my_lo || j < keep_first);
+        const bool valid = active && lane < rows && j <= pos && (j >= my_lo || j < rule.keep_first);
         if (__any_sync(0xffffffffu, valid)) {              // the tile holds at least one key this row sees
             float sc = -INFINITY;
             if (valid) {
@@ -190,8 +208,8 @@ __global__ void __launch_bounds__(WA_WARPS * 32) window_attn_kernel(
         }
     }
     if (active) {
-        const float inv = 1.0f / l;
-        const int64_t o = (((int64_t)(sp.q0 + i) * H + h) * vsets + vs) * vdim;
+        const float inv = rule.gate_of<T>(sp.q0 + i, h) / l;
+        const int64_t o = (int64_t)(sp.q0 + i) * out_stride + ((int64_t)h * vsets + vs) * vdim;
 #pragma unroll
         for (int k = 0; k < OACC; ++k) {
             const int c = lane + 32 * k;
@@ -218,7 +236,7 @@ int wa_ensure_smem(K kernel, size_t bytes) {
 template <typename T, int OACC>
 int launch_window_fma(const void* q, int64_t q_stride, const void* cache, int row_elems, int v_off, const int32_t* block_tables,
                       int bt_stride, int block_size, const int32_t* cu_q, const int32_t* cu_k, const int32_t* ctx_lens,
-                      const float* slopes, int window, int keep_first, int vsets, void* out, bool out_f32, int num_seqs, int max_q,
+                      const float* slopes, const RowRule& rule, int vsets, void* out, int64_t out_stride, bool out_f32, int num_seqs, int max_q,
                       int H, int G, int dim, int vdim, float scale, cudaStream_t stream) {
     const int D = dim + vdim;
     const size_t smem = sizeof(float) * ((size_t)WA_TILE * (D | 1) + (size_t)WA_WARPS * dim + WA_WARPS * WA_TILE);
@@ -227,8 +245,8 @@ int launch_window_fma(const void* q, int64_t q_stride, const void* cache, int ro
     dim3 grid((max_q * (H / G) + WA_WARPS - 1) / WA_WARPS, num_seqs, G * vsets);
     B200_LAUNCH((window_attn_kernel<T, OACC>), grid, WA_WARPS * 32, smem, stream, static_cast<const T*>(q), q_stride,
                 static_cast<const T*>(cache), row_elems, v_off, block_tables, bt_stride, block_size, cu_q, cu_k, ctx_lens, slopes,
-                window, keep_first, vsets, out_f32 ? nullptr : static_cast<T*>(out), out_f32 ? static_cast<float*>(out) : nullptr, H,
-                G, dim, vdim, scale);
+                rule, vsets, out_f32 ? nullptr : static_cast<T*>(out), out_f32 ? static_cast<float*>(out) : nullptr,
+                out_stride, H, G, dim, vdim, scale);
     return b200_launch_status(nullptr);
 }
 
@@ -277,8 +295,8 @@ template <int DK, int DV, bool KS, bool QREG, int BN>
 __global__ void __launch_bounds__(128) window_attn_mma_kernel(
     const __nv_bfloat16* __restrict__ q, int64_t q_stride, const __nv_bfloat16* __restrict__ cache, int row_elems, int v_off,
     const int32_t* __restrict__ block_tables, int bt_stride, int block_size, int bs_shift, const int32_t* __restrict__ cu_q,
-    const int32_t* __restrict__ cu_k, const int32_t* __restrict__ ctx_lens, const float* __restrict__ slopes, int window,
-    int keep_first, int vsets, __nv_bfloat16* __restrict__ out, float* __restrict__ out32, int H, int G, float scale, int splits,
+    const int32_t* __restrict__ cu_k, const int32_t* __restrict__ ctx_lens, const float* __restrict__ slopes, RowRule rule,
+    int vsets, __nv_bfloat16* __restrict__ out, float* __restrict__ out32, int64_t out_stride, int H, int G, float scale, int splits,
     float* __restrict__ part) {
     static_assert(!KS || BN == 64, "the key-sharing form shares out 64-key tiles");
     B200_PDL_SYNC();
@@ -301,11 +319,11 @@ __global__ void __launch_bounds__(128) window_attn_mma_kernel(
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, gq = lane >> 2, t4 = lane & 3;
     const int i_lo = row0 / rep, i_hi = min(sp.qlen - 1, (row0 + BM - 1) / rep);
     const int kmax = first + i_hi + 1;
-    const int kmin = window > 0 ? max(0, first + i_lo - window + 1) : 0;
+    const int kmin = rule.first_key(first + i_lo), keep_first = rule.keep_first;
     const int t_lo = kmin / BN, t_hi = (kmax + BN - 1) / BN;    // key tiles of the window: [t_lo, t_hi)
     // kept first tokens: their tiles below the window's are walked first.  Walked tile u is key tile u when u < n_keep, else
     // key tile t_lo + (u - n_keep).
-    const int n_keep = (window > 0 && keep_first > 0) ? min((keep_first + BN - 1) / BN, t_lo) : 0;
+    const int n_keep = keep_first > 0 ? min((keep_first + BN - 1) / BN, t_lo) : 0;
     int u_lo = 0, u_hi = n_keep + (t_hi - t_lo);
     if (splits > 1) {
         const int nt = u_hi;
@@ -366,7 +384,7 @@ __global__ void __launch_bounds__(128) window_attn_mma_kernel(
     // this thread's two rows: (warp * 16 +) gq and + 8
     const int wrow = KS ? 0 : warp * 16;                  // first row of this warp within the CTA
     const int wkey = KS ? warp * 16 : 0;                  // first key of this warp within a tile
-    int pos_r[2];
+    int pos_r[2], lo_r[2];
     float slope2[2];
     bool live[2];
 #pragma unroll
@@ -375,14 +393,15 @@ __global__ void __launch_bounds__(128) window_attn_mma_kernel(
         live[hh] = rr < nrows;
         const int i = live[hh] ? rr / rep : 0;
         pos_r[hh] = first + i;
+        lo_r[hh] = rule.first_key(first + i);
         slope2[hh] = (live[hh] && slopes) ? slopes[g * rep + (rr - i * rep)] * WM_LOG2E : 0.f;
     }
     // keys any row of this warp sees: [w_lo, w_hi]; keys every row of this warp sees: [f_lo, f_hi] (empty unless all 16 rows are live)
     const int wr0 = row0 + wrow, wr1 = min(nrows - 1, wr0 + 15);
     const int w_hi = wr0 < nrows ? first + wr1 / rep : -1;
-    const int w_lo = window > 0 ? max(0, first + wr0 / rep - window + 1) : 0;
+    const int w_lo = rule.first_key(first + wr0 / rep);
     const int f_hi = wr0 + 15 < nrows ? first + wr0 / rep : -1;
-    const int f_lo = window > 0 ? max(0, first + wr1 / rep - window + 1) : 0;
+    const int f_lo = rule.first_key(first + max(wr1, 0) / rep);
     const float scale2 = scale * WM_LOG2E;
 
     __syncthreads();                                                     // the queries are staged: keep this warp's fragments in registers
@@ -393,6 +412,14 @@ __global__ void __launch_bounds__(128) window_attn_mma_kernel(
         for (int kk = 0; kk < DK / 16; ++kk) wm_ldsm(a_base + kk * 32, qf[kk][0], qf[kk][1], qf[kk][2], qf[kk][3]);
     }
     float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};
+    if (rule.sinks != nullptr && split == 0 && (!KS || warp == 0)) {     // one holder of a row's keys starts with the sink's term
+#pragma unroll
+        for (int hh = 0; hh < 2; ++hh)
+            if (live[hh]) {
+                m_run[hh] = rule.sinks[g * rep + (row0 + wrow + gq + 8 * hh) % rep] * WM_LOG2E;
+                l_run[hh] = t4 == 0 ? 1.f : 0.f;                         // summed over the row's four lanes at the end
+            }
+    }
     float o[DV / 8][4];
 #pragma unroll
     for (int n = 0; n < DV / 8; ++n) o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.f;
@@ -459,7 +486,7 @@ __global__ void __launch_bounds__(128) window_attn_mma_kernel(
                         const int hh = e >> 1;
                         const int jj = j0 + n * 8 + 2 * t4 + (e & 1);
                         const int dist = pos_r[hh] - jj;
-                        const bool ok = live[hh] && dist >= 0 && (window <= 0 || dist < window || jj < keep_first);
+                        const bool ok = live[hh] && dist >= 0 && (jj >= lo_r[hh] || jj < keep_first);
                         const float v = ok ? fmaf(sc[n][e], scale2, -slope2[hh] * (float)dist) : -INFINITY;
                         sc[n][e] = v;
                         m_new[hh] = fmaxf(m_new[hh], v);
@@ -567,10 +594,11 @@ __global__ void __launch_bounds__(128) window_attn_mma_kernel(
                     pp[1] = L;
                 }
                 pp[2 + c] = a;
-            } else if (out32) {
-                out32[((int64_t)(sp.q0 + i) * HV + hv) * DV + c] = a / L;
             } else {
-                out[((int64_t)(sp.q0 + i) * HV + hv) * DV + c] = __float2bfloat16_rn(a / L);
+                const float r = a / L * rule.gate_of<__nv_bfloat16>(sp.q0 + i, g * rep + (rr - i * rep));
+                const int64_t ob = (int64_t)(sp.q0 + i) * out_stride + (int64_t)hv * DV + c;
+                if (out32) out32[ob] = r;
+                else out[ob] = __float2bfloat16_rn(r);
             }
         }
     } else {
@@ -591,8 +619,8 @@ __global__ void __launch_bounds__(128) window_attn_mma_kernel(
                 pp[2 + n * 8 + 2 * t4 + 1] = o[n][2 * hh + 1];
             }
         } else {
-            const float inv = 1.0f / l_run[hh];
-            const int64_t ob = ((int64_t)(sp.q0 + i) * HV + hv) * DV;
+            const float inv = rule.gate_of<__nv_bfloat16>(sp.q0 + i, g * rep + (rr - i * rep)) / l_run[hh];
+            const int64_t ob = (int64_t)(sp.q0 + i) * out_stride + (int64_t)hv * DV;
             if (out32) {
 #pragma unroll
                 for (int n = 0; n < DV / 8; ++n)
@@ -609,7 +637,7 @@ __global__ void __launch_bounds__(128) window_attn_mma_kernel(
 
 // out[s, h, :] = sum_k acc_k 2^(m_k - M) / sum_k l_k 2^(m_k - M) over the `splits` partials of a decode row
 __global__ void window_merge_kernel(const float* __restrict__ part, const int32_t* __restrict__ ctx_lens, __nv_bfloat16* __restrict__ out,
-                                    float* __restrict__ out32, int H, int vdim, int splits) {
+                                    float* __restrict__ out32, int64_t out_stride, RowRule rule, int H, int vdim, int splits) {
     B200_PDL_SYNC();
     const int s = blockIdx.x, h = blockIdx.y;
     if (ctx_lens[s] <= 0) return;
@@ -619,22 +647,22 @@ __global__ void window_merge_kernel(const float* __restrict__ part, const int32_
     for (int k = 0; k < splits; ++k) M = fmaxf(M, base[k * step]);
     float L = 0.f;
     for (int k = 0; k < splits; ++k) L += base[k * step + 1] * exp2f(base[k * step] - M);
-    const float inv = 1.0f / L;
+    const float inv = rule.gate_of<__nv_bfloat16>(s, h) / L;
     for (int c = threadIdx.x; c < vdim; c += blockDim.x) {
         float a = 0.f;
         for (int k = 0; k < splits; ++k) {
             const float mk = base[k * step];
             if (mk != -INFINITY) a = fmaf(base[k * step + 2 + c], exp2f(mk - M), a);
         }
-        if (out32) out32[((int64_t)s * H + h) * vdim + c] = a * inv;
-        else out[((int64_t)s * H + h) * vdim + c] = __float2bfloat16_rn(a * inv);
+        if (out32) out32[s * out_stride + (int64_t)h * vdim + c] = a * inv;
+        else out[s * out_stride + (int64_t)h * vdim + c] = __float2bfloat16_rn(a * inv);
     }
 }
 
 template <int DK, int DV, bool KS, bool QREG, int BN>
 int launch_window_mma_as(const void* q, int64_t q_stride, const void* cache, int row_elems, int v_off, const int32_t* block_tables,
                          int bt_stride, int block_size, const int32_t* cu_q, const int32_t* cu_k, const int32_t* ctx_lens,
-                         const float* slopes, int window, int keep_first, int vsets, void* out, bool out_f32, int num_seqs, int max_q,
+                         const float* slopes, const RowRule& rule, int vsets, void* out, int64_t out_stride, bool out_f32, int num_seqs, int max_q,
                          int H, int G, float scale, int splits, float* part, cudaStream_t stream) {
     using bf = __nv_bfloat16;
     constexpr int BM = KS ? 16 : WM_BM;
@@ -649,26 +677,26 @@ int launch_window_mma_as(const void* q, int64_t q_stride, const void* cache, int
     float* out32 = out_f32 ? static_cast<float*>(out) : nullptr;
     B200_LAUNCH((window_attn_mma_kernel<DK, DV, KS, QREG, BN>), grid, 128, smem, stream, static_cast<const bf*>(q), q_stride,
                 static_cast<const bf*>(cache), row_elems, v_off, block_tables, bt_stride, block_size, bs_shift, cu_q, cu_k, ctx_lens,
-                slopes, window, keep_first, vsets, out16, out32, H, G, scale, splits, part);
+                slopes, rule, vsets, out16, out32, out_stride, H, G, scale, splits, part);
     rc = b200_launch_status(nullptr);
     if (rc != B200_OK || splits <= 1) return rc;
-    B200_LAUNCH((window_merge_kernel), dim3(num_seqs, H * vsets), DV < 64 ? 32 : 64, 0, stream, part, ctx_lens, out16, out32, H * vsets, DV,
-                splits);
+    B200_LAUNCH((window_merge_kernel), dim3(num_seqs, H * vsets), DV < 64 ? 32 : 64, 0, stream, part, ctx_lens, out16, out32, out_stride, rule,
+                H * vsets, DV, splits);
     return b200_launch_status(nullptr);
 }
 
 template <int DK, int DV>
 int launch_window_mma(const void* q, int64_t q_stride, const void* cache, int row_elems, int v_off, const int32_t* block_tables,
                       int bt_stride, int block_size, const int32_t* cu_q, const int32_t* cu_k, const int32_t* ctx_lens,
-                      const float* slopes, int window, int keep_first, int vsets, void* out, bool out_f32, int num_seqs, int max_q, int H,
+                      const float* slopes, const RowRule& rule, int vsets, void* out, int64_t out_stride, bool out_f32, int num_seqs, int max_q, int H,
                       int G, float scale, int splits, float* part, cudaStream_t stream) {
     if (cu_q == nullptr && H / G <= 16)                   // single-token step: the four warps share every key tile
         return launch_window_mma_as<DK, DV, true, true, 64>(q, q_stride, cache, row_elems, v_off, block_tables, bt_stride, block_size, cu_q, cu_k,
-                                                  ctx_lens, slopes, window, keep_first, vsets, out, out_f32, num_seqs, max_q, H, G, scale, splits, part, stream);
+                                                  ctx_lens, slopes, rule, vsets, out, out_stride, out_f32, num_seqs, max_q, H, G, scale, splits, part, stream);
     // row-tiled form: query fragments are re-read from shared memory per key tile (measured faster than 32 more live registers)
     // (32-key tiles, which let four CTAs instead of two share an SM at 128-wide heads, were measured and are not faster)
     return launch_window_mma_as<DK, DV, false, false, 64>(q, q_stride, cache, row_elems, v_off, block_tables, bt_stride, block_size, cu_q, cu_k,
-                                                          ctx_lens, slopes, window, keep_first, vsets, out, out_f32, num_seqs, max_q, H, G, scale, splits, part, stream);
+                                                          ctx_lens, slopes, rule, vsets, out, out_stride, out_f32, num_seqs, max_q, H, G, scale, splits, part, stream);
 }
 
 }  // namespace
@@ -696,26 +724,30 @@ extern "C" int b200m_qk_norm_store(void* qkv, int64_t stride, int q_cols, int k_
 extern "C" int b200m_window_attention(const void* q, int64_t q_stride, const void* cache, int row_elems, int v_off,
                                       const int32_t* block_tables, int bt_stride, int block_size, const int32_t* cu_q,
                                       const int32_t* cu_k, const int32_t* ctx_lens, const float* slopes, int window, int keep_first,
-                                      int all_values, void* out, int total_q, int num_seqs, int max_q, int num_heads, int num_kv_heads,
+                                      int chunk, const float* sinks, const void* gate, int64_t gate_stride, int all_values, void* out, int64_t out_stride, int total_q, int num_seqs, int max_q, int num_heads, int num_kv_heads,
                                       int dim, int vdim, float scale, int is32, int flags, int splits, float* part, void* stream) {
     if (!q || !cache || !block_tables || !out || total_q < 0 || num_seqs < 0 || num_heads <= 0 || num_kv_heads <= 0 ||
-        num_heads % num_kv_heads || dim <= 0 || vdim <= 0 || block_size <= 0 || keep_first < 0)
+        num_heads % num_kv_heads || dim <= 0 || vdim <= 0 || block_size <= 0 || keep_first < 0 || chunk < 0 ||
+        (chunk > 0 && window > 0) || (gate && all_values))
         return B200_EINVAL;
     const int vsets = all_values ? num_kv_heads : 1;
+    if (out_stride < (int64_t)num_heads * vsets * vdim) return B200_EINVAL;
+    // kept first tokens belong to a window or a chunk: without one every earlier key is visible anyway
+    const RowRule rule{window, window > 0 || chunk > 0 ? keep_first : 0, chunk, sinks, gate, gate_stride};
     const bool out_f32 = (flags & 2) != 0 && !is32;
     if ((cu_q == nullptr) != (cu_k == nullptr) || (cu_q == nullptr && ctx_lens == nullptr)) return B200_EINVAL;
     if (total_q == 0 || num_seqs == 0 || max_q <= 0) return B200_OK;
     if (vdim > 512) return B200_EUNSUPPORTED;
     cudaStream_t st = static_cast<cudaStream_t>(stream);
     const bool aligned = ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(cache)) % 16 == 0) && q_stride % 8 == 0 &&
-                         row_elems % 8 == 0 && v_off % 8 == 0;
+                         row_elems % 8 == 0 && v_off % 8 == 0 && out_stride % 2 == 0 && reinterpret_cast<uintptr_t>(out) % 8 == 0;
     if (!is32 && !(flags & 1) && aligned && (dim == 32 || dim == 64 || dim == 128) && (vdim == 32 || vdim == 64 || vdim == 128)) {
         if (cu_q != nullptr || splits < 1) splits = 1;                  // keys are split for single-token steps only
         if (splits > 1 && !part) return B200_EINVAL;
 #define WA_MMA(DK, DV)                                                                                                           \
     if (dim == DK && vdim == DV)                                                                                                 \
         return launch_window_mma<DK, DV>(q, q_stride, cache, row_elems, v_off, block_tables, bt_stride, block_size, cu_q, cu_k,  \
-                                         ctx_lens, slopes, window, keep_first, vsets, out, out_f32, num_seqs, max_q, num_heads,  \
+                                         ctx_lens, slopes, rule, vsets, out, out_stride, out_f32, num_seqs, max_q, num_heads,  \
                                          num_kv_heads, scale, splits, part, st)
         WA_MMA(32, 32);
         WA_MMA(32, 64);
@@ -730,8 +762,8 @@ extern "C" int b200m_window_attention(const void* q, int64_t q_stride, const voi
     }
 #define WA_FMA(OACC)                                                                                                             \
     B200M_DISPATCH(is32, return (launch_window_fma<T, OACC>(q, q_stride, cache, row_elems, v_off, block_tables, bt_stride,       \
-                                                            block_size, cu_q, cu_k, ctx_lens, slopes, window, keep_first, vsets, \
-                                                            out, out_f32, num_seqs, max_q, num_heads, num_kv_heads, dim, vdim,   \
+                                                            block_size, cu_q, cu_k, ctx_lens, slopes, rule, vsets,               \
+                                                            out, out_stride, out_f32, num_seqs, max_q, num_heads, num_kv_heads, dim, vdim,   \
                                                             scale, st)))
     const int oacc = (vdim + 31) / 32;
     if (oacc <= 1) WA_FMA(1);
@@ -747,7 +779,8 @@ extern "C" int b200m_window_attention(const void* q, int64_t q_stride, const voi
 // Per-head query/key norm with a partial pair rotation, unit-RMS values, and the mixing of the heads' attention weights.
 //
 //   headnorm_rope_store_kernel : per token and head, q <- rms_norm(q) * wq (one weight vector of `dim` elements shared by all
-//                                heads), the pairs (2i, 2i + 1), i < rope_dims / 2, turned by the token's position, in place;
+//                                heads), the pairs (2i, 2i + 1) (or, by layout, (i, i + rope_dims / 2)), i < rope_dims / 2, turned
+//                                by the token's position, in place;
 //                                keys the same with wk and scattered to the token's cache row; values divided by their root mean
 //                                square (no weight) and scattered next to the keys.  One warp per head, fp32 throughout, one
 //                                rounding at the store.
@@ -762,7 +795,7 @@ template <typename T>
 __global__ void __launch_bounds__(128) headnorm_rope_store_kernel(T* __restrict__ x, int64_t stride, int q_off, int k_off, int v_off, int H,
                                                                   int G, int dim, int vdim, const T* __restrict__ wq,
                                                                   const T* __restrict__ wk, int v_unit, const float* __restrict__ cos_sin,
-                                                                  int rope_dims, const float* __restrict__ v_cos_sin, int v_rope_dims,
+                                                                  int layout, int rope_dims, const float* __restrict__ v_cos_sin, int v_rope_dims,
                                                                   const int64_t* __restrict__ positions,
                                                                   const int32_t* __restrict__ slots, T* __restrict__ cache, float eps) {
     B200_PDL_SYNC();
@@ -792,23 +825,23 @@ __global__ void __launch_bounds__(128) headnorm_rope_store_kernel(T* __restrict_
         }
         // queries and keys turn by one table, values (when asked for) by their own, over their own width
         const float* rcs = (is_q || is_k) ? cs : vcs;
-        const bool rot = rcs != nullptr;
-        const int half = ((is_q || is_k) ? rope_dims : v_rope_dims) / 2;
-        for (int c = 2 * lane; c < d; c += 64) {           // a lane owns whole pairs
-            float a = ldf(src + c) * rstd, b = c + 1 < d ? ldf(src + c + 1) * rstd : 0.f;
+        const int rdims = rcs == nullptr ? 0 : (is_q || is_k) ? rope_dims : v_rope_dims, half = rdims / 2;
+        const bool split = layout != 0 && (is_q || is_k);  // rotated pairs (i, i + half) instead of (2i, 2i + 1)
+        for (int p = lane; 2 * p < d; p += 32) {           // a lane owns whole pairs: the rotated ones first, then the rest two at a time
+            const int c0 = (split && p < half) ? p : 2 * p, c1 = (split && p < half) ? p + half : 2 * p + 1;
+            float a = ldf(src + c0) * rstd, b = c1 < d ? ldf(src + c1) * rstd : 0.f;
             if (w) {
-                a *= ldf(w + c);
-                if (c + 1 < d) b *= ldf(w + c + 1);
+                a *= ldf(w + c0);
+                if (c1 < d) b *= ldf(w + c1);
             }
-            const int i = c >> 1;
-            if (rot && i < half) {
-                const float co = rcs[i], si = rcs[half + i];
+            if (p < half) {
+                const float co = rcs[p], si = rcs[half + p];
                 const float ra = a * co - b * si, rb = b * co + a * si;
                 a = ra;
                 b = rb;
             }
-            stf(dst + c, a);
-            if (c + 1 < d) stf(dst + c + 1, b);
+            stf(dst + c0, a);
+            if (c1 < d) stf(dst + c1, b);
         }
     }
 }
@@ -938,7 +971,7 @@ __global__ void __launch_bounds__(256) head_mix_gate_kernel(const A* __restrict_
 
 extern "C" int b200m_headnorm_rope_store(void* x, int64_t stride, int q_off, int k_off, int v_off, int num_heads, int num_kv_heads, int dim,
                                          int vdim, const void* q_norm_w, const void* k_norm_w, int v_unit_norm, const float* cos_sin,
-                                         int rope_dims, const float* v_cos_sin, int v_rope_dims, const int64_t* positions,
+                                         int layout, int rope_dims, const float* v_cos_sin, int v_rope_dims, const int64_t* positions,
                                          const int32_t* slots, void* cache, int n, float eps, int is32, void* stream) {
     if (!x || n < 0 || num_heads <= 0 || num_kv_heads <= 0 || dim <= 0 || vdim <= 0 || rope_dims < 0 || rope_dims > dim || (rope_dims & 1))
         return B200_EINVAL;
@@ -949,7 +982,7 @@ extern "C" int b200m_headnorm_rope_store(void* x, int64_t stride, int q_off, int
     if (rope_dims == 0) cos_sin = nullptr;
     B200M_DISPATCH(is32, B200_LAUNCH((headnorm_rope_store_kernel<T>), n, 128, 0, static_cast<cudaStream_t>(stream), static_cast<T*>(x), stride,
                                      q_off, k_off, v_off, num_heads, num_kv_heads, dim, vdim, static_cast<const T*>(q_norm_w),
-                                     static_cast<const T*>(k_norm_w), v_unit_norm, cos_sin, rope_dims, v_cos_sin, v_rope_dims, positions, slots,
+                                     static_cast<const T*>(k_norm_w), v_unit_norm, cos_sin, layout, rope_dims, v_cos_sin, v_rope_dims, positions, slots,
                                      static_cast<T*>(cache), eps));
     return b200_launch_status(nullptr);
 }

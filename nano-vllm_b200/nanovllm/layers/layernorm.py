@@ -112,3 +112,38 @@ class GatedScaledSandwich:
         from .. import mixops
         return mixops.gated_add_normed_norm(x, y, gate, self.w_out, self.eps, self.dtype, next_scale=1.0 if then is not None else None,
                                             w_next=then.w_in32 if then is not None else None)
+
+
+class ParallelNorms:
+    """The two biased layer norms of a parallel block, ``x <- x + m (f1(ln1(x)) + f2(ln2(x)))`` over an fp32 stream: both read the same x,
+    so one pass forms the statistics once and writes both results.  ``advance`` closes a block (the scaled update with the summed
+    branches, then optionally another fp32 stream added on top) and opens the next one in the same pass.  ``second=False``: a block
+    with one branch."""
+
+    def __init__(self, width: int, eps: float, dtype, device, second: bool = True):
+        self.eps = eps
+        self.norm1 = (torch.ones(width, dtype=dtype, device=device), torch.zeros(width, dtype=dtype, device=device))
+        self.norm2 = (torch.ones(width, dtype=dtype, device=device), torch.zeros(width, dtype=dtype, device=device)) if second else None
+
+    def load(self, leaf: str, w: torch.Tensor) -> bool:
+        named = {"norm1": self.norm1[0], "norm1.b": self.norm1[1]}
+        if self.norm2 is not None:
+            named.update({"norm2": self.norm2[0], "norm2.b": self.norm2[1]})
+        if leaf not in named:
+            return False
+        named[leaf].copy_(w)
+        return True
+
+    def weight_shapes(self, width: int) -> dict:
+        return {k: (width,) for k in ("norm1", "norm1.b") + (("norm2", "norm2.b") if self.norm2 is not None else ())}
+
+    def open(self, x, add=None, rows_idx=None):
+        """(ln1(x), ln2(x) or None) after ``x += add``."""
+        from .. import mixops
+        return mixops.add_layernorm2(x, self.eps, add=add, norm1=self.norm1, norm2=self.norm2, rows_idx=rows_idx)
+
+    def advance(self, x, y, mult: float, then: "ParallelNorms | None" = None, add=None, x_out=None):
+        """x_out (None: x itself) = x + mult * y + add; with ``then`` also that block's (ln1, ln2) of the result."""
+        from .. import mixops
+        return mixops.add_layernorm2(x, self.eps, y=y, mult=mult, add=add, x_out=x_out, norm1=then.norm1 if then is not None else None,
+                                     norm2=then.norm2 if then is not None else None)

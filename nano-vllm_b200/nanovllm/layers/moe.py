@@ -31,10 +31,12 @@ from .. import mixops
 
 
 class GatedDenseFF:
-    def __init__(self, width: int, mlp: dict, dtype, device):
+    def __init__(self, width: int, mlp: dict, dtype, device, w_down=None):
+        """``w_down`` (a view): this block's columns of an output projection that another branch shares (``ParallelBranches``)."""
         self.ff = int(mlp["ff"])
         self.w_gate_up = torch.empty(2 * self.ff, width, dtype=dtype, device=device)
-        self.w_down = torch.empty(width, self.ff, dtype=dtype, device=device)
+        self.w_down = w_down if w_down is not None else torch.empty(width, self.ff, dtype=dtype, device=device)
+        assert self.w_down.shape == (width, self.ff)
 
     def load(self, leaf: str, w: torch.Tensor) -> bool:
         if leaf == "gate":
@@ -47,9 +49,16 @@ class GatedDenseFF:
             return False
         return True
 
+    def weight_shapes(self, width: int) -> dict:
+        return {"gate": (self.ff, width), "up": (self.ff, width), "down": (width, self.ff)}
+
+    def hidden(self, h: torch.Tensor, out: torch.Tensor | None = None) -> torch.Tensor:
+        """gelu_tanh(W_gate h) * (W_up h), the down projection's operand; ``out`` may be a row-strided view."""
+        return mixops.ff_act(F.linear(h, self.w_gate_up), mixops.FF_GELU_TANH_MUL, out=out)
+
     def forward(self, h: torch.Tensor):
         """-> (T tensor, None)"""
-        return F.linear(mixops.ff_act(F.linear(h, self.w_gate_up), mixops.FF_GELU_TANH_MUL), self.w_down), None
+        return F.linear(self.hidden(h), self.w_down), None
 
 
 class BiasedDenseFF:

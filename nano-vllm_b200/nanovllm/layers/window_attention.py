@@ -302,3 +302,99 @@ class RotatedValueAttention:
         o = mixops.head_rotate_gate(acc.view(n, self.heads, self.vdim), self.dtype, self.v_cos_sin, positions, sign=-1.0,
                                     layout=mixops.ROT_PAIRS)
         return F.linear(o, self.w_o), (proj[:, self.in_cols:] if self.extra else None)
+
+
+class ChunkedSinkAttention:
+    """Grouped-query attention inside chunks of positions, with a half-split partial rotation, a zero-score sink in the softmax and one
+    output gate per head.
+
+        q = W_q h + b_q,  k = W_k h + b_k,  v = W_v h + b_v
+        q[h] <- rotate(q[h], p),  k[g] <- rotate(k[g], p)             (the first rot.dims elements turn, pair (i, i + dims / 2) by p * base^(-2i / dims))
+        s[h, i, j] = (q_i[h] . k_j[h // (H / G)]) * scale,  visible j: j <= i and i // chunk == j // chunk      (no chunk size: every j <= i)
+        p_j = exp(s_j) / (exp(sink[h]) + sum_j exp(s_j)),  sink = 0
+        out = W_o concat_h (sigmoid(W_g h)_h * sum_j p_ij v_j)
+
+    One row ``[k (G * dim) | v (G * vdim)]`` per token, layer instance and page slot, keys after their rotation.  Chunks are counted
+    from the sequence's first position.  The gate's rows ride in the input projection (padded to whole 16-byte rows) and are applied in the
+    attention kernel's epilogue.  ``w_o`` may be a view into an output projection shared with another branch, whose operand ``mix`` fills.
+    """
+    kind = "attention"
+
+    def __init__(self, width: int, m: dict, eps: float, dtype, device, max_position: int, w_o=None):
+        from .rotary_embedding import build_banded_cos_sin
+        self.width, self.dtype, self.device = width, dtype, device
+        self.heads, self.kv_heads = int(m["heads"]), int(m["kv_heads"])
+        self.dim, self.vdim = int(m["dim"]), int(m["vdim"])
+        self.scale = float(m["scale"])
+        self.chunk = int((m.get("mask") or {}).get("size") or 0)            # 0: every earlier token is visible
+        if self.heads % self.kv_heads:
+            raise ValueError("heads must be a multiple of kv_heads")
+        if self.vdim > 512:
+            raise ValueError(f"vdim {self.vdim}: the attention kernels hold at most 512 output columns per query row")
+        H, G, d, vd = self.heads, self.kv_heads, self.dim, self.vdim
+        self.q_cols, self.k_cols, self.v_cols, self.out_cols = H * d, G * d, G * vd, H * vd
+        self.g_off = self.q_cols + self.k_cols + self.v_cols
+        self.in_cols = -(-(self.g_off + H) // 8) * 8
+        rot = m.get("rot")
+        self.cos_sin, self.rot_key = None, None
+        if rot and int(rot.get("dims") or 0) > 0:
+            dims, base = int(rot["dims"]), float(rot["base"])
+            if dims > d or dims % 2:
+                raise ValueError("rot.dims must be even and at most dim")
+            self.rot_key = ("halves", dims, base, max_position)
+            self.cos_sin = build_banded_cos_sin(dims, max_position, base, None, device)
+        self.w_in = torch.zeros(self.in_cols, width, dtype=dtype, device=device)     # [W_q ; W_k ; W_v ; W_g ; padding]: one GEMM reads h once
+        self.b_in = torch.zeros(self.in_cols, dtype=dtype, device=device)
+        self.w_o = w_o if w_o is not None else torch.empty(width, self.out_cols, dtype=dtype, device=device)
+        assert self.w_o.shape == (width, self.out_cols)
+        self.sinks = torch.zeros(H, dtype=torch.float32, device=device)
+        self.cache: list = []                                              # per instance [num_blocks * block_size, G * (dim + vdim)]
+        self.block_size = 0
+
+    @staticmethod
+    def operand_cols(m: dict) -> int:
+        return int(m["heads"]) * int(m["vdim"])
+
+    def load(self, leaf: str, w: torch.Tensor) -> bool:
+        q, k, v, g = self.q_cols, self.k_cols, self.v_cols, self.g_off
+        spans = {"q": (0, q), "k": (q, q + k), "v": (q + k, q + k + v), "g": (g, g + self.heads)}
+        if leaf in spans:
+            self.w_in[spans[leaf][0]:spans[leaf][1]].copy_(w)
+        elif leaf in ("q.b", "k.b", "v.b"):
+            self.b_in[spans[leaf[0]][0]:spans[leaf[0]][1]].copy_(w)
+        elif leaf == "o":
+            self.w_o.copy_(w)
+        else:
+            return False
+        return True
+
+    def weight_shapes(self, width: int) -> dict:
+        return {"q": (self.q_cols, width), "q.b": (self.q_cols,), "k": (self.k_cols, width), "k.b": (self.k_cols,), "v": (self.v_cols, width),
+                "v.b": (self.v_cols,), "g": (self.heads, width), "o": (width, self.out_cols)}
+
+    def cache_row_elems(self) -> int:
+        return self.k_cols + self.v_cols
+
+    def state_slot_bytes(self) -> int:
+        return 0
+
+    def bind(self, num_blocks: int, block_size: int, num_slots: int, copies: int = 1) -> None:
+        self.block_size = block_size
+        self.cache = [torch.zeros(num_blocks * block_size, self.cache_row_elems(), dtype=self.dtype, device=self.device) for _ in range(copies)]
+
+    def unbind(self) -> None:
+        self.cache = []
+
+    def mix(self, h: torch.Tensor, positions, ctx, spans: mixops.StepSpans, inst: int = 0, out: torch.Tensor | None = None) -> torch.Tensor:
+        """-> the output projection's operand [n, heads * vdim]."""
+        q, k = self.q_cols, self.k_cols
+        proj = F.linear(h, self.w_in, self.b_in)
+        cache = self.cache[inst]
+        mixops.headnorm_rope_store(proj, 0, q, q + k, self.heads, self.kv_heads, self.dim, self.vdim, None, None, False, self.cos_sin, positions,
+                                   ctx.slot_mapping, cache, 0.0, layout=mixops.ROT_HALVES)
+        return mixops.window_attention(proj, cache, ctx.block_tables, self.block_size, spans, self.heads, self.kv_heads, self.dim, self.vdim,
+                                       self.scale, None, 0, chunk=self.chunk, sinks=self.sinks,
+                                       gate=proj[:, self.g_off:self.g_off + self.heads], out=out)
+
+    def forward(self, h: torch.Tensor, positions, ctx, spans: mixops.StepSpans, inst: int = 0) -> torch.Tensor:
+        return F.linear(self.mix(h, positions, ctx, spans, inst), self.w_o)

@@ -163,6 +163,34 @@ def add_layernorm(x: torch.Tensor, weight: torch.Tensor | None, eps: float, a=No
     return out if norm else None
 
 
+def add_layernorm2(x: torch.Tensor, eps: float, y: torch.Tensor | None = None, mult: float = 1.0, add: torch.Tensor | None = None,
+                   x_out: torch.Tensor | None = None, norm1=None, norm2=None, rows_idx: torch.Tensor | None = None):
+    """x_out = x + mult * y + add (fp32; ``x_out`` None: in place), then up to two biased layer norms of the result, ``norm1`` and
+    ``norm2`` = (weight, bias): -> (out1, out2) in the weights' dtype, None where a norm is not given.  ``rows_idx`` (int32):
+    norms of these rows only, nothing is added."""
+    assert x.dtype == torch.float32 and x.is_contiguous() and x.dim() == 2
+    rows, cols = x.shape
+    ref = norm1[0] if norm1 else norm2[0] if norm2 else y
+    is32 = _is32(ref) if ref is not None else 1
+    _same(is32, y, *(norm1 or ()), *(norm2 or ()))
+    assert y is None or (y.is_contiguous() and y.shape == x.shape)
+    assert add is None or (add.dtype == torch.float32 and add.is_contiguous() and add.shape == x.shape)
+    if rows_idx is not None:
+        assert rows_idx.dtype == torch.int32 and y is None and add is None
+        rows = rows_idx.numel()
+    if x_out is None:
+        x_out = x if (y is not None or add is not None) else None
+    assert x_out is None or (x_out.dtype == torch.float32 and x_out.is_contiguous() and x_out.shape == x.shape)
+    outs, args = [], []
+    for n in (norm1, norm2):
+        assert n is None or (n[0].numel() == cols and n[1].numel() == cols)
+        o = torch.empty(rows, cols, dtype=n[0].dtype, device=x.device) if n else None
+        outs.append(o)
+        args += [_p(n[0]) if n else None, _p(n[1]) if n else None, _p(o)]
+    _call("b200m_add_layernorm2", x.data_ptr(), _p(x_out), _p(y), mult, _p(add), *args, _p(rows_idx), rows, cols, eps, is32, _stream())
+    return tuple(outs)
+
+
 def rmsnorm(x: torch.Tensor, weight: torch.Tensor, eps: float, cols: int | None = None, out: torch.Tensor | None = None) -> torch.Tensor:
     """RMS norm over the first ``cols`` elements of each row of a 2-D, unit-inner-stride x."""
     assert x.dim() == 2 and x.stride(1) == 1
@@ -215,11 +243,13 @@ def softcap_(x: torch.Tensor, cap: float) -> torch.Tensor:
 
 
 def ff_act(x: torch.Tensor, kind: int, out: torch.Tensor | None = None) -> torch.Tensor:
+    """``out`` may be a row-strided view (the feed-forward's columns of a wider operand)."""
     assert x.dim() == 2 and x.is_contiguous()
     n = x.shape[1] if kind in (FF_RELU2, FF_GELU_TANH) else x.shape[1] // 2
     if out is None:
         out = torch.empty(x.shape[0], n, dtype=x.dtype, device=x.device)
-    _call("b200m_ff_act", x.data_ptr(), out.data_ptr(), x.shape[0], n, kind, _is32(x), _stream())
+    assert out.dtype == x.dtype and out.shape == (x.shape[0], n) and out.stride(1) == 1
+    _call("b200m_ff_act", x.data_ptr(), out.data_ptr(), out.stride(0), x.shape[0], n, kind, _is32(x), _stream())
     return out
 
 
@@ -286,21 +316,28 @@ def qk_norm_store(qkv: torch.Tensor, q_cols: int, k_cols: int, v_cols: int, q_no
 def window_attention(q: torch.Tensor, cache: torch.Tensor, block_tables: torch.Tensor, block_size: int, spans: StepSpans,
                      heads: int, kv_heads: int, dim: int, vdim: int, scale: float, slopes: torch.Tensor | None = None,
                      window: int = 0, fma: bool = False, splits: int | None = None, keep_first: int = 0, all_values: bool = False,
-                     out_f32: bool = False) -> torch.Tensor:
+                     out_f32: bool = False, chunk: int = 0, sinks: torch.Tensor | None = None, gate: torch.Tensor | None = None,
+                     out: torch.Tensor | None = None) -> torch.Tensor:
     """q [n, >= heads * dim] (row-strided view), cache [slots, kv_heads * (dim + vdim)] -> [n, heads * vdim].
     ``keep_first``: the first tokens of a sequence that stay visible beyond the window.  ``all_values``: every head's weights
-    meet the values of every value head, -> [n, heads, kv_heads, vdim] (``head_mix_gate`` mixes them).  ``out_f32``: fp32 result."""
+    meet the values of every value head, -> [n, heads, kv_heads, vdim] (``head_mix_gate`` mixes them).  ``out_f32``: fp32 result.
+    ``chunk``: only keys of the query's own chunk of positions (instead of a window).  ``sinks`` (fp32 [heads]): scores of a valueless
+    extra term of each head's softmax.  ``gate`` ([n, heads], a row-strided view): head h times sigmoid(gate[:, h]).  ``out`` may be a row-strided view."""
     n = q.shape[0]
     assert q.dim() == 2 and q.stride(1) == 1 and cache.is_contiguous() and cache.shape[-1] == kv_heads * (dim + vdim)
     assert block_tables.dtype == torch.int32 and block_tables.stride(1) == 1
     assert slopes is None or (slopes.dtype == torch.float32 and slopes.numel() == heads)
     is32 = _is32(q)
     _same(is32, cache)
+    assert sinks is None or (sinks.dtype == torch.float32 and sinks.is_contiguous() and sinks.numel() == heads)
+    assert gate is None or (gate.dtype == q.dtype and gate.shape == (n, heads) and gate.stride(1) == 1 and not all_values)
     vsets = kv_heads if all_values else 1
-    out = torch.empty(n, heads * vsets * vdim, dtype=torch.float32 if out_f32 else q.dtype, device=q.device)
+    if out is None:
+        out = torch.empty(n, heads * vsets * vdim, dtype=torch.float32 if out_f32 else q.dtype, device=q.device)
+    assert out.dtype == (torch.float32 if out_f32 else q.dtype) and out.shape == (n, heads * vsets * vdim) and out.stride(1) == 1
     part, nsplit = None, 1
     if splits is None:
-        splits = window_attention_splits(spans, block_tables.shape[1] * block_size, window, kv_heads * vsets, keep_first) \
+        splits = window_attention_splits(spans, block_tables.shape[1] * block_size, chunk or window, kv_heads * vsets, keep_first) \
             if (not is32 and not fma) else 1
     if splits > 1 and spans.cu_q is None and not is32 and not fma:
         nsplit = splits
@@ -308,7 +345,8 @@ def window_attention(q: torch.Tensor, cache: torch.Tensor, block_tables: torch.T
         ops.LAUNCHES[0] += 1
     _call("b200m_window_attention", q.data_ptr(), q.stride(0), cache.data_ptr(), cache.shape[-1], kv_heads * dim,
           block_tables.data_ptr(), block_tables.stride(0), block_size, _p(spans.cu_q), _p(spans.cu_k), _p(spans.ctx_lens),
-          _p(slopes), int(window), int(keep_first), int(all_values), out.data_ptr(), n, spans.num_seqs, spans.max_q, heads, kv_heads,
+          _p(slopes), int(window), int(keep_first), int(chunk), _p(sinks), _p(gate), gate.stride(0) if gate is not None else 0, int(all_values),
+          out.data_ptr(), out.stride(0), n, spans.num_seqs, spans.max_q, heads, kv_heads,
           dim, vdim, scale, is32, int(fma) | (2 if out_f32 else 0), nsplit, _p(part), _stream())
     return out.view(n, heads, vsets, vdim) if all_values else out
 
@@ -326,11 +364,11 @@ def window_attention_splits(spans: StepSpans, max_keys: int, window: int, kv_hea
 def headnorm_rope_store(x: torch.Tensor, q_off: int, k_off: int, v_off: int, heads: int, kv_heads: int, dim: int, vdim: int,
                         q_norm: torch.Tensor | None, k_norm: torch.Tensor | None, v_unit_norm: bool, cos_sin: torch.Tensor | None,
                         positions: torch.Tensor | None, slots: torch.Tensor | None, cache: torch.Tensor | None, eps: float,
-                        v_cos_sin: torch.Tensor | None = None) -> None:
+                        v_cos_sin: torch.Tensor | None = None, layout: int = ROT_PAIRS) -> None:
     """x [n, cols] (q heads at q_off, key heads at k_off, value heads at v_off): per-head RMS norm of q and k with one weight of
     ``dim`` elements shared by the heads, pair rotation by cos_sin [positions, rope_dims] (fp32), q in place; normed, rotated keys
     and (unit-RMS) values into cache rows [k (kv_heads * dim) | v (kv_heads * vdim)] at ``slots``.  ``v_cos_sin`` (fp32
-    [positions, v_dims]): the value pairs are turned by the token's position before the store."""
+    [positions, v_dims]): the value pairs are turned by the token's position before the store.  ``layout``: which query / key elements pair."""
     assert x.dim() == 2 and x.stride(1) == 1
     is32 = _is32(x)
     _same(is32, q_norm, k_norm, cache)
@@ -345,7 +383,7 @@ def headnorm_rope_store(x: torch.Tensor, q_off: int, k_off: int, v_off: int, hea
     if cache is not None:
         assert cache.is_contiguous() and cache.shape[-1] == kv_heads * (dim + vdim) and slots.dtype == torch.int32 and slots.numel() == x.shape[0]
     _call("b200m_headnorm_rope_store", x.data_ptr(), x.stride(0), q_off, k_off, v_off, heads, kv_heads, dim, vdim, _p(q_norm), _p(k_norm),
-          int(v_unit_norm), _p(cos_sin), rope_dims, _p(v_cos_sin), v_dims, _p(positions), _p(slots), _p(cache), x.shape[0], eps, is32,
+          int(v_unit_norm), _p(cos_sin), int(layout), rope_dims, _p(v_cos_sin), v_dims, _p(positions), _p(slots), _p(cache), x.shape[0], eps, is32,
           _stream())
 
 
@@ -421,6 +459,32 @@ def gated_delta(x: torch.Tensor, q_off: int, k_off: int, v_off: int, ba: torch.T
     _call("b200m_gated_delta", x.data_ptr(), x.stride(0), q_off, k_off, v_off, ba.data_ptr(), ba.stride(0), rate.data_ptr(), dt_bias.data_ptr(),
           state.data_ptr(), state_slots.data_ptr(), _p(spans.cu_q), _p(spans.cu_k), _p(spans.ctx_lens), out.data_ptr(), spans.num_seqs, heads,
           kv_heads, dim, vdim, q_scale, _is32(x), _stream())
+    return out
+
+
+def channel_state(x: torch.Tensor, q_off: int, k_off: int, v_off: int, write: torch.Tensor | None, decay_in: torch.Tensor, rate: torch.Tensor,
+                  decay_bias: torch.Tensor, decay_sign: float, state: torch.Tensor, state_slots: torch.Tensor, spans: StepSpans, heads: int,
+                  kv_heads: int, dim: int, vdim: int, q_scale: float, decays_first: bool | None = None) -> torch.Tensor:
+    """Matrix state with one decay per head and key channel, exp(rate[h] * softplus(sign * (decay_in + decay_bias))).
+    x [n, cols]: q, k ([kv_heads, dim] at q_off / k_off) and v ([heads, vdim] at v_off); ``write`` [n, heads] (a row-strided view): delta rule
+    with unit-norm q and k; None: gated linear attention.  decay_in fp32 [n, heads * dim] (prompt steps, ``decays_first``: overwritten by the
+    decays, formed once instead of in every column tile of a head); state fp32 [slots, heads, vdim, dim] -> fp32 [n, heads, vdim]."""
+    n = x.shape[0]
+    is32 = _is32(x)
+    assert x.dim() == 2 and x.stride(1) == 1 and decay_in.dtype == torch.float32 and decay_in.stride(1) == 1 and decay_in.shape == (n, heads * dim)
+    assert rate.dtype == torch.float32 and decay_bias.dtype == torch.float32 and rate.numel() == heads and decay_bias.numel() == heads * dim
+    assert state.dtype == torch.float32 and state.is_contiguous() and state.shape[1:] == (heads, vdim, dim)
+    assert write is None or (write.shape == (n, heads) and write.stride(1) == 1)
+    _same(is32, write)
+    out = torch.empty(n, heads, vdim, dtype=torch.float32, device=x.device)
+    if decays_first is None:
+        decays_first = spans.max_q > 1
+    if decays_first:
+        _call("b200m_channel_decay", decay_in.data_ptr(), decay_in.stride(0), rate.data_ptr(), decay_bias.data_ptr(), decay_sign, n, heads, dim, _stream())
+    _call("b200m_channel_state", x.data_ptr(), x.stride(0), q_off, k_off, v_off, _p(write), write.stride(0) if write is not None else 0,
+          decay_in.data_ptr(), decay_in.stride(0), rate.data_ptr(), decay_bias.data_ptr(), decay_sign, int(decays_first), state.data_ptr(),
+          state_slots.data_ptr(), _p(spans.cu_q), _p(spans.cu_k), _p(spans.ctx_lens), out.data_ptr(), spans.num_seqs, heads, kv_heads, dim, vdim,
+          q_scale, is32, _stream())
     return out
 
 

@@ -53,8 +53,20 @@ def _fegolorn_config(raw: dict):
     return FegolornConfig(raw)
 
 
-MODELS = {"Qwen3ForCausalLM": _qwen3, "Qwen2ForCausalLM": _qwen3, "Tafopel": _tafopel, "Tipetar": _tipetar, "Musavik": _musavik, "Fegolorn": _fegolorn}
-CONFIG_READERS = {"Tafopel": _tafopel_config, "Tipetar": _tipetar_config, "Musavik": _musavik_config, "Fegolorn": _fegolorn_config}
+def _zuvepel():
+    from .zuvepel import ZuvepelForCausalLM
+    return ZuvepelForCausalLM
+
+
+def _zuvepel_config(raw: dict):
+    from .zuvepel import ZuvepelConfig
+    return ZuvepelConfig(raw)
+
+
+MODELS = {"Qwen3ForCausalLM": _qwen3, "Qwen2ForCausalLM": _qwen3, "Tafopel": _tafopel, "Tipetar": _tipetar, "Musavik": _musavik, "Fegolorn": _fegolorn,
+          "Zuvepel": _zuvepel}
+CONFIG_READERS = {"Tafopel": _tafopel_config, "Tipetar": _tipetar_config, "Musavik": _musavik_config, "Fegolorn": _fegolorn_config,
+                  "Zuvepel": _zuvepel_config}
 
 
 def architecture_of(hf_config) -> str:

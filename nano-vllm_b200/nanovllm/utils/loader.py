@@ -20,6 +20,12 @@ def load_model(model, path: str, allow_random: bool = False, seed: int = 0) -> i
             raise FileNotFoundError(f"no *.safetensors under {path}")
         return _random_fill(model, seed)
     from safetensors import safe_open
+    if hasattr(model, "declare_shapes"):           # sizes that only the checkpoint's tensors give: told before any tensor is placed
+        shapes = {}
+        for file in files:
+            with safe_open(file, "pt", "cpu") as f:
+                shapes.update({name: tuple(f.get_slice(name).get_shape()) for name in f.keys()})
+        model.declare_shapes(shapes)
     n = 0
     for file in files:
         with safe_open(file, "pt", "cpu") as f:
