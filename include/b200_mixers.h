@@ -215,8 +215,8 @@ int b200m_diag_scan(const void* u, int64_t u_stride, const float* gates, int64_t
  * state fp32 [slots, num_heads, vdim, dim]; out fp32 [n, num_heads, vdim].  dim <= 256. */
 int b200m_gated_delta(const void* x, int64_t stride, int q_off, int k_off, int v_off, const float* ba, int64_t ba_stride,
                       const float* rate, const float* dt_bias, float* state, const int32_t* state_slots, const int32_t* cu_q,
-                      const int32_t* cu_k, const int32_t* ctx_lens, float* out, int num_seqs, int num_heads, int num_kv_heads, int dim,
-                      int vdim, float q_scale, int is32, void* stream);
+                      const int32_t* cu_k, const int32_t* ctx_lens, float* out, int num_seqs, int max_q, int num_heads, int num_kv_heads,
+                      int dim, int vdim, float q_scale, int is32, void* stream);
 
 /* Matrix state with a decay per (head, key channel): g = exp(rate[h] * softplus(sign * (decay_in[t, h * dim + c] + decay_bias[h * dim + c]))),
  * or decay_in itself when decay_done (after b200m_channel_decay).  x and the state as for b200m_gated_delta.
@@ -226,8 +226,8 @@ int b200m_gated_delta(const void* x, int64_t stride, int q_off, int k_off, int v
 int b200m_channel_state(const void* x, int64_t stride, int q_off, int k_off, int v_off, const void* write_in, int64_t write_stride,
                         const float* decay_in, int64_t decay_stride, const float* rate, const float* decay_bias, float decay_sign,
                         int decay_done, float* state, const int32_t* state_slots, const int32_t* cu_q, const int32_t* cu_k,
-                        const int32_t* ctx_lens, float* out, int num_seqs, int num_heads, int num_kv_heads, int dim, int vdim,
-                        float q_scale, int is32, void* stream);
+                        const int32_t* ctx_lens, float* out, int num_seqs, int max_q, int num_heads, int num_kv_heads, int dim,
+                        int vdim, float q_scale, int is32, void* stream);
 
 /* a[t, h * dim + c] <- exp(rate[h] * softplus(sign * (a[t, h * dim + c] + bias[h * dim + c]))), fp32, in place: the decays of many tokens
  * formed once (b200m_channel_state forms them itself in each of a head's CTAs otherwise). */

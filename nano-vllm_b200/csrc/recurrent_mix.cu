@@ -378,11 +378,468 @@ __global__ void __launch_bounds__(256) channel_decay_kernel(float* __restrict__ 
     }
 }
 
+// ---------------------------------------------------------------------------------------------------------------------------
+// Prompt portions: the same rules four tokens at a time.  With P_t = g_1 ... g_t the products of a block's decays (per channel) and
+// R_s = g_(s+1) ... g_4, and S the state before the block,
+//     d_t = S^T (P_t k_t),  o'_t = S^T (P_t q_t),  A_ts = (R-weighted) k_s g_(s+1)..g_t . k_t,  B_ts likewise with q_t
+//     u_t = beta_t (v_t - d_t - sum_(s<t) A_ts u_s)       (linear attention: u_t = v_t)
+//     o_t = o'_t + sum_(s<=t) B_ts u_s,       S <- P_4 S + sum_s (R_s k_s) u_s
+// which is the token-by-token recurrence regrouped: only products of decays (never quotients), everything in fp32.  Four producer
+// warps form the scaled vectors and the small coefficient sets, a block each, up to two stages of sixteen tokens ahead; four consumer
+// warps hold the state (eight lanes x COLS columns, packed pairs of fp32 in 64-bit registers for the two-wide FMA) and do the four
+// tokens' column sums in one shuffle tree.  The two sides meet at named barriers (full / empty per stage).
+// ---------------------------------------------------------------------------------------------------------------------------
+constexpr int MB_T = 4, MB_BLOCKS = 4, MB_STAGE = MB_T * MB_BLOCKS, MB_LANES = 8, MB_THREADS = 256;
+
+__device__ __forceinline__ uint64_t fma2_(uint64_t a, uint64_t b, uint64_t c) {
+    uint64_t d;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+    return d;
+}
+__device__ __forceinline__ uint64_t mul2_(uint64_t a, uint64_t b) {
+    uint64_t d;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+    return d;
+}
+__device__ __forceinline__ uint64_t pack2_(float lo, float hi) {
+    uint64_t d;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(d) : "f"(lo), "f"(hi));
+    return d;
+}
+__device__ __forceinline__ float2 unpack2_(uint64_t v) {
+    float2 f;
+    asm("mov.b64 {%0, %1}, %2;" : "=f"(f.x), "=f"(f.y) : "l"(v));
+    return f;
+}
+template <int ID0>
+__device__ __forceinline__ void named_sync(int s) { asm volatile("bar.sync %0, %1;" ::"r"(ID0 + s), "n"(MB_THREADS) : "memory"); }
+template <int ID0>
+__device__ __forceinline__ void named_arrive(int s) { asm volatile("bar.arrive %0, %1;" ::"r"(ID0 + s), "n"(MB_THREADS) : "memory"); }
+
+// N consecutive elements as 32-bit words (two bf16 or one float each), without conversion, so that a load stays in flight until its use
+template <typename T, int N>
+struct RawCols {
+    static constexpr int W = (N * (int)sizeof(T) + 3) / 4;
+    uint32_t w[W];
+    __device__ __forceinline__ void zero() {
+#pragma unroll
+        for (int i = 0; i < W; ++i) w[i] = 0;
+    }
+    __device__ __forceinline__ void load(const T* p, int avail, bool vec) {      // the first `avail` elements; vec: all or none, aligned
+        zero();
+        if (vec) {
+            if (avail <= 0) return;
+            if constexpr (N * sizeof(T) == 4) w[0] = *reinterpret_cast<const uint32_t*>(p);
+            else if constexpr (N * sizeof(T) == 8) *reinterpret_cast<uint2*>(w) = *reinterpret_cast<const uint2*>(p);
+            else if constexpr (N * sizeof(T) % 16 == 0) {
+#pragma unroll
+                for (int i = 0; i < W / 4; ++i) {
+                    const uint4 v = reinterpret_cast<const uint4*>(p)[i];
+                    w[4 * i] = v.x, w[4 * i + 1] = v.y, w[4 * i + 2] = v.z, w[4 * i + 3] = v.w;
+                }
+            } else {
+                w[0] = *reinterpret_cast<const unsigned short*>(p);
+            }
+            return;
+        }
+#pragma unroll
+        for (int e = 0; e < N; ++e)
+            if (e < avail) {
+                if constexpr (sizeof(T) == 4) w[e] = reinterpret_cast<const uint32_t*>(p)[e];
+                else w[e / 2] |= (uint32_t)reinterpret_cast<const unsigned short*>(p)[e] << (16 * (e & 1));
+            }
+    }
+    __device__ __forceinline__ float at(int e) const {
+        if constexpr (sizeof(T) == 4) return __uint_as_float(w[e]);
+        else return (e & 1) ? bf16hi(w[e / 2]) : bf16lo(w[e / 2]);
+    }
+};
+
+template <int DPL, int COLS>
+struct BlockShape {
+    static constexpr int DP = MB_LANES * DPL, SEG = DPL + 4, ROW = MB_LANES * SEG, GC = 16 * COLS;
+    // one stage: P k, P q, R k rows of its tokens, the blocks' whole decays, values, coefficients (32 per block)
+    static constexpr int KD = 0, QD = MB_STAGE * ROW, KR = 2 * MB_STAGE * ROW, PE = 3 * MB_STAGE * ROW, VS = PE + MB_BLOCKS * ROW,
+                         CF = VS + MB_STAGE * GC, FLOATS = CF + MB_BLOCKS * 32;
+};
+// coefficient places of a block: key normalisers, query normalisers (* scale), A (t, s < t), B (t, s <= t), write strengths * key normaliser
+constexpr int CF_RK = 0, CF_RQ = 4, CF_A = 8, CF_B = 14, CF_W = 24;
+
+template <typename T, int DPL, int COLS, bool CH, bool DELTA>
+__global__ void __launch_bounds__(MB_THREADS) matrix_state_block_kernel(
+    const T* __restrict__ x, int64_t stride, int q_off, int k_off, int v_off, const float* __restrict__ write_in,
+    const T* __restrict__ write_t, int64_t write_stride, DecayIn dec, float* __restrict__ state, const int32_t* __restrict__ state_slots,
+    const int32_t* __restrict__ cu_q, const int32_t* __restrict__ cu_k, const int32_t* __restrict__ ctx_lens, float* __restrict__ out, int H,
+    int G, int dim, int vdim, float q_scale, int vec_x, int vec_g) {
+    B200_PDL_SYNC();
+    using SH = BlockShape<DPL, COLS>;
+    constexpr int FULL = 1, EMPTY = 3;
+    extern __shared__ __align__(16) float mb_smem[];       // two stages
+    const int h = blockIdx.x, s = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const SeqSpan sp = seq_span(cu_q, cu_k, ctx_lens, s);
+    if (sp.qlen <= 0) return;
+    const int nst = (sp.qlen + MB_STAGE - 1) / MB_STAGE;
+    const int col0 = blockIdx.z * SH::GC;
+    if (warp >= 4) {
+        // ---- producers: warp - 4 is the block of a stage, a lane owns CPL consecutive channels ----
+        constexpr int CPL = SH::DP / 32;
+        const int b = warp - 4, c0 = lane * CPL, avail = dim - c0;
+        const int at = (c0 / DPL) * SH::SEG + c0 % DPL;     // CPL <= DPL: a lane's channels stay inside one segment
+        const T* qp = x + q_off + (int64_t)(h / (H / G)) * dim + c0;
+        const T* kp = x + k_off + (int64_t)(h / (H / G)) * dim + c0;
+        const T* vp = x + v_off + (int64_t)h * vdim + col0;
+        const float* gp = CH ? dec.in + (int64_t)h * dim + c0 : dec.in + h;
+        const float rt = dec.done ? 0.f : dec.rate[h];
+        float gb[CH ? CPL : 1];
+#pragma unroll
+        for (int e = 0; e < (CH ? CPL : 1); ++e) gb[e] = dec.done ? 0.f : CH ? (e < avail ? dec.bias[(int64_t)h * dim + c0 + e] : 0.f) : dec.bias[h];
+        constexpr int VPL = MB_T * SH::GC / 32;             // value elements of a block per lane
+        RawCols<T, CPL> rk[MB_T], rq[MB_T];
+        RawCols<float, CH ? CPL : 1> rg[MB_T];
+        RawCols<T, 1> rv[VPL], rw;
+        float rwf = 0.f;
+        auto fetch = [&](int it) {
+            const int i0 = it * MB_STAGE + b * MB_T;
+#pragma unroll
+            for (int t = 0; t < MB_T; ++t) {
+                const int64_t row = sp.q0 + i0 + t;
+                const int have = i0 + t < sp.qlen ? avail : 0;
+                rk[t].load(kp + row * stride, have, vec_x);
+                rq[t].load(qp + row * stride, have, vec_x);
+                if constexpr (CH) rg[t].load(gp + row * dec.stride, have, vec_g);
+                else rg[t].load(gp + row * dec.stride, i0 + t < sp.qlen, false);
+            }
+#pragma unroll
+            for (int j = 0; j < VPL; ++j) {
+                const int e = lane + 32 * j, t = e / SH::GC, c = e % SH::GC;
+                rv[j].load(vp + (int64_t)(sp.q0 + i0 + t) * stride + c, i0 + t < sp.qlen && col0 + c < vdim, false);
+            }
+            if constexpr (DELTA) {
+                const bool have = lane < MB_T && i0 + lane < sp.qlen;
+                const int64_t row = sp.q0 + i0 + lane;
+                if (write_in) rwf = have ? write_in[row * write_stride + h] : 0.f;
+                else rw.load(write_t + row * write_stride + h, have, false);
+            }
+        };
+        fetch(0);
+        for (int it = 0; it < nst; ++it) {
+            const int i0 = it * MB_STAGE + b * MB_T, st = it & 1;
+            float* sm = mb_smem + st * SH::FLOATS;
+            if (it >= 2) named_sync<EMPTY>(st);
+            if (i0 < sp.qlen) {
+                float sum[32];
+#pragma unroll
+                for (int i = 0; i < 32; ++i) sum[i] = 0.f;
+                float pe[CPL], kd[MB_T][CPL], qd[MB_T][CPL], kr[MB_T][CPL];
+#pragma unroll
+                for (int e = 0; e < CPL; ++e) {
+                    float g[MB_T], k[MB_T], q[MB_T];
+#pragma unroll
+                    for (int t = 0; t < MB_T; ++t) {
+                        k[t] = rk[t].at(e);
+                        q[t] = rq[t].at(e);
+                        const float raw = rg[t].at(CH ? e : 0);
+                        g[t] = i0 + t >= sp.qlen ? 1.f : dec.done ? raw : decay_of(raw, rt, gb[CH ? e : 0], dec.sign);
+                    }
+                    float p = 1.f;
+#pragma unroll
+                    for (int t = 0; t < MB_T; ++t) {
+                        p *= g[t];
+                        kd[t][e] = p * k[t];
+                        qd[t][e] = p * q[t];
+                    }
+                    pe[e] = p;
+#pragma unroll
+                    for (int a = 0; a < MB_T; ++a) {
+                        float w = k[a];
+                        if constexpr (DELTA) {
+                            sum[CF_RK + a] = fmaf(k[a], k[a], sum[CF_RK + a]);
+                            sum[CF_RQ + a] = fmaf(q[a], q[a], sum[CF_RQ + a]);
+                        }
+                        sum[CF_B + a * (a + 1) / 2 + a] = fmaf(w, q[a], sum[CF_B + a * (a + 1) / 2 + a]);
+#pragma unroll
+                        for (int t = a + 1; t < MB_T; ++t) {
+                            w *= g[t];
+                            if constexpr (DELTA) sum[CF_A + t * (t - 1) / 2 + a] = fmaf(w, k[t], sum[CF_A + t * (t - 1) / 2 + a]);
+                            sum[CF_B + t * (t + 1) / 2 + a] = fmaf(w, q[t], sum[CF_B + t * (t + 1) / 2 + a]);
+                        }
+                        kr[a][e] = w;
+                    }
+                }
+                auto put = [&](float* dst, const float (&v)[CPL]) {
+                    if constexpr (CPL % 4 == 0) {
+#pragma unroll
+                        for (int e = 0; e < CPL; e += 4) *reinterpret_cast<float4*>(dst + e) = make_float4(v[e], v[e + 1], v[e + 2], v[e + 3]);
+                    } else if constexpr (CPL == 2) {
+                        *reinterpret_cast<float2*>(dst) = make_float2(v[0], v[1]);
+                    } else {
+                        dst[0] = v[0];
+                    }
+                };
+#pragma unroll
+                for (int t = 0; t < MB_T; ++t) {
+                    const int r = (b * MB_T + t) * SH::ROW + at;
+                    if constexpr (DELTA) put(sm + SH::KD + r, kd[t]);
+                    put(sm + SH::QD + r, qd[t]);
+                    put(sm + SH::KR + r, kr[t]);
+                }
+                put(sm + SH::PE + b * SH::ROW + at, pe);
+#pragma unroll
+                for (int j = 0; j < VPL; ++j) {
+                    const int e = lane + 32 * j;
+                    sm[SH::VS + b * MB_T * SH::GC + e] = rv[j].at(0);
+                }
+                // lane i ends with the warp's sum number i
+#pragma unroll
+                for (int o = 16; o > 0; o >>= 1) {
+                    const bool hi = lane & o;
+#pragma unroll
+                    for (int i = 0; i < o; ++i) {
+                        const float send = hi ? sum[i] : sum[i + o], keep = hi ? sum[i + o] : sum[i];
+                        sum[i] = keep + __shfl_xor_sync(0xffffffffu, send, o);
+                    }
+                }
+                float* cf = sm + SH::CF + b * 32;
+                if constexpr (DELTA) {
+                    const float r = 1.0f / sqrtf(sum[0] + 1e-6f);
+                    if (lane < 4) {
+                        const float beta = i0 + lane < sp.qlen ? sigmoidf_(write_in ? rwf : rw.at(0)) : 0.f;
+                        cf[CF_RK + lane] = r;
+                        cf[CF_W + lane] = beta * r;
+                    } else if (lane < 8) {
+                        cf[lane] = r * q_scale;
+                    } else if (lane < 24) {
+                        cf[lane] = sum[0];
+                    }
+                } else if (lane >= CF_B && lane < CF_B + 10) {
+                    cf[lane] = sum[0] * q_scale;
+                }
+            }
+            if (it + 1 < nst) fetch(it + 1);
+            named_arrive<FULL>(st);
+        }
+        return;
+    }
+    // ---- consumers ----
+    const int sub = lane & (MB_LANES - 1), grp = warp * 4 + (lane >> 3);
+    const int mycol = col0 + grp * COLS;
+    float* stp = state + ((int64_t)state_slots[s] * H + h) * vdim * dim + sub * DPL;
+    const bool has_hist = sp.klen - sp.qlen > 0, vec_state = dim % 4 == 0;
+    uint64_t S[COLS][DPL / 2];
+#pragma unroll
+    for (int c = 0; c < COLS; ++c) {
+        const bool have = has_hist && mycol + c < vdim;
+        const float* sr = stp + (int64_t)(mycol + c) * dim;
+#pragma unroll
+        for (int k = 0; k < DPL / 4; ++k) {
+            float4 f = make_float4(0.f, 0.f, 0.f, 0.f);
+            const int d = sub * DPL + 4 * k;
+            if (have && vec_state) {
+                if (d < dim) f = reinterpret_cast<const float4*>(sr)[k];
+            } else if (have) {
+                if (d < dim) f.x = sr[4 * k];
+                if (d + 1 < dim) f.y = sr[4 * k + 1];
+                if (d + 2 < dim) f.z = sr[4 * k + 2];
+                if (d + 3 < dim) f.w = sr[4 * k + 3];
+            }
+            S[c][2 * k] = pack2_(f.x, f.y);
+            S[c][2 * k + 1] = pack2_(f.z, f.w);
+        }
+    }
+    // After the shuffle tree a lane holds, for one column, either all four d sums or all four o sums (delta rule), or the o sums
+    // of some tokens (linear attention).
+    constexpr int KINDS = DELTA ? 2 : 1, COMBOS = COLS * KINDS;          // 8, 4 or 2 sets of four sums
+    constexpr int OT = DELTA ? 4 : COMBOS * 4 / 8;                        // linear attention: 16 or 8 sums spread over the eight lanes
+    const int own = DELTA ? (sub & (COMBOS - 1)) / 2 : sub / (8 / COLS);   // this lane's column
+    const int ocol = mycol + own;
+    const bool odd = sub & 1;
+    for (int it = 0; it < nst; ++it) {
+        const int st = it & 1, i0 = it * MB_STAGE;
+        const float* sm = mb_smem + st * SH::FLOATS;
+        named_sync<FULL>(st);
+        for (int b = 0; b < MB_BLOCKS && i0 + b * MB_T < sp.qlen; ++b) {
+            const float* cf = sm + SH::CF + b * 32;
+            float w[COMBOS][MB_T];
+#pragma unroll
+            for (int t = 0; t < MB_T; ++t) {
+                const float* kd = sm + SH::KD + (b * MB_T + t) * SH::ROW + sub * SH::SEG;
+                const float* qd = sm + SH::QD + (b * MB_T + t) * SH::ROW + sub * SH::SEG;
+                uint64_t a[COLS][KINDS];
+#pragma unroll
+                for (int k = 0; k < DPL / 4; ++k) {
+                    const ulonglong2 q2 = *reinterpret_cast<const ulonglong2*>(qd + 4 * k);
+                    ulonglong2 k2 = q2;
+                    if constexpr (DELTA) k2 = *reinterpret_cast<const ulonglong2*>(kd + 4 * k);
+#pragma unroll
+                    for (int c = 0; c < COLS; ++c) {
+                        if constexpr (DELTA) {
+                            a[c][0] = k == 0 ? mul2_(S[c][0], k2.x) : fma2_(S[c][2 * k], k2.x, a[c][0]);
+                            a[c][0] = fma2_(S[c][2 * k + 1], k2.y, a[c][0]);
+                        }
+                        a[c][KINDS - 1] = k == 0 ? mul2_(S[c][0], q2.x) : fma2_(S[c][2 * k], q2.x, a[c][KINDS - 1]);
+                        a[c][KINDS - 1] = fma2_(S[c][2 * k + 1], q2.y, a[c][KINDS - 1]);
+                    }
+                }
+#pragma unroll
+                for (int c = 0; c < COLS; ++c)
+#pragma unroll
+                    for (int n = 0; n < KINDS; ++n) {
+                        const float2 f = unpack2_(a[c][n]);
+                        w[c * KINDS + n][t] = f.x + f.y;
+                    }
+            }
+            float u[COLS][MB_T];
+            const float* vs = sm + SH::VS + b * MB_T * SH::GC + grp * COLS;
+            if constexpr (DELTA) {
+                if constexpr (COMBOS == 4) {
+#pragma unroll
+                    for (int i = 0; i < 4; ++i)
+#pragma unroll
+                        for (int t = 0; t < MB_T; ++t) w[i][t] += __shfl_xor_sync(0xffffffffu, w[i][t], 4);
+                }
+#pragma unroll
+                for (int o = COMBOS / 2; o > 0; o >>= 1) {
+                    const bool hi = sub & o;
+#pragma unroll
+                    for (int i = 0; i < o; ++i)
+#pragma unroll
+                        for (int t = 0; t < MB_T; ++t) {
+                            const float send = hi ? w[i][t] : w[i + o][t], keep = hi ? w[i + o][t] : w[i][t];
+                            w[i][t] = keep + __shfl_xor_sync(0xffffffffu, send, o);
+                        }
+                }
+                float mu[MB_T];                            // u times the key's normaliser (correct on the lanes with the d sums)
+#pragma unroll
+                for (int t = 0; t < MB_T; ++t) {
+                    float acc = w[0][t];
+#pragma unroll
+                    for (int a = 0; a < t; ++a) acc = fmaf(cf[CF_A + t * (t - 1) / 2 + a], mu[a], acc);
+                    mu[t] = cf[CF_W + t] * fmaf(-cf[CF_RK + t], acc, vs[t * SH::GC + own]);
+                }
+#pragma unroll
+                for (int t = 0; t < MB_T; ++t)
+#pragma unroll
+                    for (int c = 0; c < COLS; ++c) u[c][t] = __shfl_sync(0xffffffffu, mu[t], (lane & ~7) | (2 * c));
+#pragma unroll
+                for (int t = 0; t < MB_T; ++t) {
+                    const float e = __shfl_xor_sync(0xffffffffu, mu[t], 1);
+                    mu[t] = odd ? e : mu[t];
+                }
+#pragma unroll
+                for (int t = 0; t < MB_T; ++t) {
+                    float acc = w[0][t];
+#pragma unroll
+                    for (int a = 0; a <= t; ++a) acc = fmaf(cf[CF_B + t * (t + 1) / 2 + a], mu[a], acc);
+                    const int i = i0 + b * MB_T + t;
+                    if (odd && sub < COMBOS && ocol < vdim && i < sp.qlen) out[((int64_t)(sp.q0 + i) * H + h) * vdim + ocol] = acc * cf[CF_RQ + t];
+                }
+            } else {
+#pragma unroll
+                for (int t = 0; t < MB_T; ++t)
+#pragma unroll
+                    for (int c = 0; c < COLS; ++c) u[c][t] = vs[t * SH::GC + c];
+                // 4 * COLS sums as eight sets of OT: set number = column * (8 / COLS) + token / OT
+                float r[8][OT];
+#pragma unroll
+                for (int i = 0; i < 8; ++i)
+#pragma unroll
+                    for (int j = 0; j < OT; ++j) r[i][j] = w[i / (8 / COLS)][(i % (8 / COLS)) * OT + j];
+#pragma unroll
+                for (int o = 4; o > 0; o >>= 1) {
+                    const bool hi = sub & o;
+#pragma unroll
+                    for (int i = 0; i < o; ++i)
+#pragma unroll
+                        for (int j = 0; j < OT; ++j) {
+                            const float send = hi ? r[i][j] : r[i + o][j], keep = hi ? r[i + o][j] : r[i][j];
+                            r[i][j] = keep + __shfl_xor_sync(0xffffffffu, send, o);
+                        }
+                }
+                float mv[MB_T];
+#pragma unroll
+                for (int t = 0; t < MB_T; ++t) mv[t] = vs[t * SH::GC + own];
+#pragma unroll
+                for (int j = 0; j < OT; ++j) {
+                    const int t = (sub % (8 / COLS)) * OT + j, i = i0 + b * MB_T + t;
+                    float acc = r[0][j] * q_scale;
+#pragma unroll
+                    for (int a = 0; a < MB_T; ++a)
+                        if (a <= t) acc = fmaf(cf[CF_B + t * (t + 1) / 2 + a], mv[a], acc);
+                    if (ocol < vdim && i < sp.qlen) out[((int64_t)(sp.q0 + i) * H + h) * vdim + ocol] = acc;
+                }
+            }
+            const float* pe = sm + SH::PE + b * SH::ROW + sub * SH::SEG;
+            const float* kr = sm + SH::KR + b * MB_T * SH::ROW + sub * SH::SEG;
+#pragma unroll
+            for (int k = 0; k < DPL / 4; ++k) {
+                const ulonglong2 p2 = *reinterpret_cast<const ulonglong2*>(pe + 4 * k);
+#pragma unroll
+                for (int c = 0; c < COLS; ++c) {
+                    S[c][2 * k] = mul2_(S[c][2 * k], p2.x);
+                    S[c][2 * k + 1] = mul2_(S[c][2 * k + 1], p2.y);
+                }
+#pragma unroll
+                for (int t = 0; t < MB_T; ++t) {
+                    const ulonglong2 r2 = *reinterpret_cast<const ulonglong2*>(kr + t * SH::ROW + 4 * k);
+#pragma unroll
+                    for (int c = 0; c < COLS; ++c) {
+                        const uint64_t uu = pack2_(u[c][t], u[c][t]);
+                        S[c][2 * k] = fma2_(r2.x, uu, S[c][2 * k]);
+                        S[c][2 * k + 1] = fma2_(r2.y, uu, S[c][2 * k + 1]);
+                    }
+                }
+            }
+        }
+        if (it + 2 < nst) named_arrive<EMPTY>(st);
+    }
+#pragma unroll
+    for (int c = 0; c < COLS; ++c) {
+        if (mycol + c >= vdim) break;
+        float* sr = stp + (int64_t)(mycol + c) * dim;
+#pragma unroll
+        for (int k = 0; k < DPL / 4; ++k) {
+            const float2 lo = unpack2_(S[c][2 * k]), hi = unpack2_(S[c][2 * k + 1]);
+            const int d = sub * DPL + 4 * k;
+            if (vec_state) {
+                if (d < dim) reinterpret_cast<float4*>(sr)[k] = make_float4(lo.x, lo.y, hi.x, hi.y);
+            } else {
+                if (d < dim) sr[4 * k] = lo.x;
+                if (d + 1 < dim) sr[4 * k + 1] = lo.y;
+                if (d + 2 < dim) sr[4 * k + 2] = hi.x;
+                if (d + 3 < dim) sr[4 * k + 3] = hi.y;
+            }
+        }
+    }
+}
+
 template <typename T, bool CH, bool DELTA>
 int launch_matrix_state(const void* x, int64_t stride, int q_off, int k_off, int v_off, const float* write_in, const void* write_t,
                         int64_t write_stride, const DecayIn& dec, float* state, const int32_t* state_slots, const int32_t* cu_q,
-                        const int32_t* cu_k, const int32_t* ctx_lens, float* out, int num_seqs, int H, int G, int dim, int vdim,
+                        const int32_t* cu_k, const int32_t* ctx_lens, float* out, int num_seqs, int max_q, int H, int G, int dim, int vdim,
                         float q_scale, cudaStream_t st) {
+    if (dim > 256) return B200_EUNSUPPORTED;
+#define MB_GO(DPL, COLS)                                                                                                           \
+    do {                                                                                                                           \
+        using SH = BlockShape<DPL, COLS>;                                                                                          \
+        constexpr int CPL = SH::DP / 32;                                                                                           \
+        const size_t smem = sizeof(float) * 2 * SH::FLOATS;                                                                        \
+        static B200SmemOptIn opt;                                                                                                  \
+        if (opt.ensure(matrix_state_block_kernel<T, DPL, COLS, CH, DELTA>, smem) != cudaSuccess) return B200_ECUDA;                \
+        const int vx = dim % CPL == 0 && stride % CPL == 0 && q_off % CPL == 0 && k_off % CPL == 0 &&                              \
+                       reinterpret_cast<uintptr_t>(x) % 16 == 0;                                                                   \
+        const int vg = CH && dim % CPL == 0 && dec.stride % (CPL < 4 ? CPL : 4) == 0 && reinterpret_cast<uintptr_t>(dec.in) % 16 == 0;  \
+        B200_LAUNCH((matrix_state_block_kernel<T, DPL, COLS, CH, DELTA>), dim3(H, num_seqs, (vdim + SH::GC - 1) / SH::GC), MB_THREADS,  \
+                    smem, st, static_cast<const T*>(x), stride, q_off, k_off, v_off, write_in, static_cast<const T*>(write_t),     \
+                    write_stride, dec, state, state_slots, cu_q, cu_k, ctx_lens, out, H, G, dim, vdim, q_scale, vx, vg);           \
+        return b200_launch_status(nullptr);                                                                                        \
+    } while (0)
+    if (cu_q != nullptr && max_q > MB_T) {                  // prompt portions: four tokens at a time
+        if (dim <= 32) MB_GO(4, 4);
+        if (dim <= 64) MB_GO(8, 4);
+        if (dim <= 128) MB_GO(16, 4);
+        MB_GO(32, 2);
+    }
+#undef MB_GO
 #define MS_GO(DPL, LANES, COLS)                                                                                                    \
     do {                                                                                                                           \
         constexpr int GC = MS_THREADS / LANES * COLS;                                                                              \
@@ -462,7 +919,7 @@ extern "C" int b200m_diag_scan(const void* u, int64_t u_stride, const float* gat
 
 extern "C" int b200m_gated_delta(const void* x, int64_t stride, int q_off, int k_off, int v_off, const float* ba, int64_t ba_stride,
                                  const float* rate, const float* dt_bias, float* state, const int32_t* state_slots, const int32_t* cu_q,
-                                 const int32_t* cu_k, const int32_t* ctx_lens, float* out, int num_seqs, int num_heads, int num_kv_heads,
+                                 const int32_t* cu_k, const int32_t* ctx_lens, float* out, int num_seqs, int max_q, int num_heads, int num_kv_heads,
                                  int dim, int vdim, float q_scale, int is32, void* stream) {
     if (!x || !ba || !rate || !dt_bias || !state || !state_slots || !out) return B200_EINVAL;
     if ((cu_q == nullptr) != (cu_k == nullptr) || (cu_q == nullptr && ctx_lens == nullptr)) return B200_EINVAL;
@@ -470,7 +927,7 @@ extern "C" int b200m_gated_delta(const void* x, int64_t stride, int q_off, int k
     if (num_seqs <= 0) return B200_OK;
     const DecayIn dec{ba + num_heads, ba_stride, rate, dt_bias, 1.0f, 0};
     B200M_DISPATCH(is32, return (launch_matrix_state<T, false, true>(x, stride, q_off, k_off, v_off, ba, nullptr, ba_stride, dec, state,
-                                                                     state_slots, cu_q, cu_k, ctx_lens, out, num_seqs, num_heads,
+                                                                     state_slots, cu_q, cu_k, ctx_lens, out, num_seqs, max_q, num_heads,
                                                                      num_kv_heads, dim, vdim, q_scale, static_cast<cudaStream_t>(stream))));
     return B200_EUNSUPPORTED;
 }
@@ -489,7 +946,7 @@ extern "C" int b200m_channel_state(const void* x, int64_t stride, int q_off, int
                                    int64_t write_stride, const float* decay_in, int64_t decay_stride, const float* rate,
                                    const float* decay_bias, float decay_sign, int decay_done, float* state,
                                    const int32_t* state_slots, const int32_t* cu_q, const int32_t* cu_k, const int32_t* ctx_lens,
-                                   float* out, int num_seqs, int num_heads, int num_kv_heads, int dim, int vdim, float q_scale,
+                                   float* out, int num_seqs, int max_q, int num_heads, int num_kv_heads, int dim, int vdim, float q_scale,
                                    int is32, void* stream) {
     if (!x || !decay_in || !state || !state_slots || !out || (!decay_done && (!rate || !decay_bias))) return B200_EINVAL;
     if ((cu_q == nullptr) != (cu_k == nullptr) || (cu_q == nullptr && ctx_lens == nullptr)) return B200_EINVAL;
@@ -499,11 +956,11 @@ extern "C" int b200m_channel_state(const void* x, int64_t stride, int q_off, int
     cudaStream_t st = static_cast<cudaStream_t>(stream);
     if (write_in) {
         B200M_DISPATCH(is32, return (launch_matrix_state<T, true, true>(x, stride, q_off, k_off, v_off, nullptr, write_in, write_stride, dec,
-                                                                        state, state_slots, cu_q, cu_k, ctx_lens, out, num_seqs, num_heads,
+                                                                        state, state_slots, cu_q, cu_k, ctx_lens, out, num_seqs, max_q, num_heads,
                                                                         num_kv_heads, dim, vdim, q_scale, st)));
     } else {
         B200M_DISPATCH(is32, return (launch_matrix_state<T, true, false>(x, stride, q_off, k_off, v_off, nullptr, nullptr, 0, dec, state,
-                                                                         state_slots, cu_q, cu_k, ctx_lens, out, num_seqs, num_heads,
+                                                                         state_slots, cu_q, cu_k, ctx_lens, out, num_seqs, max_q, num_heads,
                                                                          num_kv_heads, dim, vdim, q_scale, st)));
     }
     return B200_EUNSUPPORTED;

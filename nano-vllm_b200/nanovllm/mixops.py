@@ -457,8 +457,8 @@ def gated_delta(x: torch.Tensor, q_off: int, k_off: int, v_off: int, ba: torch.T
     assert state.dtype == torch.float32 and state.is_contiguous() and state.shape[1:] == (heads, vdim, dim)
     out = torch.empty(n, heads, vdim, dtype=torch.float32, device=x.device)
     _call("b200m_gated_delta", x.data_ptr(), x.stride(0), q_off, k_off, v_off, ba.data_ptr(), ba.stride(0), rate.data_ptr(), dt_bias.data_ptr(),
-          state.data_ptr(), state_slots.data_ptr(), _p(spans.cu_q), _p(spans.cu_k), _p(spans.ctx_lens), out.data_ptr(), spans.num_seqs, heads,
-          kv_heads, dim, vdim, q_scale, _is32(x), _stream())
+          state.data_ptr(), state_slots.data_ptr(), _p(spans.cu_q), _p(spans.cu_k), _p(spans.ctx_lens), out.data_ptr(), spans.num_seqs, spans.max_q,
+          heads, kv_heads, dim, vdim, q_scale, _is32(x), _stream())
     return out
 
 
@@ -483,7 +483,7 @@ def channel_state(x: torch.Tensor, q_off: int, k_off: int, v_off: int, write: to
         _call("b200m_channel_decay", decay_in.data_ptr(), decay_in.stride(0), rate.data_ptr(), decay_bias.data_ptr(), decay_sign, n, heads, dim, _stream())
     _call("b200m_channel_state", x.data_ptr(), x.stride(0), q_off, k_off, v_off, _p(write), write.stride(0) if write is not None else 0,
           decay_in.data_ptr(), decay_in.stride(0), rate.data_ptr(), decay_bias.data_ptr(), decay_sign, int(decays_first), state.data_ptr(),
-          state_slots.data_ptr(), _p(spans.cu_q), _p(spans.cu_k), _p(spans.ctx_lens), out.data_ptr(), spans.num_seqs, heads, kv_heads, dim, vdim,
+          state_slots.data_ptr(), _p(spans.cu_q), _p(spans.cu_k), _p(spans.ctx_lens), out.data_ptr(), spans.num_seqs, spans.max_q, heads, kv_heads, dim, vdim,
           q_scale, is32, _stream())
     return out
 
