@@ -555,6 +555,11 @@ def main():
                          "attention with rotated values, windowed latent attention, experts chosen by logit) beside Tafopel, Tipetar and Qwen3 at "
                          "equal size, with a per-kernel roofline table (profiles/gated_bench.py); one GPU")
     ap.add_argument("--gated-sizes", default="w1024,w2048")
+    ap.add_argument("--channel", action="store_true",
+                    help="instead of the headline workload: prefill / decode throughput of the Zuvepel decoder (parallel layers, chunked attention with "
+                         "a sink, delta rule with channel decays, gated linear attention) beside Musavik, Tafopel, Tipetar and Qwen3 at equal size, "
+                         "with a per-kernel roofline table (profiles/channel_bench.py); one GPU")
+    ap.add_argument("--channel-sizes", default="w1024,w2048")
     args = ap.parse_args()
     if args.windowed:
         sys.path.insert(0, os.path.join(os.path.dirname(os.path.abspath(__file__)), "profiles"))
@@ -565,6 +570,11 @@ def main():
         sys.path.insert(0, os.path.join(os.path.dirname(os.path.abspath(__file__)), "profiles"))
         import gated_bench
         gated_bench.main(["--sizes", args.gated_sizes])
+        return
+    if args.channel:
+        sys.path.insert(0, os.path.join(os.path.dirname(os.path.abspath(__file__)), "profiles"))
+        import channel_bench
+        channel_bench.main(["--sizes", args.channel_sizes])
         return
     if args.recurrent:
         sys.path.insert(0, os.path.join(os.path.dirname(os.path.abspath(__file__)), "profiles"))

@@ -218,21 +218,16 @@ int b200m_gated_delta(const void* x, int64_t stride, int q_off, int k_off, int v
                       const int32_t* cu_k, const int32_t* ctx_lens, float* out, int num_seqs, int max_q, int num_heads, int num_kv_heads,
                       int dim, int vdim, float q_scale, int is32, void* stream);
 
-/* Matrix state with a decay per (head, key channel): g = exp(rate[h] * softplus(sign * (decay_in[t, h * dim + c] + decay_bias[h * dim + c]))),
- * or decay_in itself when decay_done (after b200m_channel_decay).  x and the state as for b200m_gated_delta.
+/* Matrix state with a decay per (head, key channel): g = exp(rate[h] * softplus(sign * (decay_in[t, h * dim + c] + decay_bias[h * dim + c]))).
+ * x and the state as for b200m_gated_delta; n rows in all.  decay_in (fp32) is scratch afterwards: single-token steps overwrite it with g.
  * write_in given (activation type, [n, num_heads] with row stride write_stride): the delta rule,
  *     q, k as for b200m_gated_delta;  S <- diag(g) S;  u = sigmoid(write_in) (v - S^T k);  S <- S + k u^T;  out = S^T q
  * write_in NULL: gated linear attention,  S <- diag(g) S + k v^T;  out = q_scale * S^T q.   dim <= 256. */
 int b200m_channel_state(const void* x, int64_t stride, int q_off, int k_off, int v_off, const void* write_in, int64_t write_stride,
-                        const float* decay_in, int64_t decay_stride, const float* rate, const float* decay_bias, float decay_sign,
-                        int decay_done, float* state, const int32_t* state_slots, const int32_t* cu_q, const int32_t* cu_k,
-                        const int32_t* ctx_lens, float* out, int num_seqs, int max_q, int num_heads, int num_kv_heads, int dim,
-                        int vdim, float q_scale, int is32, void* stream);
-
-/* a[t, h * dim + c] <- exp(rate[h] * softplus(sign * (a[t, h * dim + c] + bias[h * dim + c]))), fp32, in place: the decays of many tokens
- * formed once (b200m_channel_state forms them itself in each of a head's CTAs otherwise). */
-int b200m_channel_decay(float* a, int64_t stride, const float* rate, const float* bias, float sign, int n, int num_heads, int dim,
-                        void* stream);
+                        float* decay_in, int64_t decay_stride, const float* rate, const float* decay_bias, float decay_sign,
+                        float* state, const int32_t* state_slots, const int32_t* cu_q, const int32_t* cu_k, const int32_t* ctx_lens,
+                        float* out, int n, int num_seqs, int max_q, int num_heads, int num_kv_heads, int dim, int vdim, float q_scale,
+                        int is32, void* stream);
 
 /* out[t, h, :] = out_scale * x[t, h, :] / sqrt(mean(x[t, h, :]^2) + eps) * w * act(gate[t, h, :]); x fp32 [n, num_heads, vdim];
  * w [vdim] shared by the heads (NULL: none); gate with row stride gate_stride (NULL: none); act 0 = sigmoid, 1 = silu; out with

@@ -119,12 +119,11 @@ __global__ void __launch_bounds__(128) diag_carry_kernel(float* __restrict__ ws,
 constexpr int MS_THREADS = 128;
 
 struct DecayIn {
-    const float* in;          // pre-activations (or, with `done`, the decays themselves): CH: [n, >= H * dim], else one per head
+    const float* in;          // pre-activations, CH: [n, >= H * dim], else one per head.  (The token-at-a-time kernel reads CH decays ready-made.)
     int64_t stride;
     const float* rate;        // [H]
     const float* bias;        // CH: [H * dim], else [H]
     float sign;               // g = exp(rate_h * softplus(sign * (in + bias)))
-    int done;
 };
 __device__ __forceinline__ float decay_of(float a, float rate, float bias, float sign) { return expf(rate * softplus_(sign * (a + bias))); }
 
@@ -174,7 +173,7 @@ __global__ void __launch_bounds__(MS_THREADS) matrix_state_kernel(
             for (int k = 0; k < DPL; ++k) S[c][k] = (have && sub * DPL + k < dim) ? sr[k] : 0.f;
         }
     }
-    const float rt = dec.done ? 0.f : dec.rate[h], db = (CH || dec.done) ? 0.f : dec.bias[h];
+    const float rt = CH ? 0.f : dec.rate[h], db = CH ? 0.f : dec.bias[h];
     const T* qp = x + q_off + (int64_t)g * dim;
     const T* kp = x + k_off + (int64_t)g * dim;
     const T* vp = x + v_off + (int64_t)h * vdim + col0;
@@ -209,7 +208,7 @@ __global__ void __launch_bounds__(MS_THREADS) matrix_state_kernel(
             const int at = (d / DPL) * SEG + (d % DPL);
             ks[buf][t][at] = fk[j];
             qs[buf][t][at] = DELTA ? fq[j] : fq[j] * q_scale;
-            if constexpr (CH) gs[buf][t][at] = d < dim ? (dec.done ? fg[j] : decay_of(fg[j], rt, dec.bias[(int64_t)h * dim + d], dec.sign)) : 0.f;
+            if constexpr (CH) gs[buf][t][at] = fg[j];      // zero beyond dim
         }
 #pragma unroll
         for (int j = 0; j < PV; ++j) {
@@ -218,7 +217,7 @@ __global__ void __launch_bounds__(MS_THREADS) matrix_state_kernel(
         }
         if (tid < TB) {
             if constexpr (DELTA) sc[buf][tid][2] = sigmoidf_(fb);
-            if constexpr (!CH) sd[buf][tid] = dec.done ? fa : decay_of(fa, rt, db, dec.sign);
+            if constexpr (!CH) sd[buf][tid] = decay_of(fa, rt, db, dec.sign);
         }
     };
     auto factors = [&](int buf) {                          // after a barrier: the unit-norm factors and k . q of the chunk's tokens
@@ -367,7 +366,8 @@ __global__ void __launch_bounds__(MS_THREADS) matrix_state_kernel(
     }
 }
 
-// Decay pre-activations of many tokens -> decays, in place: a[t, h, c] <- exp(rate[h] * softplus(sign * (a + bias[h, c]))).
+// Decay pre-activations -> decays, in place: a[t, h, c] <- exp(rate[h] * softplus(sign * (a + bias[h, c]))).  In front of the
+// token-at-a-time kernel, whose column tiles would otherwise each form a head's decays on their critical path.
 __global__ void __launch_bounds__(256) channel_decay_kernel(float* __restrict__ a, int64_t stride, const float* __restrict__ rate,
                                                             const float* __restrict__ bias, float sign, int cols, int dim) {
     B200_PDL_SYNC();
@@ -412,9 +412,15 @@ __device__ __forceinline__ float2 unpack2_(uint64_t v) {
     return f;
 }
 template <int ID0>
-__device__ __forceinline__ void named_sync(int s) { asm volatile("bar.sync %0, %1;" ::"r"(ID0 + s), "n"(MB_THREADS) : "memory"); }
+__device__ __forceinline__ void named_sync(int s) {       // barrier ID0 or ID0 + 1 (as constants: a barrier number in a register reserves all sixteen)
+    if (s == 0) asm volatile("bar.sync %0, %1;" ::"n"(ID0), "n"(MB_THREADS) : "memory");
+    else asm volatile("bar.sync %0, %1;" ::"n"(ID0 + 1), "n"(MB_THREADS) : "memory");
+}
 template <int ID0>
-__device__ __forceinline__ void named_arrive(int s) { asm volatile("bar.arrive %0, %1;" ::"r"(ID0 + s), "n"(MB_THREADS) : "memory"); }
+__device__ __forceinline__ void named_arrive(int s) {
+    if (s == 0) asm volatile("bar.arrive %0, %1;" ::"n"(ID0), "n"(MB_THREADS) : "memory");
+    else asm volatile("bar.arrive %0, %1;" ::"n"(ID0 + 1), "n"(MB_THREADS) : "memory");
+}
 
 // N consecutive elements as 32-bit words (two bf16 or one float each), without conversion, so that a load stays in flight until its use
 template <typename T, int N>
@@ -466,7 +472,7 @@ struct BlockShape {
 constexpr int CF_RK = 0, CF_RQ = 4, CF_A = 8, CF_B = 14, CF_W = 24;
 
 template <typename T, int DPL, int COLS, bool CH, bool DELTA>
-__global__ void __launch_bounds__(MB_THREADS) matrix_state_block_kernel(
+__global__ void __launch_bounds__(MB_THREADS, DPL <= 16 ? 2 : 1) matrix_state_block_kernel(
     const T* __restrict__ x, int64_t stride, int q_off, int k_off, int v_off, const float* __restrict__ write_in,
     const T* __restrict__ write_t, int64_t write_stride, DecayIn dec, float* __restrict__ state, const int32_t* __restrict__ state_slots,
     const int32_t* __restrict__ cu_q, const int32_t* __restrict__ cu_k, const int32_t* __restrict__ ctx_lens, float* __restrict__ out, int H,
@@ -489,10 +495,10 @@ __global__ void __launch_bounds__(MB_THREADS) matrix_state_block_kernel(
         const T* kp = x + k_off + (int64_t)(h / (H / G)) * dim + c0;
         const T* vp = x + v_off + (int64_t)h * vdim + col0;
         const float* gp = CH ? dec.in + (int64_t)h * dim + c0 : dec.in + h;
-        const float rt = dec.done ? 0.f : dec.rate[h];
+        const float rt = dec.rate[h];
         float gb[CH ? CPL : 1];
 #pragma unroll
-        for (int e = 0; e < (CH ? CPL : 1); ++e) gb[e] = dec.done ? 0.f : CH ? (e < avail ? dec.bias[(int64_t)h * dim + c0 + e] : 0.f) : dec.bias[h];
+        for (int e = 0; e < (CH ? CPL : 1); ++e) gb[e] = CH ? (e < avail ? dec.bias[(int64_t)h * dim + c0 + e] : 0.f) : dec.bias[h];
         constexpr int VPL = MB_T * SH::GC / 32;             // value elements of a block per lane
         RawCols<T, CPL> rk[MB_T], rq[MB_T];
         RawCols<float, CH ? CPL : 1> rg[MB_T];
@@ -539,7 +545,7 @@ __global__ void __launch_bounds__(MB_THREADS) matrix_state_block_kernel(
                         k[t] = rk[t].at(e);
                         q[t] = rq[t].at(e);
                         const float raw = rg[t].at(CH ? e : 0);
-                        g[t] = i0 + t >= sp.qlen ? 1.f : dec.done ? raw : decay_of(raw, rt, gb[CH ? e : 0], dec.sign);
+                        g[t] = i0 + t < sp.qlen ? decay_of(raw, rt, gb[CH ? e : 0], dec.sign) : 1.f;
                     }
                     float p = 1.f;
 #pragma unroll
@@ -815,8 +821,8 @@ __global__ void __launch_bounds__(MB_THREADS) matrix_state_block_kernel(
 template <typename T, bool CH, bool DELTA>
 int launch_matrix_state(const void* x, int64_t stride, int q_off, int k_off, int v_off, const float* write_in, const void* write_t,
                         int64_t write_stride, const DecayIn& dec, float* state, const int32_t* state_slots, const int32_t* cu_q,
-                        const int32_t* cu_k, const int32_t* ctx_lens, float* out, int num_seqs, int max_q, int H, int G, int dim, int vdim,
-                        float q_scale, cudaStream_t st) {
+                        const int32_t* cu_k, const int32_t* ctx_lens, float* out, int total_rows, int num_seqs, int max_q, int H, int G, int dim,
+                        int vdim, float q_scale, cudaStream_t st) {
     if (dim > 256) return B200_EUNSUPPORTED;
 #define MB_GO(DPL, COLS)                                                                                                           \
     do {                                                                                                                           \
@@ -840,6 +846,13 @@ int launch_matrix_state(const void* x, int64_t stride, int q_off, int k_off, int
         MB_GO(32, 2);
     }
 #undef MB_GO
+    if constexpr (CH) {
+        const int cols = H * dim, rows = cu_q ? total_rows : num_seqs;
+        B200_LAUNCH((channel_decay_kernel), dim3(rows, (unsigned)((cols + 1023) / 1024)), 256, 0, st, const_cast<float*>(dec.in), dec.stride,
+                    dec.rate, dec.bias, dec.sign, cols, dim);
+        const int rc = b200_launch_status(nullptr);
+        if (rc != B200_OK) return rc;
+    }
 #define MS_GO(DPL, LANES, COLS)                                                                                                    \
     do {                                                                                                                           \
         constexpr int GC = MS_THREADS / LANES * COLS;                                                                              \
@@ -925,42 +938,33 @@ extern "C" int b200m_gated_delta(const void* x, int64_t stride, int q_off, int k
     if ((cu_q == nullptr) != (cu_k == nullptr) || (cu_q == nullptr && ctx_lens == nullptr)) return B200_EINVAL;
     if (num_heads <= 0 || num_kv_heads <= 0 || num_heads % num_kv_heads || dim <= 0 || vdim <= 0) return B200_EINVAL;
     if (num_seqs <= 0) return B200_OK;
-    const DecayIn dec{ba + num_heads, ba_stride, rate, dt_bias, 1.0f, 0};
+    const DecayIn dec{ba + num_heads, ba_stride, rate, dt_bias, 1.0f};
     B200M_DISPATCH(is32, return (launch_matrix_state<T, false, true>(x, stride, q_off, k_off, v_off, ba, nullptr, ba_stride, dec, state,
-                                                                     state_slots, cu_q, cu_k, ctx_lens, out, num_seqs, max_q, num_heads,
+                                                                     state_slots, cu_q, cu_k, ctx_lens, out, 0, num_seqs, max_q, num_heads,
                                                                      num_kv_heads, dim, vdim, q_scale, static_cast<cudaStream_t>(stream))));
     return B200_EUNSUPPORTED;
 }
 
-extern "C" int b200m_channel_decay(float* a, int64_t stride, const float* rate, const float* bias, float sign, int n, int num_heads,
-                                   int dim, void* stream) {
-    if (!a || !rate || !bias || n < 0 || num_heads <= 0 || dim <= 0 || stride < (int64_t)num_heads * dim) return B200_EINVAL;
-    if (n == 0) return B200_OK;
-    const int cols = num_heads * dim;
-    B200_LAUNCH((channel_decay_kernel), dim3(n, (unsigned)((cols + 1023) / 1024)), 256, 0, static_cast<cudaStream_t>(stream), a, stride, rate, bias, sign,
-                cols, dim);
-    return b200_launch_status(nullptr);
-}
-
 extern "C" int b200m_channel_state(const void* x, int64_t stride, int q_off, int k_off, int v_off, const void* write_in,
-                                   int64_t write_stride, const float* decay_in, int64_t decay_stride, const float* rate,
-                                   const float* decay_bias, float decay_sign, int decay_done, float* state,
-                                   const int32_t* state_slots, const int32_t* cu_q, const int32_t* cu_k, const int32_t* ctx_lens,
-                                   float* out, int num_seqs, int max_q, int num_heads, int num_kv_heads, int dim, int vdim, float q_scale,
-                                   int is32, void* stream) {
-    if (!x || !decay_in || !state || !state_slots || !out || (!decay_done && (!rate || !decay_bias))) return B200_EINVAL;
+                                   int64_t write_stride, float* decay_in, int64_t decay_stride, const float* rate,
+                                   const float* decay_bias, float decay_sign, float* state, const int32_t* state_slots,
+                                   const int32_t* cu_q, const int32_t* cu_k, const int32_t* ctx_lens, float* out, int n, int num_seqs,
+                                   int max_q, int num_heads, int num_kv_heads, int dim, int vdim, float q_scale, int is32,
+                                   void* stream) {
+    if (!x || !decay_in || !state || !state_slots || !out || !rate || !decay_bias) return B200_EINVAL;
     if ((cu_q == nullptr) != (cu_k == nullptr) || (cu_q == nullptr && ctx_lens == nullptr)) return B200_EINVAL;
     if (num_heads <= 0 || num_kv_heads <= 0 || num_heads % num_kv_heads || dim <= 0 || vdim <= 0) return B200_EINVAL;
-    if (num_seqs <= 0) return B200_OK;
-    const DecayIn dec{decay_in, decay_stride, rate, decay_bias, decay_sign, decay_done};
+    if (decay_stride < (int64_t)num_heads * dim || n < 0) return B200_EINVAL;
+    if (num_seqs <= 0 || n == 0) return B200_OK;
+    const DecayIn dec{decay_in, decay_stride, rate, decay_bias, decay_sign};
     cudaStream_t st = static_cast<cudaStream_t>(stream);
     if (write_in) {
         B200M_DISPATCH(is32, return (launch_matrix_state<T, true, true>(x, stride, q_off, k_off, v_off, nullptr, write_in, write_stride, dec,
-                                                                        state, state_slots, cu_q, cu_k, ctx_lens, out, num_seqs, max_q, num_heads,
+                                                                        state, state_slots, cu_q, cu_k, ctx_lens, out, n, num_seqs, max_q, num_heads,
                                                                         num_kv_heads, dim, vdim, q_scale, st)));
     } else {
         B200M_DISPATCH(is32, return (launch_matrix_state<T, true, false>(x, stride, q_off, k_off, v_off, nullptr, nullptr, 0, dec, state,
-                                                                         state_slots, cu_q, cu_k, ctx_lens, out, num_seqs, max_q, num_heads,
+                                                                         state_slots, cu_q, cu_k, ctx_lens, out, n, num_seqs, max_q, num_heads,
                                                                          num_kv_heads, dim, vdim, q_scale, st)));
     }
     return B200_EUNSUPPORTED;

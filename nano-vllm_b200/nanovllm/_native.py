@@ -65,9 +65,8 @@ MIX_SIGNATURES = {
     "b200m_head_mix_gate": (_i, [_vp, _i, _vp, _vp, _i64, _vp, _i64, _f, _i, _i, _i, _i, _i, _vp]),
     "b200m_diag_scan": (_i, [_vp, _i64, _vp, _i64, _vp, _vp, _vp, _i64, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _vp, _i, _vp]),
     "b200m_gated_delta": (_i, [_vp, _i64, _i, _i, _i, _vp, _i64, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _f, _i, _vp]),
-    "b200m_channel_state": (_i, [_vp, _i64, _i, _i, _i, _vp, _i64, _vp, _i64, _vp, _vp, _f, _i, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i,
+    "b200m_channel_state": (_i, [_vp, _i64, _i, _i, _i, _vp, _i64, _vp, _i64, _vp, _vp, _f, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i,
                                  _i, _f, _i, _vp]),
-    "b200m_channel_decay": (_i, [_vp, _i64, _vp, _vp, _f, _i, _i, _i, _vp]),
     "b200m_head_rmsnorm_gate": (_i, [_vp, _vp, _vp, _i64, _i, _vp, _i64, _f, _i, _i, _i, _f, _i, _vp]),
     "b200m_moe_route_grouped": (_i, [_vp, _i64, _i, _i, _i, _vp, _i, _i, _i, _i, _i, _f, _vp, _vp, _vp]),
     "b200m_add_layernorm": (_i, [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _f, _i, _vp]),

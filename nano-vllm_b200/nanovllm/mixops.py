@@ -464,11 +464,11 @@ def gated_delta(x: torch.Tensor, q_off: int, k_off: int, v_off: int, ba: torch.T
 
 def channel_state(x: torch.Tensor, q_off: int, k_off: int, v_off: int, write: torch.Tensor | None, decay_in: torch.Tensor, rate: torch.Tensor,
                   decay_bias: torch.Tensor, decay_sign: float, state: torch.Tensor, state_slots: torch.Tensor, spans: StepSpans, heads: int,
-                  kv_heads: int, dim: int, vdim: int, q_scale: float, decays_first: bool | None = None) -> torch.Tensor:
+                  kv_heads: int, dim: int, vdim: int, q_scale: float) -> torch.Tensor:
     """Matrix state with one decay per head and key channel, exp(rate[h] * softplus(sign * (decay_in + decay_bias))).
     x [n, cols]: q, k ([kv_heads, dim] at q_off / k_off) and v ([heads, vdim] at v_off); ``write`` [n, heads] (a row-strided view): delta rule
-    with unit-norm q and k; None: gated linear attention.  decay_in fp32 [n, heads * dim] (prompt steps, ``decays_first``: overwritten by the
-    decays, formed once instead of in every column tile of a head); state fp32 [slots, heads, vdim, dim] -> fp32 [n, heads, vdim]."""
+    with unit-norm q and k; None: gated linear attention.  decay_in fp32 [n, heads * dim] is scratch (single-token steps
+    form the decays in place first); state fp32 [slots, heads, vdim, dim] -> fp32 [n, heads, vdim]."""
     n = x.shape[0]
     is32 = _is32(x)
     assert x.dim() == 2 and x.stride(1) == 1 and decay_in.dtype == torch.float32 and decay_in.stride(1) == 1 and decay_in.shape == (n, heads * dim)
@@ -477,13 +477,11 @@ def channel_state(x: torch.Tensor, q_off: int, k_off: int, v_off: int, write: to
     assert write is None or (write.shape == (n, heads) and write.stride(1) == 1)
     _same(is32, write)
     out = torch.empty(n, heads, vdim, dtype=torch.float32, device=x.device)
-    if decays_first is None:
-        decays_first = spans.max_q > 1
-    if decays_first:
-        _call("b200m_channel_decay", decay_in.data_ptr(), decay_in.stride(0), rate.data_ptr(), decay_bias.data_ptr(), decay_sign, n, heads, dim, _stream())
+    if spans.cu_q is None or spans.max_q <= 4:
+        ops.LAUNCHES[0] += 1
     _call("b200m_channel_state", x.data_ptr(), x.stride(0), q_off, k_off, v_off, _p(write), write.stride(0) if write is not None else 0,
-          decay_in.data_ptr(), decay_in.stride(0), rate.data_ptr(), decay_bias.data_ptr(), decay_sign, int(decays_first), state.data_ptr(),
-          state_slots.data_ptr(), _p(spans.cu_q), _p(spans.cu_k), _p(spans.ctx_lens), out.data_ptr(), spans.num_seqs, spans.max_q, heads, kv_heads, dim, vdim,
+          decay_in.data_ptr(), decay_in.stride(0), rate.data_ptr(), decay_bias.data_ptr(), decay_sign, state.data_ptr(),
+          state_slots.data_ptr(), _p(spans.cu_q), _p(spans.cu_k), _p(spans.ctx_lens), out.data_ptr(), n, spans.num_seqs, spans.max_q, heads, kv_heads, dim, vdim,
           q_scale, is32, _stream())
     return out
 
