@@ -247,7 +247,7 @@ def test_channel_delta_layer(dtype, m):
                                      tol=3e-4 if dtype == "float32" else 4e-2)
 
 
-GLAS = [zh.gla(), zh.gla(heads=1, dim=7, vdim=3, tau=1.0), zh.gla(heads=6, dim=48, vdim=64, tau=16.0), zh.gla(heads=2, dim=128, vdim=80, tau=2.5),
+GLAS = [zh.gla(), zh.gla(heads=1, dim=7, vdim=3, tau=1.0), zh.gla(heads=5, dim=40, vdim=56, tau=12.0), zh.gla(heads=2, dim=128, vdim=80, tau=2.5),
         zh.gla(heads=2, dim=64, vdim=33, tau=4.0), zh.gla(heads=1, dim=256, vdim=40, tau=8.0)]
 
 
