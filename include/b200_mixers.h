@@ -2,7 +2,7 @@
  * b200_mixers.h -- C ABI of libb200mix.so: sequence mixers and feed-forward pieces of hybrid decoders on B200 (sm_100a):
  * latent attention with a softmax sink over a paged cache of compressed keys, grouped-query attention with a sliding
  * window (optionally with kept first tokens and mixed heads) and a linear distance bias, recurrences with per-sequence state
- * slots (selective scan, gated diagonal recurrence, gated delta rule), routed experts, and the row-wise ops around them
+ * slots (selective scan, gated diagonal recurrence, gated delta rule, scalar linear attention), routed experts, and the row-wise ops around them
  * (embedding into an fp32 residual stream, residual update + weight-only layer norm, norm on a sublayer's output, RMS norm,
  * feed-forward activations).
  *
@@ -74,6 +74,11 @@ int b200m_add_layernorm2(const float* x_in, float* x_out, const void* y, float m
                          const void* b1, void* out1, const void* w2, const void* b2, void* out2, const int32_t* rows_idx, int rows,
                          int cols, float eps, int is32, void* stream);
 
+/* A boundary of a pre-norm layer: x[r, :] += y[r, :] (activation type; NULL: nothing), then, unless out is NULL, out[r, :] = x[r, :] /
+ * sqrt(mean(x[r, :]^2) + eps) * w * out_scale.  With rows_idx (int32 [rows], y NULL) out[i, :] is the norm of row rows_idx[i]. */
+int b200m_add_rmsnorm(float* x, const void* y, const void* w, void* out, const int32_t* rows_idx, int rows, int cols, float eps,
+                      float out_scale, int is32, void* stream);
+
 /* out = x / sqrt(mean(x^2) + eps) * w over the first `cols` elements of each (strided) row. */
 int b200m_rmsnorm(const void* x, int64_t x_stride, const void* w, void* out, int64_t out_stride, int rows, int cols,
                   float eps, int is32, void* stream);
@@ -136,10 +141,11 @@ int b200m_qk_norm_store(void* qkv, int64_t stride, int q_cols, int k_cols, int v
  * turned by cos_sin[position] = [cos (rope_dims/2) | sin (rope_dims/2)] (fp32; NULL: no rotation; layout 1: the query and key pairs are
  * (i, i + rope_dims / 2) instead), in place; keys the same with
  * k_norm_w into cache[slot] = [k (G * dim) | v (G * vdim)]; values divided by their root mean square per head (v_unit_norm) or
- * copied; v_cos_sin (optional, fp32 [positions, v_rope_dims]): the value pairs (2m, 2m+1), m < v_rope_dims / 2, are turned by the
+ * copied.  unit_after (q_norm_w and k_norm_w NULL then): q and k are divided by their root mean square over the head after the
+ * rotation (no weight); v_cos_sin (optional, fp32 [positions, v_rope_dims]): the value pairs (2m, 2m+1), m < v_rope_dims / 2, are turned by the
  * token's position before the store.  cache NULL or slot < 0: queries only. */
 int b200m_headnorm_rope_store(void* x, int64_t stride, int q_off, int k_off, int v_off, int num_heads, int num_kv_heads, int dim,
-                              int vdim, const void* q_norm_w, const void* k_norm_w, int v_unit_norm, const float* cos_sin,
+                              int vdim, const void* q_norm_w, const void* k_norm_w, int v_unit_norm, int unit_after, const float* cos_sin,
                               int layout, int rope_dims, const float* v_cos_sin, int v_rope_dims, const int64_t* positions, const int32_t* slots,
                               void* cache, int n, float eps, int is32, void* stream);
 
@@ -162,18 +168,22 @@ int b200m_head_mix_gate(const void* acc, int acc_f32, const float* mix, const vo
  * num_kv_heads)): score = q . k * scale - slopes[h] * (i - j) (slopes NULL: no bias), visible keys 0 <= i - j < window
  * or j < keep_first (window <= 0: all j <= i); chunk > 0 (window 0 then): the keys j <= i of the query's own chunk, i - i % chunk <= j,
  * or j < keep_first.  Softmax with, when sinks (fp32 [num_heads]) is given, one more term exp(sinks[h]) in the denominator that has no
- * value.  gate (optional, activation type, row stride gate_stride; not with all_values): head h of token t times sigmoid(gate[t, h]).
+ * value.  softcap > 0: the scaled product q . k * scale becomes softcap * tanh(. / softcap) first.  gate (optional, activation type, row
+ * stride gate_stride; not with all_values): head h of token t times sigmoid(gate[t, h]), or with gate_elems element by element times
+ * sigmoid(gate[t, h * vdim + c]).  The result is multiplied by out_scale.
  * all_values: every query head's weights are applied to the
  * values of EVERY value head, out [total_q, num_heads, num_kv_heads, vdim] (for b200m_head_mix_gate).  flags & 2: out is fp32.  A cache row is row_elems long: key head g at g * dim, value head g at
  * v_off + g * vdim.  q [total_q, >= num_heads * dim] with row stride q_stride; out [total_q, >= num_heads * vdim] with row stride out_stride.
- * bf16 with dim and vdim in {32, 64, 128} runs on the tensor cores unless flags & 1; everything else on the fp32 FMA pipe.
+ * bf16 with dim and vdim multiples of eight up to 128 runs on the tensor cores unless flags & 1 (32, 64 and 128 as they are, other sizes
+ * with zero columns up to 64 or 128); everything else on the fp32 FMA pipe.
  * splits > 1 (bf16 tensor-core decode steps only): the visible keys of every row are shared out over `splits` CTAs whose
  * partials, fp32 [num_seqs, splits, num_heads (x num_kv_heads with all_values), vdim + 2] in `part`, a second launch merges. */
 int b200m_window_attention(const void* q, int64_t q_stride, const void* cache, int row_elems, int v_off,
                            const int32_t* block_tables, int bt_stride, int block_size, const int32_t* cu_q,
                            const int32_t* cu_k, const int32_t* ctx_lens, const float* slopes, int window, int keep_first,
-                           int chunk, const float* sinks, const void* gate, int64_t gate_stride, int all_values, void* out, int64_t out_stride, int total_q, int num_seqs, int max_q, int num_heads, int num_kv_heads,
-                           int dim, int vdim, float scale, int is32, int flags, int splits, float* part, void* stream);
+                           int chunk, const float* sinks, float softcap, const void* gate, int64_t gate_stride, int gate_elems,
+                           float out_scale, int all_values, void* out, int64_t out_stride, int total_q, int num_seqs, int max_q,
+                           int num_heads, int num_kv_heads, int dim, int vdim, float scale, int is32, int flags, int splits, float* part, void* stream);
 
 /* ---- selective scan ------------------------------------------------------------------------------------------------ */
 
@@ -229,11 +239,41 @@ int b200m_channel_state(const void* x, int64_t stride, int q_off, int k_off, int
                         float* out, int n, int num_seqs, int max_q, int num_heads, int num_kv_heads, int dim, int vdim, float q_scale,
                         int is32, void* stream);
 
+/* Scalar linear attention: per head a matrix state with one decay and one write weight per token,
+ *     S <- g S + w k v^T;  out = q_scale * S^T q                      (S fp32 [dim, vdim], from zero for a new sequence)
+ * x as for b200m_gated_delta (q, k [num_kv_heads, dim], v [num_heads, vdim]).  step_in given (activation type, [n, num_heads] with row
+ * stride gate_stride): w = softplus(step_in + bias[h]), g = exp(rate[h] * w), a state-space step with q = C, k = B, v = x.  step_in NULL:
+ * log_decay = log g and write = w, fp32 [n, num_heads] with row stride gate_stride (b200m_mlstm_gates makes them).  ones = 1: the
+ * state has one more column whose value is always 1; state fp32 [slots, num_heads, vdim + ones, dim], out fp32 [n, num_heads, vdim + ones].
+ * dim <= 256. */
+int b200m_linear_state(const void* x, int64_t stride, int q_off, int k_off, int v_off, const void* step_in, const float* log_decay,
+                       const float* write, int64_t gate_stride, const float* rate, const float* bias, float* state,
+                       const int32_t* state_slots, const int32_t* cu_q, const int32_t* cu_k, const int32_t* ctx_lens, float* out,
+                       int num_seqs, int max_q, int num_heads, int num_kv_heads, int dim, int vdim, int ones, float q_scale, int is32,
+                       void* stream);
+
+/* Exponential gates of a matrix memory with a running maximum.  in fp32 [n, >= 2 num_heads] = [i | f] pre-activations, bias fp32 [2 num_heads]:
+ *     i = cap * tanh((in_i + bias_i) / cap);  f = logsigmoid(cap * tanh((in_f + bias_f) / cap));  m_t = max(f_t + m_(t-1), i_t)
+ *     log_decay = f_t + m_(t-1) - m_t;  write = exp(i_t - m_t);  floor = exp(-m_t)                       (fp32 [n, num_heads] each)
+ * m_state fp32 [slots, num_heads], 0 for a new sequence. */
+int b200m_mlstm_gates(const float* in, int64_t stride, const float* bias, float cap, float* m_state, const int32_t* state_slots,
+                      const int32_t* cu_q, const int32_t* cu_k, const int32_t* ctx_lens, float* log_decay, float* write, float* floor,
+                      int num_seqs, int num_heads, void* stream);
+
+/* t = (y[r, h, :] + D[h] x[r, h, :]) * silu(z[r, h, :]) over rows of num_heads * vdim columns, then every one of `groups` equal parts of the
+ * row divided by its own root mean square (sqrt(mean(t^2) + eps)), times w [num_heads * vdim].  y, D fp32; x, z, w, out in the activation
+ * type, x, z and out with row strides. */
+int b200m_skip_gate_groupnorm(const float* y, const void* x, int64_t x_stride, const float* D, const void* z, int64_t z_stride,
+                              const void* w, void* out, int64_t out_stride, int n, int num_heads, int vdim, int groups, float eps, int is32,
+                              void* stream);
+
 /* out[t, h, :] = out_scale * x[t, h, :] / sqrt(mean(x[t, h, :]^2) + eps) * w * act(gate[t, h, :]); x fp32 [n, num_heads, vdim];
- * w [vdim] shared by the heads (NULL: none); gate with row stride gate_stride (NULL: none); act 0 = sigmoid, 1 = silu; out with
- * row stride out_stride. */
-int b200m_head_rmsnorm_gate(const float* x, const void* w, const void* gate, int64_t gate_stride, int act, void* out,
-                            int64_t out_stride, float out_scale, int n, int num_heads, int vdim, float eps, int is32, void* stream);
+ * w [vdim] shared by the heads, or with w_heads [num_heads * vdim] (NULL: none); gate with row stride gate_stride (NULL: none);
+ * act 0 = sigmoid, 1 = silu; out with row stride out_stride.  floor given (fp32 [n, num_heads]): x is [n, num_heads, vdim + 1], and
+ * x[t, h, :vdim] is first divided by max(|x[t, h, vdim]|, floor[t, h]) + 1e-6. */
+int b200m_head_rmsnorm_gate(const float* x, const float* floor, const void* w, int w_heads, const void* gate, int64_t gate_stride, int act,
+                            void* out, int64_t out_stride, float out_scale, int n, int num_heads, int vdim, float eps, int is32,
+                            void* stream);
 
 /* ---- routed experts ------------------------------------------------------------------------------------------------ */
 

@@ -284,6 +284,65 @@ __global__ void __launch_bounds__(ROW_THREADS) add_layernorm2_kernel(const float
     }
 }
 
+// A boundary of a pre-norm layer:  x += y (fp32 stream; y in the activation type, optional), then
+//     out = x / sqrt(mean(x^2) + eps) * w * out_scale (optional).
+// rows_idx (optional): row i of the output is row rows_idx[i] of the stream, which is not updated then.  Registers as above.
+template <typename T, int V, int PER>
+__global__ void __launch_bounds__(ROW_THREADS) add_rmsnorm_kernel(float* x, const T* __restrict__ y, const T* __restrict__ w,
+                                                                  T* __restrict__ out, const int32_t* __restrict__ rows_idx, int cols,
+                                                                  float eps, float out_scale) {
+    B200_PDL_SYNC();
+    __shared__ float red[ROW_THREADS / 32];
+    const int64_t row = rows_idx ? rows_idx[blockIdx.x] : blockIdx.x, base = row * cols, obase = (int64_t)blockIdx.x * cols;
+    const int step = blockDim.x * V;
+    auto updated = [&](int c, float (&f)[V]) {
+        load_cols<float, V>(x + base + c, f);
+        if (y) {
+            float a[V];
+            load_cols<T, V>(y + base + c, a);
+#pragma unroll
+            for (int e = 0; e < V; ++e) f[e] += a[e];
+            store_cols<float, V>(x + base + c, f);
+        }
+    };
+    float r[PER][V];
+    float q = 0.f;
+#pragma unroll
+    for (int k = 0; k < PER; ++k) {
+        const int c = threadIdx.x * V + k * step;
+#pragma unroll
+        for (int e = 0; e < V; ++e) r[k][e] = 0.f;
+        if (c < cols) updated(c, r[k]);
+#pragma unroll
+        for (int e = 0; e < V; ++e) q = fmaf(r[k][e], r[k][e], q);
+    }
+    for (int c = threadIdx.x * V + PER * step; c < cols; c += step) {
+        float f[V];
+        updated(c, f);
+#pragma unroll
+        for (int e = 0; e < V; ++e) q = fmaf(f[e], f[e], q);
+    }
+    if (out == nullptr) return;
+    const float rstd = 1.0f / sqrtf(block_sum(q, red) / (float)cols + eps);
+    auto emit = [&](int c, float (&f)[V]) {
+        float g[V];
+        load_cols<T, V>(w + c, g);
+#pragma unroll
+        for (int e = 0; e < V; ++e) f[e] = f[e] * rstd * g[e] * out_scale;
+        store_cols<T, V>(out + obase + c, f);
+    };
+#pragma unroll
+    for (int k = 0; k < PER; ++k) {
+        const int c = threadIdx.x * V + k * step;
+        if (c < cols) emit(c, r[k]);
+    }
+    for (int c = threadIdx.x * V + PER * step; c < cols; c += step) {      // the same thread wrote these elements: no fence needed
+        float f[V];
+        load_cols<float, V>(x + base + c, f);
+        emit(c, f);
+    }
+}
+
 template <typename T>
 __global__ void __launch_bounds__(ROW_THREADS) rmsnorm_any_kernel(const T* __restrict__ x, int64_t x_stride, const T* __restrict__ w,
                                                                   T* __restrict__ out, int64_t out_stride, int cols, float eps) {
@@ -454,7 +513,7 @@ __global__ void __launch_bounds__(256) softcap_kernel(float* __restrict__ x, int
 
 }  // namespace
 
-extern "C" int b200m_abi_version(void) { return 5; }
+extern "C" int b200m_abi_version(void) { return 6; }
 
 extern "C" int b200m_ff_glu_clamped(const void* x, int64_t x_stride, void* out, int64_t rows, int n, float limit, float alpha, int is32,
                                     void* stream) {
@@ -589,6 +648,25 @@ extern "C" int b200m_add_layernorm2(const float* x_in, float* x_out, const void*
     else if (vec) LN2_GO(4, 4);
     else LN2_GO(1, 4);
 #undef LN2_GO
+    return b200_launch_status(nullptr);
+}
+
+extern "C" int b200m_add_rmsnorm(float* x, const void* y, const void* w, void* out, const int32_t* rows_idx, int rows, int cols, float eps,
+                                 float out_scale, int is32, void* stream) {
+    if (!x || rows < 0 || cols <= 0 || (out && !w) || (y && rows_idx) || (!y && !out)) return B200_EINVAL;      // an update covers whole steps
+    if (rows == 0) return B200_OK;
+    cudaStream_t st = static_cast<cudaStream_t>(stream);
+    uintptr_t bits = 0;
+    for (const void* p : {static_cast<const void*>(x), y, w, static_cast<const void*>(out)}) bits |= reinterpret_cast<uintptr_t>(p);
+    const bool vec = cols % 4 == 0 && bits % 16 == 0;
+#define RMS_GO(V, PER)                                                                                                             \
+    B200M_DISPATCH(is32, B200_LAUNCH((add_rmsnorm_kernel<T, V, PER>), rows, ROW_THREADS, 0, st, x, static_cast<const T*>(y),       \
+                                     static_cast<const T*>(w), static_cast<T*>(out), rows_idx, cols, eps, out_scale))
+    if (vec && cols <= 4 * ROW_THREADS) RMS_GO(4, 1);
+    else if (vec && cols <= 8 * ROW_THREADS) RMS_GO(4, 2);
+    else if (vec) RMS_GO(4, 4);
+    else RMS_GO(1, 4);
+#undef RMS_GO
     return b200_launch_status(nullptr);
 }
 

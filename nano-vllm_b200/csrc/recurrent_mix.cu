@@ -14,12 +14,16 @@
 //   zero keeping (product of a, end state), a serial pass over the chunk summaries that leaves every chunk's start state, and
 //   every chunk again from its start state writing the output.
 //
-// Matrix states (per head S [dim, vdim]; query/key head h / (H / G)); one kernel, three rules:
+// Matrix states (per head S [dim, vdim]; query/key head h / (H / G)); one kernel, four rules:
 //   gated delta rule            q <- q / sqrt(|q|^2 + 1e-6) * q_scale,  k <- k / sqrt(|k|^2 + 1e-6)
 //                               g = exp(rate_h softplus(a_t + dt_bias_h)),  beta = sigmoid(b_t)
 //                               S <- g S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q
 //   delta rule, channel decays  the same with g per (head, key channel) on the rows of S
 //   gated linear attention      S <- diag(g) S + k (q_scale q, k as they are) v^T;  o = S^T q;  g per (head, key channel)
+//   scalar linear attention     S <- g S + w k v^T  (q_scale q, k as they are);  o = S^T q;  g and w one number per head: either
+//                               w = softplus(a_t + bias_h), g = exp(rate_h w) (a state-space step), or log g and w ready-made (a
+//                               matrix memory with exponential gates, mlstm_gates_kernel).  `ones`: one more state column whose
+//                               value is always 1, the running sum of weighted keys that normalises the read-out
 //   Channel decays are g = exp(rate_h softplus(sign (a + bias))): sign 1 is the softplus form; sigmoid(z)^(1 / tau) is rate
 //   -1 / tau with sign -1.  Columns of S are independent: a lane group owns one or two of them and walks the tokens.
 #include "mix_common.cuh"
@@ -127,14 +131,34 @@ struct DecayIn {
 };
 __device__ __forceinline__ float decay_of(float a, float rate, float bias, float sign) { return expf(rate * softplus_(sign * (a + bias))); }
 
+// What scalar linear attention (neither CH nor DELTA) does with a token: raw fp32 (or T) inputs -> (log decay, write weight).
+template <typename T>
+struct ScalarGate {
+    const T* raw;             // step-size pre-activations (n, >= H), or NULL: `log_decay` and `write` are given
+    const float *log_decay, *write;
+    int64_t stride;           // of whichever is read
+    const float *rate, *bias;
+    __device__ __forceinline__ float2 fetch(int64_t row, int h) const {      // loads only
+        if (raw) return make_float2(ldf(raw + row * stride + h), 0.f);
+        return make_float2(log_decay[row * stride + h], write[row * stride + h]);
+    }
+    __device__ __forceinline__ float2 gates(float2 f, float rt, float b) const {
+        if (!raw) return f;
+        const float dt = softplus_(f.x + b);
+        return make_float2(rt * dt, dt);
+    }
+};
+
 template <typename T, int DPL, int LANES, int COLS, bool CH, bool DELTA>
 __global__ void __launch_bounds__(MS_THREADS) matrix_state_kernel(
     const T* __restrict__ x, int64_t stride, int q_off, int k_off, int v_off,     // per token: q, k [G, dim], v [H, vdim]
     const float* __restrict__ write_in, const T* __restrict__ write_t, int64_t write_stride,      // DELTA: H write strengths (pre-activation), fp32 or T
-    DecayIn dec, float* __restrict__ state, const int32_t* __restrict__ state_slots, const int32_t* __restrict__ cu_q,
-    const int32_t* __restrict__ cu_k, const int32_t* __restrict__ ctx_lens, float* __restrict__ out,      // [n, H, vdim] fp32
-    int H, int G, int dim, int vdim, float q_scale) {
+    DecayIn dec, ScalarGate<T> sg, float* __restrict__ state, const int32_t* __restrict__ state_slots, const int32_t* __restrict__ cu_q,
+    const int32_t* __restrict__ cu_k, const int32_t* __restrict__ ctx_lens, float* __restrict__ out,      // [n, H, vcols] fp32
+    int H, int G, int dim, int vdim, int ones, float q_scale) {
     B200_PDL_SYNC();
+    constexpr bool LIN = !CH && !DELTA;
+    const int vcols = LIN ? vdim + ones : vdim;            // columns of the state
     constexpr int NT = MS_THREADS, GC = NT / LANES * COLS;  // columns of the CTA
     constexpr int DP = LANES * DPL, SEG = DPL + 4, ROW = LANES * SEG;
     constexpr int TB = DP >= 256 ? 4 : (DP >= 128 || CH) ? 8 : 16;
@@ -153,13 +177,13 @@ __global__ void __launch_bounds__(MS_THREADS) matrix_state_kernel(
     const int sub = tid % LANES, grp = tid / LANES;
     const int col0 = blockIdx.z * GC, mycol = col0 + grp * COLS;
     const int g = h / (H / G);
-    float* st = state + ((int64_t)state_slots[s] * H + h) * vdim * dim + sub * DPL;      // + column * dim
+    float* st = state + ((int64_t)state_slots[s] * H + h) * vcols * dim + sub * DPL;     // + column * dim
     const bool has_hist = sp.klen - sp.qlen > 0;
     const bool vec_state = dim % 4 == 0;                    // 16-byte aligned segments: 128-bit state accesses
     float S[COLS][DPL];
 #pragma unroll
     for (int c = 0; c < COLS; ++c) {
-        const bool have = has_hist && mycol + c < vdim;
+        const bool have = has_hist && mycol + c < vcols;
         const float* sr = st + (int64_t)(mycol + c) * dim;
         if (vec_state) {
 #pragma unroll
@@ -173,7 +197,8 @@ __global__ void __launch_bounds__(MS_THREADS) matrix_state_kernel(
             for (int k = 0; k < DPL; ++k) S[c][k] = (have && sub * DPL + k < dim) ? sr[k] : 0.f;
         }
     }
-    const float rt = CH ? 0.f : dec.rate[h], db = CH ? 0.f : dec.bias[h];
+    const float* rate = LIN ? sg.rate : dec.rate;
+    const float rt = (CH || rate == nullptr) ? 0.f : rate[h], db = (CH || rate == nullptr) ? 0.f : (LIN ? sg.bias : dec.bias)[h];
     const T* qp = x + q_off + (int64_t)g * dim;
     const T* kp = x + k_off + (int64_t)g * dim;
     const T* vp = x + v_off + (int64_t)h * vdim + col0;
@@ -193,11 +218,17 @@ __global__ void __launch_bounds__(MS_THREADS) matrix_state_kernel(
         for (int j = 0; j < PV; ++j) {
             const int e = tid + NT * j, t = e / GC, c = e - t * GC;
             fv[j] = (t < TB && i0 + t < sp.qlen && col0 + c < vdim) ? ldf(vp + (int64_t)(sp.q0 + i0 + t) * stride + c) : 0.f;
+            if (LIN && ones && col0 + c == vdim) fv[j] = 1.0f;
         }
         if (tid < TB && i0 + tid < sp.qlen) {
             const int64_t row = sp.q0 + i0 + tid;
             if constexpr (DELTA) fb = write_in ? write_in[row * write_stride + h] : ldf(write_t + row * write_stride + h);
-            if constexpr (!CH) fa = gp[row * dec.stride];
+            if constexpr (LIN) {
+                const float2 f = sg.fetch(row, h);
+                fa = f.x, fb = f.y;
+            } else if constexpr (!CH) {
+                fa = gp[row * dec.stride];
+            }
         }
     };
     auto land = [&](int buf) {                             // registers -> shared memory
@@ -217,7 +248,13 @@ __global__ void __launch_bounds__(MS_THREADS) matrix_state_kernel(
         }
         if (tid < TB) {
             if constexpr (DELTA) sc[buf][tid][2] = sigmoidf_(fb);
-            if constexpr (!CH) sd[buf][tid] = decay_of(fa, rt, db, dec.sign);
+            if constexpr (LIN) {
+                const float2 f = sg.gates(make_float2(fa, fb), rt, db);
+                sd[buf][tid] = expf(f.x);
+                sc[buf][tid][2] = f.y;
+            } else if constexpr (!CH) {
+                sd[buf][tid] = decay_of(fa, rt, db, dec.sign);
+            }
         }
     };
     auto factors = [&](int buf) {                          // after a barrier: the unit-norm factors and k . q of the chunk's tokens
@@ -263,7 +300,7 @@ __global__ void __launch_bounds__(MS_THREADS) matrix_state_kernel(
         }
     };
     const int ocol = mycol + (COLS == 2 ? (sub & 1) : 0);  // the column whose sum this lane holds after reduce()
-    const bool writer = sub < COLS && ocol < vdim;
+    const bool writer = sub < COLS && ocol < vcols;
     fetch(0);
     land(0);
     __syncthreads();
@@ -282,6 +319,7 @@ __global__ void __launch_bounds__(MS_THREADS) matrix_state_kernel(
 #pragma unroll
             for (int c = 0; c < COLS; ++c) {
                 v[c] = vs[buf][t][grp * COLS + c];
+                if constexpr (LIN) v[c] *= sc[buf][t][2];
                 o[c] = 0.f;
             }
             if constexpr (DELTA) {
@@ -307,7 +345,7 @@ __global__ void __launch_bounds__(MS_THREADS) matrix_state_kernel(
                 const float4 f = *reinterpret_cast<const float4*>(sc[buf][t]);
                 const float vo = COLS == 2 ? ((sub & 1) ? v[COLS - 1] : v[0]) : v[0];
                 const float ub = f.z * (vo - dk * f.x) * f.x;             // u times the key's normaliser: S += (k rk) u
-                if (writer) out[((int64_t)(sp.q0 + i0 + t) * H + h) * vdim + ocol] = fmaf(ub, f.w, oq * f.y);
+                if (writer) out[((int64_t)(sp.q0 + i0 + t) * H + h) * vcols + ocol] = fmaf(ub, f.w, oq * f.y);
                 float u[COLS];
                 if constexpr (COLS == 2) {
                     const float other = __shfl_xor_sync(0xffffffffu, ub, 1);
@@ -339,7 +377,7 @@ __global__ void __launch_bounds__(MS_THREADS) matrix_state_kernel(
                     }
                 }
                 const float oq = reduce(o);
-                if (writer) out[((int64_t)(sp.q0 + i0 + t) * H + h) * vdim + ocol] = oq;
+                if (writer) out[((int64_t)(sp.q0 + i0 + t) * H + h) * vcols + ocol] = oq;
             }
         }
         if (more) {
@@ -351,7 +389,7 @@ __global__ void __launch_bounds__(MS_THREADS) matrix_state_kernel(
     }
 #pragma unroll
     for (int c = 0; c < COLS; ++c) {
-        if (mycol + c >= vdim) break;
+        if (mycol + c >= vcols) break;
         float* sr = st + (int64_t)(mycol + c) * dim;
         if (vec_state) {
 #pragma unroll
@@ -474,10 +512,12 @@ constexpr int CF_RK = 0, CF_RQ = 4, CF_A = 8, CF_B = 14, CF_W = 24;
 template <typename T, int DPL, int COLS, bool CH, bool DELTA>
 __global__ void __launch_bounds__(MB_THREADS, DPL <= 16 ? 2 : 1) matrix_state_block_kernel(
     const T* __restrict__ x, int64_t stride, int q_off, int k_off, int v_off, const float* __restrict__ write_in,
-    const T* __restrict__ write_t, int64_t write_stride, DecayIn dec, float* __restrict__ state, const int32_t* __restrict__ state_slots,
-    const int32_t* __restrict__ cu_q, const int32_t* __restrict__ cu_k, const int32_t* __restrict__ ctx_lens, float* __restrict__ out, int H,
-    int G, int dim, int vdim, float q_scale, int vec_x, int vec_g) {
+    const T* __restrict__ write_t, int64_t write_stride, DecayIn dec, ScalarGate<T> sg, float* __restrict__ state,
+    const int32_t* __restrict__ state_slots, const int32_t* __restrict__ cu_q, const int32_t* __restrict__ cu_k,
+    const int32_t* __restrict__ ctx_lens, float* __restrict__ out, int H, int G, int dim, int vdim, int ones, float q_scale, int vec_x, int vec_g) {
     B200_PDL_SYNC();
+    constexpr bool LIN = !CH && !DELTA;
+    const int vcols = LIN ? vdim + ones : vdim;            // columns of the state
     using SH = BlockShape<DPL, COLS>;
     constexpr int FULL = 1, EMPTY = 3;
     extern __shared__ __align__(16) float mb_smem[];       // two stages
@@ -495,13 +535,16 @@ __global__ void __launch_bounds__(MB_THREADS, DPL <= 16 ? 2 : 1) matrix_state_bl
         const T* kp = x + k_off + (int64_t)(h / (H / G)) * dim + c0;
         const T* vp = x + v_off + (int64_t)h * vdim + col0;
         const float* gp = CH ? dec.in + (int64_t)h * dim + c0 : dec.in + h;
-        const float rt = dec.rate[h];
+        const float* rate = LIN ? sg.rate : dec.rate;
+        const float rt = rate ? rate[h] : 0.f;
         float gb[CH ? CPL : 1];
 #pragma unroll
-        for (int e = 0; e < (CH ? CPL : 1); ++e) gb[e] = CH ? (e < avail ? dec.bias[(int64_t)h * dim + c0 + e] : 0.f) : dec.bias[h];
+        for (int e = 0; e < (CH ? CPL : 1); ++e)
+            gb[e] = CH ? (e < avail ? dec.bias[(int64_t)h * dim + c0 + e] : 0.f) : rate ? (LIN ? sg.bias : dec.bias)[h] : 0.f;
         constexpr int VPL = MB_T * SH::GC / 32;             // value elements of a block per lane
         RawCols<T, CPL> rk[MB_T], rq[MB_T];
         RawCols<float, CH ? CPL : 1> rg[MB_T];
+        float2 rs[MB_T];                                    // LIN: the tokens' gate inputs
         RawCols<T, 1> rv[VPL], rw;
         float rwf = 0.f;
         auto fetch = [&](int it) {
@@ -513,6 +556,7 @@ __global__ void __launch_bounds__(MB_THREADS, DPL <= 16 ? 2 : 1) matrix_state_bl
                 rk[t].load(kp + row * stride, have, vec_x);
                 rq[t].load(qp + row * stride, have, vec_x);
                 if constexpr (CH) rg[t].load(gp + row * dec.stride, have, vec_g);
+                else if constexpr (LIN) rs[t] = i0 + t < sp.qlen ? sg.fetch(row, h) : make_float2(0.f, 0.f);
                 else rg[t].load(gp + row * dec.stride, i0 + t < sp.qlen, false);
             }
 #pragma unroll
@@ -537,6 +581,15 @@ __global__ void __launch_bounds__(MB_THREADS, DPL <= 16 ? 2 : 1) matrix_state_bl
 #pragma unroll
                 for (int i = 0; i < 32; ++i) sum[i] = 0.f;
                 float pe[CPL], kd[MB_T][CPL], qd[MB_T][CPL], kr[MB_T][CPL];
+                float gt[MB_T], wt[MB_T];                   // LIN: decay and write weight of every token
+                if constexpr (LIN) {
+#pragma unroll
+                    for (int t = 0; t < MB_T; ++t) {
+                        const float2 f = sg.gates(rs[t], rt, gb[0]);
+                        gt[t] = i0 + t < sp.qlen ? expf(f.x) : 1.f;
+                        wt[t] = i0 + t < sp.qlen ? f.y : 0.f;
+                    }
+                }
 #pragma unroll
                 for (int e = 0; e < CPL; ++e) {
                     float g[MB_T], k[MB_T], q[MB_T];
@@ -544,8 +597,8 @@ __global__ void __launch_bounds__(MB_THREADS, DPL <= 16 ? 2 : 1) matrix_state_bl
                     for (int t = 0; t < MB_T; ++t) {
                         k[t] = rk[t].at(e);
                         q[t] = rq[t].at(e);
-                        const float raw = rg[t].at(CH ? e : 0);
-                        g[t] = i0 + t < sp.qlen ? decay_of(raw, rt, gb[CH ? e : 0], dec.sign) : 1.f;
+                        if constexpr (LIN) g[t] = gt[t];
+                        else g[t] = i0 + t < sp.qlen ? decay_of(rg[t].at(CH ? e : 0), rt, gb[CH ? e : 0], dec.sign) : 1.f;
                     }
                     float p = 1.f;
 #pragma unroll
@@ -593,7 +646,12 @@ __global__ void __launch_bounds__(MB_THREADS, DPL <= 16 ? 2 : 1) matrix_state_bl
 #pragma unroll
                 for (int j = 0; j < VPL; ++j) {
                     const int e = lane + 32 * j;
-                    sm[SH::VS + b * MB_T * SH::GC + e] = rv[j].at(0);
+                    float v = rv[j].at(0);
+                    if constexpr (LIN) {
+                        if (ones && col0 + e % SH::GC == vdim) v = 1.0f;
+                        v *= wt[(32 * j) / SH::GC];             // a warp's 32 values belong to one token
+                    }
+                    sm[SH::VS + b * MB_T * SH::GC + e] = v;
                 }
                 // lane i ends with the warp's sum number i
 #pragma unroll
@@ -629,12 +687,12 @@ __global__ void __launch_bounds__(MB_THREADS, DPL <= 16 ? 2 : 1) matrix_state_bl
     // ---- consumers ----
     const int sub = lane & (MB_LANES - 1), grp = warp * 4 + (lane >> 3);
     const int mycol = col0 + grp * COLS;
-    float* stp = state + ((int64_t)state_slots[s] * H + h) * vdim * dim + sub * DPL;
+    float* stp = state + ((int64_t)state_slots[s] * H + h) * vcols * dim + sub * DPL;
     const bool has_hist = sp.klen - sp.qlen > 0, vec_state = dim % 4 == 0;
     uint64_t S[COLS][DPL / 2];
 #pragma unroll
     for (int c = 0; c < COLS; ++c) {
-        const bool have = has_hist && mycol + c < vdim;
+        const bool have = has_hist && mycol + c < vcols;
         const float* sr = stp + (int64_t)(mycol + c) * dim;
 #pragma unroll
         for (int k = 0; k < DPL / 4; ++k) {
@@ -659,11 +717,12 @@ __global__ void __launch_bounds__(MB_THREADS, DPL <= 16 ? 2 : 1) matrix_state_bl
     const int own = DELTA ? (sub & (COMBOS - 1)) / 2 : sub / (8 / COLS);   // this lane's column
     const int ocol = mycol + own;
     const bool odd = sub & 1;
+    const bool idle = col0 + warp * 4 * COLS >= vcols;      // no column of this warp exists: it only keeps the barriers company
     for (int it = 0; it < nst; ++it) {
         const int st = it & 1, i0 = it * MB_STAGE;
         const float* sm = mb_smem + st * SH::FLOATS;
         named_sync<FULL>(st);
-        for (int b = 0; b < MB_BLOCKS && i0 + b * MB_T < sp.qlen; ++b) {
+        for (int b = 0; b < MB_BLOCKS && i0 + b * MB_T < sp.qlen && !idle; ++b) {
             const float* cf = sm + SH::CF + b * 32;
             float w[COMBOS][MB_T];
 #pragma unroll
@@ -737,7 +796,7 @@ __global__ void __launch_bounds__(MB_THREADS, DPL <= 16 ? 2 : 1) matrix_state_bl
 #pragma unroll
                     for (int a = 0; a <= t; ++a) acc = fmaf(cf[CF_B + t * (t + 1) / 2 + a], mu[a], acc);
                     const int i = i0 + b * MB_T + t;
-                    if (odd && sub < COMBOS && ocol < vdim && i < sp.qlen) out[((int64_t)(sp.q0 + i) * H + h) * vdim + ocol] = acc * cf[CF_RQ + t];
+                    if (odd && sub < COMBOS && ocol < vcols && i < sp.qlen) out[((int64_t)(sp.q0 + i) * H + h) * vcols + ocol] = acc * cf[CF_RQ + t];
                 }
             } else {
 #pragma unroll
@@ -771,7 +830,7 @@ __global__ void __launch_bounds__(MB_THREADS, DPL <= 16 ? 2 : 1) matrix_state_bl
 #pragma unroll
                     for (int a = 0; a < MB_T; ++a)
                         if (a <= t) acc = fmaf(cf[CF_B + t * (t + 1) / 2 + a], mv[a], acc);
-                    if (ocol < vdim && i < sp.qlen) out[((int64_t)(sp.q0 + i) * H + h) * vdim + ocol] = acc;
+                    if (ocol < vcols && i < sp.qlen) out[((int64_t)(sp.q0 + i) * H + h) * vcols + ocol] = acc;
                 }
             }
             const float* pe = sm + SH::PE + b * SH::ROW + sub * SH::SEG;
@@ -800,7 +859,7 @@ __global__ void __launch_bounds__(MB_THREADS, DPL <= 16 ? 2 : 1) matrix_state_bl
     }
 #pragma unroll
     for (int c = 0; c < COLS; ++c) {
-        if (mycol + c >= vdim) break;
+        if (mycol + c >= vcols) break;
         float* sr = stp + (int64_t)(mycol + c) * dim;
 #pragma unroll
         for (int k = 0; k < DPL / 4; ++k) {
@@ -822,8 +881,9 @@ template <typename T, bool CH, bool DELTA>
 int launch_matrix_state(const void* x, int64_t stride, int q_off, int k_off, int v_off, const float* write_in, const void* write_t,
                         int64_t write_stride, const DecayIn& dec, float* state, const int32_t* state_slots, const int32_t* cu_q,
                         const int32_t* cu_k, const int32_t* ctx_lens, float* out, int total_rows, int num_seqs, int max_q, int H, int G, int dim,
-                        int vdim, float q_scale, cudaStream_t st) {
+                        int vdim, float q_scale, cudaStream_t st, const ScalarGate<T>& sg = {}, int ones = 0) {
     if (dim > 256) return B200_EUNSUPPORTED;
+    const int vcols = vdim + ones;
 #define MB_GO(DPL, COLS)                                                                                                           \
     do {                                                                                                                           \
         using SH = BlockShape<DPL, COLS>;                                                                                          \
@@ -834,9 +894,9 @@ int launch_matrix_state(const void* x, int64_t stride, int q_off, int k_off, int
         const int vx = dim % CPL == 0 && stride % CPL == 0 && q_off % CPL == 0 && k_off % CPL == 0 &&                              \
                        reinterpret_cast<uintptr_t>(x) % 16 == 0;                                                                   \
         const int vg = CH && dim % CPL == 0 && dec.stride % (CPL < 4 ? CPL : 4) == 0 && reinterpret_cast<uintptr_t>(dec.in) % 16 == 0;  \
-        B200_LAUNCH((matrix_state_block_kernel<T, DPL, COLS, CH, DELTA>), dim3(H, num_seqs, (vdim + SH::GC - 1) / SH::GC), MB_THREADS,  \
+        B200_LAUNCH((matrix_state_block_kernel<T, DPL, COLS, CH, DELTA>), dim3(H, num_seqs, (vcols + SH::GC - 1) / SH::GC), MB_THREADS, \
                     smem, st, static_cast<const T*>(x), stride, q_off, k_off, v_off, write_in, static_cast<const T*>(write_t),     \
-                    write_stride, dec, state, state_slots, cu_q, cu_k, ctx_lens, out, H, G, dim, vdim, q_scale, vx, vg);           \
+                    write_stride, dec, sg, state, state_slots, cu_q, cu_k, ctx_lens, out, H, G, dim, vdim, ones, q_scale, vx, vg); \
         return b200_launch_status(nullptr);                                                                                        \
     } while (0)
     if (cu_q != nullptr && max_q > MB_T) {                  // prompt portions: four tokens at a time
@@ -856,9 +916,9 @@ int launch_matrix_state(const void* x, int64_t stride, int q_off, int k_off, int
 #define MS_GO(DPL, LANES, COLS)                                                                                                    \
     do {                                                                                                                           \
         constexpr int GC = MS_THREADS / LANES * COLS;                                                                              \
-        B200_LAUNCH((matrix_state_kernel<T, DPL, LANES, COLS, CH, DELTA>), dim3(H, num_seqs, (vdim + GC - 1) / GC), MS_THREADS, 0, st,  \
+        B200_LAUNCH((matrix_state_kernel<T, DPL, LANES, COLS, CH, DELTA>), dim3(H, num_seqs, (vcols + GC - 1) / GC), MS_THREADS, 0, st, \
                     static_cast<const T*>(x), stride, q_off, k_off, v_off, write_in, static_cast<const T*>(write_t), write_stride, dec, \
-                    state, state_slots, cu_q, cu_k, ctx_lens, out, H, G, dim, vdim, q_scale);                                       \
+                    sg, state, state_slots, cu_q, cu_k, ctx_lens, out, H, G, dim, vdim, ones, q_scale);                             \
         return b200_launch_status(nullptr);                                                                                        \
     } while (0)
     if (dim <= 16) MS_GO(4, 4, 1);
@@ -870,22 +930,80 @@ int launch_matrix_state(const void* x, int64_t stride, int q_off, int k_off, int
     return B200_EUNSUPPORTED;
 }
 
+// Exponential gates of a matrix memory: from pre-activations (i | f) of H heads each, i <- cap tanh((i + b) / cap), f <- logsigmoid(cap
+// tanh((f + b) / cap)), the running maximum m_t = max(f_t + m_(t-1), i_t) (from 0 for a new sequence), and with it
+//     log_decay = f_t + m_(t-1) - m_t,   write = exp(i_t - m_t),   floor = exp(-m_t)                        (all fp32)
+// One warp per (sequence, head), 32 tokens per step: (f, i) pairs compose as (f1 + f2, max(i1 + f2, i2)), a scan over the lanes.
+__global__ void __launch_bounds__(128) mlstm_gates_kernel(const float* __restrict__ in, int64_t stride, const float* __restrict__ bias, float cap,
+                                                          float* __restrict__ mstate, const int32_t* __restrict__ state_slots,
+                                                          const int32_t* __restrict__ cu_q, const int32_t* __restrict__ cu_k,
+                                                          const int32_t* __restrict__ ctx_lens, float* __restrict__ log_decay,
+                                                          float* __restrict__ write, float* __restrict__ flr, int H) {
+    B200_PDL_SYNC();
+    const int s = blockIdx.y, h = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+    const SeqSpan sp = seq_span(cu_q, cu_k, ctx_lens, s);
+    if (sp.qlen <= 0 || h >= H) return;
+    float* mp = mstate + (int64_t)state_slots[s] * H + h;
+    float m = sp.klen - sp.qlen > 0 ? *mp : 0.f;
+    const float bi = bias[h], bf = bias[H + h];
+    float ri = 0.f, rf = 0.f;
+    auto fetch = [&](int i0) {
+        if (i0 + lane < sp.qlen) {
+            const float* row = in + (int64_t)(sp.q0 + i0 + lane) * stride + h;
+            ri = row[0], rf = row[H];
+        }
+    };
+    fetch(0);
+    for (int i0 = 0; i0 < sp.qlen; i0 += 32) {
+        const bool ok = i0 + lane < sp.qlen;
+        const float gi = cap * tanhf((ri + bi) / cap), gf = -softplus_(-cap * tanhf((rf + bf) / cap));
+        fetch(i0 + 32);
+        float F = ok ? gf : 0.f, I = ok ? gi : -INFINITY;
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) {
+            const float pf = __shfl_up_sync(0xffffffffu, F, o), pi = __shfl_up_sync(0xffffffffu, I, o);
+            if (lane >= o) {
+                I = fmaxf(pi + F, I);
+                F += pf;
+            }
+        }
+        const float mt = fmaxf(F + m, I);
+        float prev = __shfl_up_sync(0xffffffffu, mt, 1);
+        if (lane == 0) prev = m;
+        if (ok) {
+            const int64_t at = (int64_t)(sp.q0 + i0 + lane) * H + h;
+            log_decay[at] = gf + prev - mt;
+            write[at] = expf(gi - mt);
+            flr[at] = expf(-mt);
+        }
+        m = __shfl_sync(0xffffffffu, mt, 31);                // lanes past the end carry the last token's maximum on
+    }
+    if (lane == 0) *mp = m;
+}
+
 // out[t, h, :] = c * o / sqrt(mean(o^2) + eps) * w * act(gate[t, h, :]) for o = x[t, h, :] (fp32), one warp per (token, head).
-// act 0: sigmoid, 1: silu.  w (optional): [vdim], shared by the heads.
+// act 0: sigmoid, 1: silu.  w (optional): [vdim], shared by the heads, or (w_heads) [H * vdim].  flr (optional, [n, H]): rows of x have one
+// more element z, and o is first divided by max(|z|, flr) + 1e-6.
 template <typename T>
-__global__ void __launch_bounds__(128) head_rmsnorm_gate_kernel(const float* __restrict__ x, const T* __restrict__ w, const T* __restrict__ gate,
-                                                                int64_t gate_stride, int act, T* __restrict__ out, int64_t out_stride,
-                                                                float out_scale, int64_t rows, int H, int vdim, float eps) {
+__global__ void __launch_bounds__(128) head_rmsnorm_gate_kernel(const float* __restrict__ x, const float* __restrict__ flr, const T* __restrict__ w,
+                                                                int w_heads, const T* __restrict__ gate, int64_t gate_stride, int act,
+                                                                T* __restrict__ out, int64_t out_stride, float out_scale, int64_t rows, int H,
+                                                                int vdim, float eps) {
     B200_PDL_SYNC();
     const int64_t r = (int64_t)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
     if (r >= rows) return;
     const int lane = threadIdx.x & 31;
     const int64_t t = r / H;
     const int h = (int)(r - t * H);
-    const float* o = x + r * vdim;
+    const float* o = x + r * (vdim + (flr ? 1 : 0));
+    const float inv = flr ? 1.0f / (fmaxf(fabsf(o[vdim]), flr[r]) + 1e-6f) : 1.0f;
+    if (w && w_heads) w += (int64_t)h * vdim;
     float ss = 0.f;
-    for (int c = lane; c < vdim; c += 32) ss = fmaf(o[c], o[c], ss);
-    const float rstd = 1.0f / sqrtf(warp_sum(ss) / (float)vdim + eps);
+    for (int c = lane; c < vdim; c += 32) {
+        const float v = o[c] * inv;
+        ss = fmaf(v, v, ss);
+    }
+    const float rstd = inv / sqrtf(warp_sum(ss) / (float)vdim + eps);
     for (int c = lane; c < vdim; c += 32) {
         float v = o[c] * rstd;
         if (w) v *= ldf(w + c);
@@ -894,6 +1012,79 @@ __global__ void __launch_bounds__(128) head_rmsnorm_gate_kernel(const float* __r
             v *= act ? siluf_(z) : sigmoidf_(z);
         }
         stf(out + t * out_stride + (int64_t)h * vdim + c, v * out_scale);
+    }
+}
+
+// The close of a state-space mixer: t = (y[r, h, :] + D_h x[r, h, :]) * silu(z[r, :]), then every one of `groups` equal parts of the row
+// divided by its own root mean square, times w.  One CTA per (row, part); V columns per access, PER such groups per thread stay
+// in registers (wider parts are formed again).
+template <typename T, int V, int PER>
+__global__ void __launch_bounds__(128) skip_gate_groupnorm_kernel(const float* __restrict__ y, const T* __restrict__ x, int64_t x_stride,
+                                                                  const float* __restrict__ D, const T* __restrict__ z, int64_t z_stride,
+                                                                  const T* __restrict__ w, T* __restrict__ out, int64_t out_stride,
+                                                                  int inner, int vdim, int part, float eps) {
+    B200_PDL_SYNC();
+    __shared__ float red[4];
+    const int64_t row = blockIdx.x;
+    const int p0 = blockIdx.y * part;
+    auto ld = [](const auto* p, float (&f)[V]) {
+        if constexpr (V == 1) {
+            f[0] = ldf(p);
+        } else if constexpr (sizeof(*p) == 4) {
+            const float4 v = *reinterpret_cast<const float4*>(p);
+            f[0] = v.x, f[1] = v.y, f[2] = v.z, f[3] = v.w;
+        } else {
+            const uint2 v = *reinterpret_cast<const uint2*>(p);
+            f[0] = bf16lo(v.x), f[1] = bf16hi(v.x), f[2] = bf16lo(v.y), f[3] = bf16hi(v.y);
+        }
+    };
+    auto gated = [&](int c, float (&f)[V]) {
+        float a[V], b[V];
+        ld(y + row * inner + c, f);
+        ld(x + row * x_stride + c, a);
+        ld(z + row * z_stride + c, b);
+        const float d = D[c / vdim];                         // V columns never straddle two heads
+#pragma unroll
+        for (int e = 0; e < V; ++e) f[e] = fmaf(d, a[e], f[e]) * siluf_(b[e]);
+    };
+    const int step = 128 * V;
+    float r[PER][V];
+    float q = 0.f;
+#pragma unroll
+    for (int k = 0; k < PER; ++k) {
+        const int c = threadIdx.x * V + k * step;
+#pragma unroll
+        for (int e = 0; e < V; ++e) r[k][e] = 0.f;
+        if (c < part) gated(p0 + c, r[k]);
+#pragma unroll
+        for (int e = 0; e < V; ++e) q = fmaf(r[k][e], r[k][e], q);
+    }
+    for (int c = threadIdx.x * V + PER * step; c < part; c += step) {
+        float f[V];
+        gated(p0 + c, f);
+#pragma unroll
+        for (int e = 0; e < V; ++e) q = fmaf(f[e], f[e], q);
+    }
+    const float rstd = 1.0f / sqrtf(block_sum(q, red) / (float)part + eps);
+    auto emit = [&](int c, const float (&f)[V]) {
+        float g[V];
+        ld(w + c, g);
+#pragma unroll
+        for (int e = 0; e < V; ++e) g[e] *= f[e] * rstd;
+        T* o = out + row * out_stride + c;
+        if constexpr (V == 1) stf(o, g[0]);
+        else if constexpr (sizeof(T) == 4) *reinterpret_cast<float4*>(o) = make_float4(g[0], g[1], g[2], g[3]);
+        else *reinterpret_cast<uint2*>(o) = make_uint2(pack_bf16x2(g[0], g[1]), pack_bf16x2(g[2], g[3]));
+    };
+#pragma unroll
+    for (int k = 0; k < PER; ++k) {
+        const int c = threadIdx.x * V + k * step;
+        if (c < part) emit(p0 + c, r[k]);
+    }
+    for (int c = threadIdx.x * V + PER * step; c < part; c += step) {
+        float f[V];
+        gated(p0 + c, f);
+        emit(p0 + c, f);
     }
 }
 
@@ -970,14 +1161,63 @@ extern "C" int b200m_channel_state(const void* x, int64_t stride, int q_off, int
     return B200_EUNSUPPORTED;
 }
 
-extern "C" int b200m_head_rmsnorm_gate(const float* x, const void* w, const void* gate, int64_t gate_stride, int act, void* out,
-                                       int64_t out_stride, float out_scale, int n, int num_heads, int vdim, float eps, int is32,
+extern "C" int b200m_mlstm_gates(const float* in, int64_t stride, const float* bias, float cap, float* m_state, const int32_t* state_slots,
+                                 const int32_t* cu_q, const int32_t* cu_k, const int32_t* ctx_lens, float* log_decay, float* write, float* floor,
+                                 int num_seqs, int num_heads, void* stream) {
+    if (!in || !bias || !m_state || !state_slots || !log_decay || !write || !floor || num_heads <= 0 || !(cap > 0.f) || stride < 2 * num_heads)
+        return B200_EINVAL;
+    if ((cu_q == nullptr) != (cu_k == nullptr) || (cu_q == nullptr && ctx_lens == nullptr)) return B200_EINVAL;
+    if (num_seqs <= 0) return B200_OK;
+    B200_LAUNCH((mlstm_gates_kernel), dim3((num_heads + 3) / 4, num_seqs), 128, 0, static_cast<cudaStream_t>(stream), in, stride, bias, cap, m_state,
+                state_slots, cu_q, cu_k, ctx_lens, log_decay, write, floor, num_heads);
+    return b200_launch_status(nullptr);
+}
+
+extern "C" int b200m_linear_state(const void* x, int64_t stride, int q_off, int k_off, int v_off, const void* step_in, const float* log_decay,
+                                  const float* write, int64_t gate_stride, const float* rate, const float* bias, float* state,
+                                  const int32_t* state_slots, const int32_t* cu_q, const int32_t* cu_k, const int32_t* ctx_lens, float* out,
+                                  int num_seqs, int max_q, int num_heads, int num_kv_heads, int dim, int vdim, int ones, float q_scale,
+                                  int is32, void* stream) {
+    if (!x || !state || !state_slots || !out || (step_in ? (!rate || !bias) : (!log_decay || !write))) return B200_EINVAL;
+    if ((cu_q == nullptr) != (cu_k == nullptr) || (cu_q == nullptr && ctx_lens == nullptr)) return B200_EINVAL;
+    if (num_heads <= 0 || num_kv_heads <= 0 || num_heads % num_kv_heads || dim <= 0 || vdim <= 0 || ones < 0 || ones > 1) return B200_EINVAL;
+    if (num_seqs <= 0) return B200_OK;
+    B200M_DISPATCH(is32, const ScalarGate<T> sg = (ScalarGate<T>{static_cast<const T*>(step_in), log_decay, write, gate_stride, step_in ? rate : nullptr, bias});
+                   return (launch_matrix_state<T, false, false>(x, stride, q_off, k_off, v_off, nullptr, nullptr, 0, DecayIn{}, state, state_slots,
+                                                                cu_q, cu_k, ctx_lens, out, 0, num_seqs, max_q, num_heads, num_kv_heads, dim, vdim,
+                                                                q_scale, static_cast<cudaStream_t>(stream), sg, ones)));
+    return B200_EUNSUPPORTED;
+}
+
+extern "C" int b200m_skip_gate_groupnorm(const float* y, const void* x, int64_t x_stride, const float* D, const void* z, int64_t z_stride,
+                                         const void* w, void* out, int64_t out_stride, int n, int num_heads, int vdim, int groups, float eps,
+                                         int is32, void* stream) {
+    const int inner = num_heads * vdim;
+    if (!y || !x || !D || !z || !w || !out || n < 0 || num_heads <= 0 || vdim <= 0 || groups <= 0 || inner % groups) return B200_EINVAL;
+    if (n == 0) return B200_OK;
+    const int part = inner / groups;
+    cudaStream_t st = static_cast<cudaStream_t>(stream);
+    const uintptr_t bits = reinterpret_cast<uintptr_t>(y) | reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(z) |
+                           reinterpret_cast<uintptr_t>(w) | reinterpret_cast<uintptr_t>(out);
+    const bool vec = bits % 16 == 0 && vdim % 4 == 0 && part % 4 == 0 && x_stride % 4 == 0 && z_stride % 4 == 0 && out_stride % 4 == 0;
+#define SGG_GO(V, PER)                                                                                                             \
+    B200M_DISPATCH(is32, B200_LAUNCH((skip_gate_groupnorm_kernel<T, V, PER>), dim3(n, groups), 128, 0, st, y, static_cast<const T*>(x), x_stride, D, \
+                                     static_cast<const T*>(z), z_stride, static_cast<const T*>(w), static_cast<T*>(out), out_stride, inner, vdim, part, eps))
+    if (vec && part <= 512) SGG_GO(4, 1);
+    else if (vec) SGG_GO(4, 4);
+    else SGG_GO(1, 4);
+#undef SGG_GO
+    return b200_launch_status(nullptr);
+}
+
+extern "C" int b200m_head_rmsnorm_gate(const float* x, const float* floor, const void* w, int w_heads, const void* gate, int64_t gate_stride, int act,
+                                       void* out, int64_t out_stride, float out_scale, int n, int num_heads, int vdim, float eps, int is32,
                                        void* stream) {
     if (!x || !out || n < 0 || num_heads <= 0 || vdim <= 0) return B200_EINVAL;
     if (n == 0) return B200_OK;
     const int64_t rows = (int64_t)n * num_heads;
-    B200M_DISPATCH(is32, B200_LAUNCH((head_rmsnorm_gate_kernel<T>), (unsigned)((rows + 3) / 4), 128, 0, static_cast<cudaStream_t>(stream), x,
-                                     static_cast<const T*>(w), static_cast<const T*>(gate), gate_stride, act, static_cast<T*>(out),
+    B200M_DISPATCH(is32, B200_LAUNCH((head_rmsnorm_gate_kernel<T>), (unsigned)((rows + 3) / 4), 128, 0, static_cast<cudaStream_t>(stream), x, floor,
+                                     static_cast<const T*>(w), w_heads, static_cast<const T*>(gate), gate_stride, act, static_cast<T*>(out),
                                      out_stride, out_scale, rows, num_heads, vdim, eps));
     return b200_launch_status(nullptr);
 }

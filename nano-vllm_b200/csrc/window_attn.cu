@@ -4,8 +4,9 @@
 // reads key/value head h / (H / G).  There is no rotation: position enters through the bias and the window only.
 //     s_ij = (q_i . k_j) * scale - slope[h] * (i - j),   visible: 0 <= i - j < window or j < keep_first   (window <= 0: every j <= i)
 //     or, with chunk > 0, the j <= i of i's own chunk of positions: j >= i - i % chunk
+//     with a soft cap, q_i . k_j * scale first becomes cap * tanh(. / cap)
 //     p = softmax over the visible j (with sinks: one more term exp(sink[h]) in the denominator, which has no value),
-//     out_i = sum_j p_ij v_j   (with a head gate: times sigmoid(gate[i, h]))
+//     out_i = out_scale * sum_j p_ij v_j   (with a gate: times sigmoid(gate[i, h]), or element by element sigmoid(gate[i, h * vdim + c]))
 // The kernels read whatever the cache rows hold: a design that rotates its keys stores them rotated (headnorm_rope_store_kernel).
 // Softmax statistics and the output accumulate in fp32 in both element types.
 //
@@ -15,7 +16,8 @@
 //   window_attn_kernel   : any mix of prompt portions and single tokens on the fp32 FMA pipe (one warp per (token, head),
 //                          key/value tiles shared by the warps of a CTA through shared memory)
 //   window_attn_mma_kernel (bf16): the same on the tensor cores, 64 (token, head) rows x 64-key tiles, double-buffered
-//                          asynchronous copies; single-token steps may split a long window over several CTAs
+//                          asynchronous copies; single-token steps may split a long window over several CTAs.  Head sizes other
+//                          than 32 / 64 / 128 (multiples of eight up to 128) run as 64 or 128 with zero columns
 #include "mix_common.cuh"
 
 namespace {
@@ -27,15 +29,24 @@ constexpr int WA_TILE = 32;
 struct RowRule {
     int window, keep_first, chunk;
     const float* sinks;           // [H] scores of the valueless extra term, or NULL
-    const void* gate;             // activation type, element (token, head) at token * gate_stride + head, or NULL
-    int64_t gate_stride;
+    float softcap;                // > 0: scaled scores s become softcap * tanh(s / softcap)
+    const void* gate;             // activation type, or NULL: element (token, head) at token * gate_stride + head, or with gate_cols > 0
+    int64_t gate_stride;          // element (token, head, c) at token * gate_stride + head * gate_cols + c
+    int gate_cols;
+    float out_scale;
     // first key (kept first tokens aside) that the row at position pos sees; never decreasing in pos
     __device__ __forceinline__ int first_key(int pos) const {
         return chunk > 0 ? pos - pos % chunk : window > 0 ? max(0, pos - window + 1) : 0;
     }
+    // what a whole head's result is multiplied with ...
     template <typename T>
-    __device__ __forceinline__ float gate_of(int64_t token, int h) const {
-        return gate ? sigmoidf_(ldf(static_cast<const T*>(gate) + token * gate_stride + h)) : 1.0f;
+    __device__ __forceinline__ float head_factor(int64_t token, int h) const {
+        return (gate && gate_cols == 0) ? out_scale * sigmoidf_(ldf(static_cast<const T*>(gate) + token * gate_stride + h)) : out_scale;
+    }
+    // ... and its element c besides
+    template <typename T>
+    __device__ __forceinline__ float elem_factor(int64_t token, int h, int c) const {
+        return gate_cols > 0 ? sigmoidf_(ldf(static_cast<const T*>(gate) + token * gate_stride + (int64_t)h * gate_cols + c)) : 1.0f;
     }
 };
 
@@ -187,6 +198,7 @@ __global__ void __launch_bounds__(WA_WARPS * 32) window_attn_kernel(
                 const float* kr = tile + lane * DS;
                 float a = 0.f;
                 for (int c = 0; c < dim; ++c) a = fmaf(myq[c], kr[c], a);
+                if (rule.softcap > 0.f) a = rule.softcap * tanhf(a / rule.softcap);
                 sc = a - slope * (float)(pos - j);
             }
             const float m_new = fmaxf(m, warp_max(sc));
@@ -208,14 +220,15 @@ __global__ void __launch_bounds__(WA_WARPS * 32) window_attn_kernel(
         }
     }
     if (active) {
-        const float inv = rule.gate_of<T>(sp.q0 + i, h) / l;
+        const float inv = rule.head_factor<T>(sp.q0 + i, h) / l;
         const int64_t o = (int64_t)(sp.q0 + i) * out_stride + ((int64_t)h * vsets + vs) * vdim;
 #pragma unroll
         for (int k = 0; k < OACC; ++k) {
             const int c = lane + 32 * k;
             if (c < vdim) {
-                if (out32) out32[o + c] = acc[k] * inv;
-                else stf(out + o + c, acc[k] * inv);
+                const float r = acc[k] * inv * rule.elem_factor<T>(sp.q0 + i, h, c);
+                if (out32) out32[o + c] = r;
+                else stf(out + o + c, r);
             }
         }
     }
@@ -284,6 +297,12 @@ __device__ __forceinline__ float wm_ex2(float x) {       // 2^x on the special-f
     asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
     return y;
 }
+// cap * tanh(x / cap) in base-2 units: cap2 = cap * log2(e), k = 2 log2(e) / cap * (what makes v the scaled score x); tanh(z) = 1 - 2 / (1 + e^2z)
+__device__ __forceinline__ float wm_softcap(float v, float k, float cap2) {
+    float r;
+    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.0f + wm_ex2(v * k)));
+    return fmaf(-2.0f * cap2, r, cap2);
+}
 __device__ __forceinline__ uint32_t wm_pack(float lo, float hi) {
     __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
     return *reinterpret_cast<uint32_t*>(&v);
@@ -291,13 +310,15 @@ __device__ __forceinline__ uint32_t wm_pack(float lo, float hi) {
 
 // KS (single-token steps with at most 16 query heads per key/value head): the CTA's 16 rows are shared by its four warps, each
 // of which takes 16 of a tile's 64 keys with its own running (max, sum, O); the four are merged through shared memory at the end.
-template <int DK, int DV, bool KS, bool QREG, int BN>
+// PAD: dim <= DK and vdim <= DV (multiples of eight) elements are in memory, the rest of a tile's columns is zero.
+template <int DK, int DV, bool KS, bool QREG, int BN, bool PAD>
 __global__ void __launch_bounds__(128) window_attn_mma_kernel(
     const __nv_bfloat16* __restrict__ q, int64_t q_stride, const __nv_bfloat16* __restrict__ cache, int row_elems, int v_off,
     const int32_t* __restrict__ block_tables, int bt_stride, int block_size, int bs_shift, const int32_t* __restrict__ cu_q,
     const int32_t* __restrict__ cu_k, const int32_t* __restrict__ ctx_lens, const float* __restrict__ slopes, RowRule rule,
-    int vsets, __nv_bfloat16* __restrict__ out, float* __restrict__ out32, int64_t out_stride, int H, int G, float scale, int splits,
-    float* __restrict__ part) {
+    int vsets, __nv_bfloat16* __restrict__ out, float* __restrict__ out32, int64_t out_stride, int H, int G, int dim_, int vdim_, float scale,
+    int splits, float* __restrict__ part) {
+    const int dk = PAD ? dim_ : DK, dv = PAD ? vdim_ : DV;
     static_assert(!KS || BN == 64, "the key-sharing form shares out 64-key tiles");
     B200_PDL_SYNC();
     constexpr int KSTR = DK + 8, VSTR = DV + 8;           // row strides: 16-byte multiples, odd in 16-byte units (conflict-free ldmatrix)
@@ -358,9 +379,15 @@ __global__ void __launch_bounds__(128) window_attn_mma_kernel(
             const __nv_bfloat16* src = ok ? cache + ((int64_t)pg[p] * block_size + in_page) * row_elems : cache;
             const int nb = ok ? 16 : 0;
 #pragma unroll
-            for (int c = lc; c < KC; c += 8) wm_cp16(smem_u32(kd + r * KSTR + c * 8), ok ? src + g * DK + c * 8 : src, nb);
+            for (int c = lc; c < KC; c += 8) {
+                const bool in = ok && (!PAD || c * 8 < dk);
+                wm_cp16(smem_u32(kd + r * KSTR + c * 8), in ? src + g * dk + c * 8 : src, PAD ? (in ? 16 : 0) : nb);
+            }
 #pragma unroll
-            for (int c = lc; c < VC; c += 8) wm_cp16(smem_u32(vd + r * VSTR + c * 8), ok ? src + v_off + vh * DV + c * 8 : src, nb);
+            for (int c = lc; c < VC; c += 8) {
+                const bool in = ok && (!PAD || c * 8 < dv);
+                wm_cp16(smem_u32(vd + r * VSTR + c * 8), in ? src + v_off + vh * dv + c * 8 : src, PAD ? (in ? 16 : 0) : nb);
+            }
         }
         wm_commit();
     };
@@ -374,9 +401,9 @@ __global__ void __launch_bounds__(128) window_attn_mma_kernel(
         const int r = e / (DK / 8), c = e - r * (DK / 8);
         const int rr = row0 + r;
         uint4 v = make_uint4(0, 0, 0, 0);
-        if (rr < nrows) {
+        if (rr < nrows && (!PAD || c * 8 < dk)) {
             const int i = rr / rep, h = g * rep + (rr - i * rep);
-            v = *reinterpret_cast<const uint4*>(q + (int64_t)(sp.q0 + i) * q_stride + (int64_t)h * DK + c * 8);
+            v = *reinterpret_cast<const uint4*>(q + (int64_t)(sp.q0 + i) * q_stride + (int64_t)h * dk + c * 8);
         }
         *reinterpret_cast<uint4*>(Qs + r * KSTR + c * 8) = v;
     }
@@ -402,7 +429,9 @@ __global__ void __launch_bounds__(128) window_attn_mma_kernel(
     const int w_lo = rule.first_key(first + wr0 / rep);
     const int f_hi = wr0 + 15 < nrows ? first + wr0 / rep : -1;
     const int f_lo = rule.first_key(first + max(wr1, 0) / rep);
-    const float scale2 = scale * WM_LOG2E;
+    const bool capped = rule.softcap > 0.f;
+    const float scale2 = capped ? 1.0f : scale * WM_LOG2E;             // capped scores arrive scaled and in base-2 units
+    const float cap2 = rule.softcap * WM_LOG2E, capk = capped ? 2.0f * WM_LOG2E * scale / rule.softcap : 0.f;
 
     __syncthreads();                                                     // the queries are staged: keep this warp's fragments in registers
     const uint32_t a_base = smem_u32(Qs + (wrow + (lane & 15)) * KSTR + ((lane >> 4) << 3));
@@ -464,6 +493,12 @@ __global__ void __launch_bounds__(128) window_attn_mma_kernel(
 #pragma unroll
                     for (int x = 0; x < 4; ++x) bc[x] = bn[x];
                 }
+            }
+            if (capped) {
+#pragma unroll
+                for (int n = 0; n < WK / 8; ++n)
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) sc[n][e] = wm_softcap(sc[n][e], capk, cap2);
             }
             // scale, bias, mask; running maximum.  Inside the window of every row of the warp no mask is needed: two FMAs per score.
             float m_new[2] = {m_run[0], m_run[1]};
@@ -570,7 +605,7 @@ __global__ void __launch_bounds__(128) window_attn_mma_kernel(
         for (int e = tid; e < 16 * DV; e += 128) {
             const int r = e / DV, c = e - r * DV;
             const int rr = row0 + r;
-            if (rr >= nrows) continue;
+            if (rr >= nrows || (PAD && c >= dv)) continue;
             const float* pr = scr + (size_t)r * (DV + 2);
             constexpr int WSTEP = 16 * (DV + 2);
             float M = -INFINITY;
@@ -588,15 +623,16 @@ __global__ void __launch_bounds__(128) window_attn_mma_kernel(
             }
             const int i = rr / rep, hv = (g * rep + (rr - i * rep)) * vsets + vs;
             if (splits > 1) {
-                float* pp = part + (((int64_t)s * splits + split) * HV + hv) * (DV + 2);
+                float* pp = part + (((int64_t)s * splits + split) * HV + hv) * (dv + 2);
                 if (c == 0) {
                     pp[0] = M;
                     pp[1] = L;
                 }
                 pp[2 + c] = a;
             } else {
-                const float r = a / L * rule.gate_of<__nv_bfloat16>(sp.q0 + i, g * rep + (rr - i * rep));
-                const int64_t ob = (int64_t)(sp.q0 + i) * out_stride + (int64_t)hv * DV + c;
+                const int h = g * rep + (rr - i * rep);
+                const float r = a / L * rule.head_factor<__nv_bfloat16>(sp.q0 + i, h) * rule.elem_factor<__nv_bfloat16>(sp.q0 + i, h, c);
+                const int64_t ob = (int64_t)(sp.q0 + i) * out_stride + (int64_t)hv * dv + c;
                 if (out32) out32[ob] = r;
                 else out[ob] = __float2bfloat16_rn(r);
             }
@@ -608,27 +644,32 @@ __global__ void __launch_bounds__(128) window_attn_mma_kernel(
         if (rr >= nrows) continue;
         const int i = rr / rep, hv = (g * rep + (rr - i * rep)) * vsets + vs;
         if (splits > 1) {                                                // decode rows only (one token per sequence): i == 0
-            float* pp = part + (((int64_t)s * splits + split) * HV + hv) * (DV + 2);
+            float* pp = part + (((int64_t)s * splits + split) * HV + hv) * (dv + 2);
             if (t4 == 0) {
                 pp[0] = m_run[hh];
                 pp[1] = l_run[hh];
             }
 #pragma unroll
             for (int n = 0; n < DV / 8; ++n) {
+                if (PAD && n * 8 >= dv) break;
                 pp[2 + n * 8 + 2 * t4] = o[n][2 * hh];
                 pp[2 + n * 8 + 2 * t4 + 1] = o[n][2 * hh + 1];
             }
         } else {
-            const float inv = rule.gate_of<__nv_bfloat16>(sp.q0 + i, g * rep + (rr - i * rep)) / l_run[hh];
-            const int64_t ob = (int64_t)(sp.q0 + i) * out_stride + (int64_t)hv * DV;
-            if (out32) {
+            const int h = g * rep + (rr - i * rep);
+            const float inv = rule.head_factor<__nv_bfloat16>(sp.q0 + i, h) / l_run[hh];
+            const int64_t ob = (int64_t)(sp.q0 + i) * out_stride + (int64_t)hv * dv;
 #pragma unroll
-                for (int n = 0; n < DV / 8; ++n)
-                    *reinterpret_cast<float2*>(out32 + ob + n * 8 + 2 * t4) = make_float2(o[n][2 * hh] * inv, o[n][2 * hh + 1] * inv);
-            } else {
-#pragma unroll
-                for (int n = 0; n < DV / 8; ++n)
-                    *reinterpret_cast<uint32_t*>(out + ob + n * 8 + 2 * t4) = wm_pack(o[n][2 * hh] * inv, o[n][2 * hh + 1] * inv);
+            for (int n = 0; n < DV / 8; ++n) {
+                if (PAD && n * 8 >= dv) break;
+                const int c = n * 8 + 2 * t4;
+                float r0 = o[n][2 * hh] * inv, r1 = o[n][2 * hh + 1] * inv;
+                if (rule.gate_cols > 0) {
+                    r0 *= rule.elem_factor<__nv_bfloat16>(sp.q0 + i, h, c);
+                    r1 *= rule.elem_factor<__nv_bfloat16>(sp.q0 + i, h, c + 1);
+                }
+                if (out32) *reinterpret_cast<float2*>(out32 + ob + c) = make_float2(r0, r1);
+                else *reinterpret_cast<uint32_t*>(out + ob + c) = wm_pack(r0, r1);
             }
         }
     }
@@ -647,27 +688,28 @@ __global__ void window_merge_kernel(const float* __restrict__ part, const int32_
     for (int k = 0; k < splits; ++k) M = fmaxf(M, base[k * step]);
     float L = 0.f;
     for (int k = 0; k < splits; ++k) L += base[k * step + 1] * exp2f(base[k * step] - M);
-    const float inv = rule.gate_of<__nv_bfloat16>(s, h) / L;
+    const float inv = rule.head_factor<__nv_bfloat16>(s, h) / L;
     for (int c = threadIdx.x; c < vdim; c += blockDim.x) {
         float a = 0.f;
         for (int k = 0; k < splits; ++k) {
             const float mk = base[k * step];
             if (mk != -INFINITY) a = fmaf(base[k * step + 2 + c], exp2f(mk - M), a);
         }
-        if (out32) out32[s * out_stride + (int64_t)h * vdim + c] = a * inv;
-        else out[s * out_stride + (int64_t)h * vdim + c] = __float2bfloat16_rn(a * inv);
+        const float r = a * inv * rule.elem_factor<__nv_bfloat16>(s, h, c);
+        if (out32) out32[s * out_stride + (int64_t)h * vdim + c] = r;
+        else out[s * out_stride + (int64_t)h * vdim + c] = __float2bfloat16_rn(r);
     }
 }
 
-template <int DK, int DV, bool KS, bool QREG, int BN>
+template <int DK, int DV, bool KS, bool QREG, int BN, bool PAD>
 int launch_window_mma_as(const void* q, int64_t q_stride, const void* cache, int row_elems, int v_off, const int32_t* block_tables,
                          int bt_stride, int block_size, const int32_t* cu_q, const int32_t* cu_k, const int32_t* ctx_lens,
                          const float* slopes, const RowRule& rule, int vsets, void* out, int64_t out_stride, bool out_f32, int num_seqs, int max_q,
-                         int H, int G, float scale, int splits, float* part, cudaStream_t stream) {
+                         int H, int G, int dim, int vdim, float scale, int splits, float* part, cudaStream_t stream) {
     using bf = __nv_bfloat16;
     constexpr int BM = KS ? 16 : WM_BM;
     const size_t smem = sizeof(bf) * ((size_t)BM * (DK + 8) + 2 * (size_t)BN * (DK + 8) + 2 * (size_t)BN * (DV + 8));
-    int rc = wa_ensure_smem(window_attn_mma_kernel<DK, DV, KS, QREG, BN>, smem);
+    int rc = wa_ensure_smem(window_attn_mma_kernel<DK, DV, KS, QREG, BN, PAD>, smem);
     if (rc != B200_OK) return rc;
     int bs_shift = -1;
     if ((block_size & (block_size - 1)) == 0)
@@ -675,28 +717,28 @@ int launch_window_mma_as(const void* q, int64_t q_stride, const void* cache, int
     dim3 grid((max_q * (H / G) + BM - 1) / BM, num_seqs, G * vsets * splits);
     bf* out16 = out_f32 ? nullptr : static_cast<bf*>(out);
     float* out32 = out_f32 ? static_cast<float*>(out) : nullptr;
-    B200_LAUNCH((window_attn_mma_kernel<DK, DV, KS, QREG, BN>), grid, 128, smem, stream, static_cast<const bf*>(q), q_stride,
+    B200_LAUNCH((window_attn_mma_kernel<DK, DV, KS, QREG, BN, PAD>), grid, 128, smem, stream, static_cast<const bf*>(q), q_stride,
                 static_cast<const bf*>(cache), row_elems, v_off, block_tables, bt_stride, block_size, bs_shift, cu_q, cu_k, ctx_lens,
-                slopes, rule, vsets, out16, out32, out_stride, H, G, scale, splits, part);
+                slopes, rule, vsets, out16, out32, out_stride, H, G, dim, vdim, scale, splits, part);
     rc = b200_launch_status(nullptr);
     if (rc != B200_OK || splits <= 1) return rc;
     B200_LAUNCH((window_merge_kernel), dim3(num_seqs, H * vsets), DV < 64 ? 32 : 64, 0, stream, part, ctx_lens, out16, out32, out_stride, rule,
-                H * vsets, DV, splits);
+                H * vsets, vdim, splits);
     return b200_launch_status(nullptr);
 }
 
-template <int DK, int DV>
+template <int DK, int DV, bool PAD = false>
 int launch_window_mma(const void* q, int64_t q_stride, const void* cache, int row_elems, int v_off, const int32_t* block_tables,
                       int bt_stride, int block_size, const int32_t* cu_q, const int32_t* cu_k, const int32_t* ctx_lens,
                       const float* slopes, const RowRule& rule, int vsets, void* out, int64_t out_stride, bool out_f32, int num_seqs, int max_q, int H,
-                      int G, float scale, int splits, float* part, cudaStream_t stream) {
+                      int G, int dim, int vdim, float scale, int splits, float* part, cudaStream_t stream) {
     if (cu_q == nullptr && H / G <= 16)                   // single-token step: the four warps share every key tile
-        return launch_window_mma_as<DK, DV, true, true, 64>(q, q_stride, cache, row_elems, v_off, block_tables, bt_stride, block_size, cu_q, cu_k,
-                                                  ctx_lens, slopes, rule, vsets, out, out_stride, out_f32, num_seqs, max_q, H, G, scale, splits, part, stream);
+        return launch_window_mma_as<DK, DV, true, true, 64, PAD>(q, q_stride, cache, row_elems, v_off, block_tables, bt_stride, block_size, cu_q, cu_k,
+                                                  ctx_lens, slopes, rule, vsets, out, out_stride, out_f32, num_seqs, max_q, H, G, dim, vdim, scale, splits, part, stream);
     // row-tiled form: query fragments are re-read from shared memory per key tile (measured faster than 32 more live registers)
     // (32-key tiles, which let four CTAs instead of two share an SM at 128-wide heads, were measured and are not faster)
-    return launch_window_mma_as<DK, DV, false, false, 64>(q, q_stride, cache, row_elems, v_off, block_tables, bt_stride, block_size, cu_q, cu_k,
-                                                          ctx_lens, slopes, rule, vsets, out, out_stride, out_f32, num_seqs, max_q, H, G, scale, splits, part, stream);
+    return launch_window_mma_as<DK, DV, false, false, 64, PAD>(q, q_stride, cache, row_elems, v_off, block_tables, bt_stride, block_size, cu_q, cu_k,
+                                                          ctx_lens, slopes, rule, vsets, out, out_stride, out_f32, num_seqs, max_q, H, G, dim, vdim, scale, splits, part, stream);
 }
 
 }  // namespace
@@ -724,16 +766,17 @@ extern "C" int b200m_qk_norm_store(void* qkv, int64_t stride, int q_cols, int k_
 extern "C" int b200m_window_attention(const void* q, int64_t q_stride, const void* cache, int row_elems, int v_off,
                                       const int32_t* block_tables, int bt_stride, int block_size, const int32_t* cu_q,
                                       const int32_t* cu_k, const int32_t* ctx_lens, const float* slopes, int window, int keep_first,
-                                      int chunk, const float* sinks, const void* gate, int64_t gate_stride, int all_values, void* out, int64_t out_stride, int total_q, int num_seqs, int max_q, int num_heads, int num_kv_heads,
-                                      int dim, int vdim, float scale, int is32, int flags, int splits, float* part, void* stream) {
+                                      int chunk, const float* sinks, float softcap, const void* gate, int64_t gate_stride, int gate_elems,
+                                      float out_scale, int all_values, void* out, int64_t out_stride, int total_q, int num_seqs, int max_q,
+                                      int num_heads, int num_kv_heads, int dim, int vdim, float scale, int is32, int flags, int splits, float* part, void* stream) {
     if (!q || !cache || !block_tables || !out || total_q < 0 || num_seqs < 0 || num_heads <= 0 || num_kv_heads <= 0 ||
         num_heads % num_kv_heads || dim <= 0 || vdim <= 0 || block_size <= 0 || keep_first < 0 || chunk < 0 ||
-        (chunk > 0 && window > 0) || (gate && all_values))
+        (chunk > 0 && window > 0) || (gate && all_values) || softcap < 0.f)
         return B200_EINVAL;
     const int vsets = all_values ? num_kv_heads : 1;
     if (out_stride < (int64_t)num_heads * vsets * vdim) return B200_EINVAL;
     // kept first tokens belong to a window or a chunk: without one every earlier key is visible anyway
-    const RowRule rule{window, window > 0 || chunk > 0 ? keep_first : 0, chunk, sinks, gate, gate_stride};
+    const RowRule rule{window, window > 0 || chunk > 0 ? keep_first : 0, chunk, sinks, softcap, gate, gate_stride, gate && gate_elems ? vdim : 0, out_scale};
     const bool out_f32 = (flags & 2) != 0 && !is32;
     if ((cu_q == nullptr) != (cu_k == nullptr) || (cu_q == nullptr && ctx_lens == nullptr)) return B200_EINVAL;
     if (total_q == 0 || num_seqs == 0 || max_q <= 0) return B200_OK;
@@ -741,14 +784,15 @@ extern "C" int b200m_window_attention(const void* q, int64_t q_stride, const voi
     cudaStream_t st = static_cast<cudaStream_t>(stream);
     const bool aligned = ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(cache)) % 16 == 0) && q_stride % 8 == 0 &&
                          row_elems % 8 == 0 && v_off % 8 == 0 && out_stride % 2 == 0 && reinterpret_cast<uintptr_t>(out) % 8 == 0;
-    if (!is32 && !(flags & 1) && aligned && (dim == 32 || dim == 64 || dim == 128) && (vdim == 32 || vdim == 64 || vdim == 128)) {
+    if (!is32 && !(flags & 1) && aligned && dim % 8 == 0 && vdim % 8 == 0 && dim <= 128 && vdim <= 128) {
         if (cu_q != nullptr || splits < 1) splits = 1;                  // keys are split for single-token steps only
         if (splits > 1 && !part) return B200_EINVAL;
-#define WA_MMA(DK, DV)                                                                                                           \
-    if (dim == DK && vdim == DV)                                                                                                 \
-        return launch_window_mma<DK, DV>(q, q_stride, cache, row_elems, v_off, block_tables, bt_stride, block_size, cu_q, cu_k,  \
-                                         ctx_lens, slopes, rule, vsets, out, out_stride, out_f32, num_seqs, max_q, num_heads,  \
-                                         num_kv_heads, scale, splits, part, st)
+#define WA_MMA_AS(DK, DV, PAD)                                                                                                       \
+    return launch_window_mma<DK, DV, PAD>(q, q_stride, cache, row_elems, v_off, block_tables, bt_stride, block_size, cu_q, cu_k,     \
+                                          ctx_lens, slopes, rule, vsets, out, out_stride, out_f32, num_seqs, max_q, num_heads,     \
+                                          num_kv_heads, dim, vdim, scale, splits, part, st)
+#define WA_MMA(DK, DV) \
+    if (dim == DK && vdim == DV) WA_MMA_AS(DK, DV, false)
         WA_MMA(32, 32);
         WA_MMA(32, 64);
         WA_MMA(32, 128);
@@ -758,7 +802,10 @@ extern "C" int b200m_window_attention(const void* q, int64_t q_stride, const voi
         WA_MMA(128, 32);
         WA_MMA(128, 64);
         WA_MMA(128, 128);
+        if (dim <= 64 && vdim <= 64) WA_MMA_AS(64, 64, true);            // other head sizes: zero columns up to the next tile
+        WA_MMA_AS(128, 128, true);
 #undef WA_MMA
+#undef WA_MMA_AS
     }
 #define WA_FMA(OACC)                                                                                                             \
     B200M_DISPATCH(is32, return (launch_window_fma<T, OACC>(q, q_stride, cache, row_elems, v_off, block_tables, bt_stride,       \
@@ -780,7 +827,8 @@ extern "C" int b200m_window_attention(const void* q, int64_t q_stride, const voi
 //
 //   headnorm_rope_store_kernel : per token and head, q <- rms_norm(q) * wq (one weight vector of `dim` elements shared by all
 //                                heads), the pairs (2i, 2i + 1) (or, by layout, (i, i + rope_dims / 2)), i < rope_dims / 2, turned
-//                                by the token's position, in place;
+//                                by the token's position, in place; or rotated first and then divided by the root mean square
+//                                of the head (unit_after: no weight);
 //                                keys the same with wk and scattered to the token's cache row; values divided by their root mean
 //                                square (no weight) and scattered next to the keys.  One warp per head, fp32 throughout, one
 //                                rounding at the store.
@@ -794,7 +842,7 @@ namespace {
 template <typename T>
 __global__ void __launch_bounds__(128) headnorm_rope_store_kernel(T* __restrict__ x, int64_t stride, int q_off, int k_off, int v_off, int H,
                                                                   int G, int dim, int vdim, const T* __restrict__ wq,
-                                                                  const T* __restrict__ wk, int v_unit, const float* __restrict__ cos_sin,
+                                                                  const T* __restrict__ wk, int v_unit, int unit_after, const float* __restrict__ cos_sin,
                                                                   int layout, int rope_dims, const float* __restrict__ v_cos_sin, int v_rope_dims,
                                                                   const int64_t* __restrict__ positions,
                                                                   const int32_t* __restrict__ slots, T* __restrict__ cache, float eps) {
@@ -827,6 +875,16 @@ __global__ void __launch_bounds__(128) headnorm_rope_store_kernel(T* __restrict_
         const float* rcs = (is_q || is_k) ? cs : vcs;
         const int rdims = rcs == nullptr ? 0 : (is_q || is_k) ? rope_dims : v_rope_dims, half = rdims / 2;
         const bool split = layout != 0 && (is_q || is_k);  // rotated pairs (i, i + half) instead of (2i, 2i + 1)
+        if (unit_after && (is_q || is_k)) {                // the rotation scales a pair's square by cos^2 + sin^2, whatever magnitude the table carries
+            float ss = 0.f;
+            for (int p = lane; 2 * p < d; p += 32) {
+                const int c0 = (split && p < half) ? p : 2 * p, c1 = (split && p < half) ? p + half : 2 * p + 1;
+                const float a = ldf(src + c0), b = c1 < d ? ldf(src + c1) : 0.f;
+                const float g = p < half ? fmaf(rcs[p], rcs[p], rcs[half + p] * rcs[half + p]) : 1.0f;
+                ss = fmaf(fmaf(a, a, b * b), g, ss);
+            }
+            rstd = 1.0f / sqrtf(warp_sum(ss) / (float)d + eps);
+        }
         for (int p = lane; 2 * p < d; p += 32) {           // a lane owns whole pairs: the rotated ones first, then the rest two at a time
             const int c0 = (split && p < half) ? p : 2 * p, c1 = (split && p < half) ? p + half : 2 * p + 1;
             float a = ldf(src + c0) * rstd, b = c1 < d ? ldf(src + c1) * rstd : 0.f;
@@ -970,19 +1028,20 @@ __global__ void __launch_bounds__(256) head_mix_gate_kernel(const A* __restrict_
 }  // namespace
 
 extern "C" int b200m_headnorm_rope_store(void* x, int64_t stride, int q_off, int k_off, int v_off, int num_heads, int num_kv_heads, int dim,
-                                         int vdim, const void* q_norm_w, const void* k_norm_w, int v_unit_norm, const float* cos_sin,
+                                         int vdim, const void* q_norm_w, const void* k_norm_w, int v_unit_norm, int unit_after, const float* cos_sin,
                                          int layout, int rope_dims, const float* v_cos_sin, int v_rope_dims, const int64_t* positions,
                                          const int32_t* slots, void* cache, int n, float eps, int is32, void* stream) {
     if (!x || n < 0 || num_heads <= 0 || num_kv_heads <= 0 || dim <= 0 || vdim <= 0 || rope_dims < 0 || rope_dims > dim || (rope_dims & 1))
         return B200_EINVAL;
     if ((cos_sin && rope_dims > 0 && !positions) || (cache && !slots)) return B200_EINVAL;
+    if (unit_after && (q_norm_w || k_norm_w)) return B200_EINVAL;        // one norm of q and k, before or after the rotation
     if (v_rope_dims < 0 || v_rope_dims > vdim || (v_rope_dims & 1) || (v_cos_sin && v_rope_dims > 0 && !positions)) return B200_EINVAL;
     if (v_rope_dims == 0) v_cos_sin = nullptr;
     if (n == 0) return B200_OK;
     if (rope_dims == 0) cos_sin = nullptr;
     B200M_DISPATCH(is32, B200_LAUNCH((headnorm_rope_store_kernel<T>), n, 128, 0, static_cast<cudaStream_t>(stream), static_cast<T*>(x), stride,
                                      q_off, k_off, v_off, num_heads, num_kv_heads, dim, vdim, static_cast<const T*>(q_norm_w),
-                                     static_cast<const T*>(k_norm_w), v_unit_norm, cos_sin, layout, rope_dims, v_cos_sin, v_rope_dims, positions, slots,
+                                     static_cast<const T*>(k_norm_w), v_unit_norm, unit_after, cos_sin, layout, rope_dims, v_cos_sin, v_rope_dims, positions, slots,
                                      static_cast<T*>(cache), eps));
     return b200_launch_status(nullptr);
 }

@@ -53,11 +53,11 @@ MIX_SIGNATURES = {
     "b200m_add_normed": (_i, [_vp, _vp, _vp, _vp, _f, _f, _vp, _i, _i, _f, _i, _vp]),
     "b200m_rmsnorm_rows": (_i, [_vp, _vp, _vp, _f, _vp, _i, _i, _f, _i, _vp]),
     "b200m_qk_norm_store": (_i, [_vp, _i64, _i, _i, _i, _vp, _vp, _vp, _vp, _i, _f, _i, _vp]),
-    "b200m_window_attention": (_i, [_vp, _i64, _vp, _i, _i, _vp, _i, _i, _vp, _vp, _vp, _vp, _i, _i, _i, _vp, _vp, _i64, _i, _vp, _i64, _i, _i, _i, _i,
-                                    _i, _i, _i, _f, _i, _i, _i, _vp, _vp]),
+    "b200m_window_attention": (_i, [_vp, _i64, _vp, _i, _i, _vp, _i, _i, _vp, _vp, _vp, _vp, _i, _i, _i, _vp, _f, _vp, _i64, _i, _f, _i, _vp, _i64,
+                                    _i, _i, _i, _i, _i, _i, _i, _f, _i, _i, _i, _vp, _vp]),
     "b200m_embed_pair": (_i, [_vp, _vp, _f, _vp, _i64, _i64, _i64, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i64, _i, _vp]),
     "b200m_add_normed_norm": (_i, [_vp, _vp, _vp, _vp, _f, _f, _vp, _vp, _f, _vp, _i, _i, _f, _i, _vp]),
-    "b200m_headnorm_rope_store": (_i, [_vp, _i64, _i, _i, _i, _i, _i, _i, _i, _vp, _vp, _i, _vp, _i, _i, _vp, _i, _vp, _vp, _vp, _i, _f, _i, _vp]),
+    "b200m_headnorm_rope_store": (_i, [_vp, _i64, _i, _i, _i, _i, _i, _i, _i, _vp, _vp, _i, _i, _vp, _i, _i, _vp, _i, _vp, _vp, _vp, _i, _f, _i, _vp]),
     "b200m_head_rotate_gate": (_i, [_vp, _i, _i64, _i64, _vp, _i, _i, _f, _vp, _vp, _i64, _vp, _i64, _i, _i, _i, _i, _vp]),
     "b200m_gated_add_normed_norm": (_i, [_vp, _vp, _vp, _vp, _i64, _vp, _vp, _f, _vp, _i, _i, _f, _i, _vp]),
     "b200m_ff_glu_clamped": (_i, [_vp, _i64, _vp, _i64, _i, _f, _f, _i, _vp]),
@@ -67,11 +67,16 @@ MIX_SIGNATURES = {
     "b200m_gated_delta": (_i, [_vp, _i64, _i, _i, _i, _vp, _i64, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _f, _i, _vp]),
     "b200m_channel_state": (_i, [_vp, _i64, _i, _i, _i, _vp, _i64, _vp, _i64, _vp, _vp, _f, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i,
                                  _i, _f, _i, _vp]),
-    "b200m_head_rmsnorm_gate": (_i, [_vp, _vp, _vp, _i64, _i, _vp, _i64, _f, _i, _i, _i, _f, _i, _vp]),
+    "b200m_linear_state": (_i, [_vp, _i64, _i, _i, _i, _vp, _vp, _vp, _i64, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _f,
+                                _i, _vp]),
+    "b200m_mlstm_gates": (_i, [_vp, _i64, _vp, _f, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _vp]),
+    "b200m_skip_gate_groupnorm": (_i, [_vp, _vp, _i64, _vp, _vp, _i64, _vp, _vp, _i64, _i, _i, _i, _i, _f, _i, _vp]),
+    "b200m_head_rmsnorm_gate": (_i, [_vp, _vp, _vp, _i, _vp, _i64, _i, _vp, _i64, _f, _i, _i, _i, _f, _i, _vp]),
     "b200m_moe_route_grouped": (_i, [_vp, _i64, _i, _i, _i, _vp, _i, _i, _i, _i, _i, _f, _vp, _vp, _vp]),
     "b200m_add_layernorm": (_i, [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _f, _i, _vp]),
     "b200m_rmsnorm": (_i, [_vp, _i64, _vp, _vp, _i64, _i, _i, _f, _i, _vp]),
     "b200m_add_layernorm2": (_i, [_vp, _vp, _vp, _f, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _f, _i, _vp]),
+    "b200m_add_rmsnorm": (_i, [_vp, _vp, _vp, _vp, _vp, _i, _i, _f, _f, _i, _vp]),
     "b200m_ff_act": (_i, [_vp, _vp, _i64, _i64, _i, _i, _i, _vp]),
     "b200m_latent_store": (_i, [_vp, _i64, _vp, _vp, _i, _vp, _vp, _vp, _i, _i, _i, _f, _i, _i, _vp]),
     "b200m_latent_attention": (_i, [_vp, _vp, _i64, _i, _i, _vp, _vp, _i, _i, _vp, _vp, _vp, _vp, _vp, _i, _vp, _i, _i, _i, _i, _i, _i,

@@ -114,6 +114,25 @@ class GatedScaledSandwich:
                                             w_next=then.w_in32 if then is not None else None)
 
 
+class PreNorm:
+    """The RMS norm in front of one sublayer of a pre-norm layer, ``x <- x + f(rms(x) * w)`` over an fp32 stream.  ``after`` closes the sublayer
+    before it (``x += y``) in the same pass; ``scale`` is a constant factor on the result."""
+
+    def __init__(self, width: int, eps: float, dtype, device, scale: float = 1.0):
+        self.eps, self.scale = eps, scale
+        self.weight = torch.ones(width, dtype=dtype, device=device)
+
+    def open(self, x, rows_idx=None):
+        """The norm of the stream (of the rows ``rows_idx``)."""
+        from .. import mixops
+        return mixops.add_rmsnorm(x, self.weight, self.eps, rows_idx=rows_idx, out_scale=self.scale)
+
+    def after(self, x, y):
+        """x += y in place; returns the norm of the result."""
+        from .. import mixops
+        return mixops.add_rmsnorm(x, self.weight, self.eps, y=y, out_scale=self.scale)
+
+
 class ParallelNorms:
     """The two biased layer norms of a parallel block, ``x <- x + m (f1(ln1(x)) + f2(ln2(x)))`` over an fp32 stream: both read the same x,
     so one pass forms the statistics once and writes both results.  ``advance`` closes a block (the scaled update with the summed

@@ -1,6 +1,6 @@
 """Feed-forward blocks of hybrid decoders: a gated dense block and a routed mixture of small experts.
 
-Dense:   W_down (gelu_tanh(W_gate h) * (W_up h))
+Dense:   W_down (act(W_gate h) * (W_up h)), act = the tanh form of GELU (``GatedDenseFF``) or SiLU (``SiluGatedDenseFF``)
 Biased:  W_down gelu_tanh(W_up h + b_up) + b_down
 Routed:  z = W_router h (fp32), s = sigmoid(z); the `top` experts with the largest s get weight s (not renormalised);
          the weight scales the expert's INPUT:  out = sum_e expert_e(s_e h),  expert(x) = W_down relu(W_up x)^2;
@@ -31,6 +31,8 @@ from .. import mixops
 
 
 class GatedDenseFF:
+    act = mixops.FF_GELU_TANH_MUL
+
     def __init__(self, width: int, mlp: dict, dtype, device, w_down=None):
         """``w_down`` (a view): this block's columns of an output projection that another branch shares (``ParallelBranches``)."""
         self.ff = int(mlp["ff"])
@@ -53,12 +55,16 @@ class GatedDenseFF:
         return {"gate": (self.ff, width), "up": (self.ff, width), "down": (width, self.ff)}
 
     def hidden(self, h: torch.Tensor, out: torch.Tensor | None = None) -> torch.Tensor:
-        """gelu_tanh(W_gate h) * (W_up h), the down projection's operand; ``out`` may be a row-strided view."""
-        return mixops.ff_act(F.linear(h, self.w_gate_up), mixops.FF_GELU_TANH_MUL, out=out)
+        """act(W_gate h) * (W_up h), the down projection's operand; ``out`` may be a row-strided view."""
+        return mixops.ff_act(F.linear(h, self.w_gate_up), self.act, out=out)
 
     def forward(self, h: torch.Tensor):
         """-> (T tensor, None)"""
         return F.linear(self.hidden(h), self.w_down), None
+
+
+class SiluGatedDenseFF(GatedDenseFF):
+    act = mixops.FF_SILU_MUL
 
 
 class BiasedDenseFF:

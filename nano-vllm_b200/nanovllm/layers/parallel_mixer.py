@@ -4,7 +4,7 @@
 Both read h, so their input projections are one GEMM over the merged rows ``[W_in_left ; W_in_right]`` (biases in the
 epilogue), and both end in an output projection, so ``c_l W_ol a + c_r W_or b = [W_ol | W_or] [c_l a ; c_r b]`` is one GEMM too:
 each mixer writes its scaled operand into its columns of one buffer.  The sub-mixers hold views into the merged weights and load
-their own tensors (``left.*`` / ``right.*``).
+their own tensors (``left.*`` / ``right.*``).  Each mixer's rows of the merged input projection start on a 16-byte column of its result.
 """
 from __future__ import annotations
 
@@ -23,13 +23,17 @@ class ParallelMixer:
         self.left_scale, self.right_scale = float(left_scale), float(right_scale)
         probe_l, probe_r = left_cls.projection_cols(left_cfg), right_cls.projection_cols(right_cfg)
         (li, lo), (ri, ro) = probe_l, probe_r
-        self.w_in = torch.empty(li + ri, width, dtype=dtype, device=device)
-        self.b_in = torch.zeros(li + ri, dtype=dtype, device=device)
+        pad8 = lambda n: -(-n // 8) * 8
+        start = pad8(li)                                  # where the right mixer's columns start
+        self.w_in = torch.zeros(pad8(start + ri), width, dtype=dtype, device=device)
+        bias = getattr(left_cls, "bias", True)
+        self.b_in = torch.zeros(self.w_in.shape[0], dtype=dtype, device=device) if bias else None
         self.w_o = torch.empty(width, lo + ro, dtype=dtype, device=device)
-        self.left = left_cls(width, left_cfg, dtype=dtype, device=device, w_in=self.w_in[:li], b_in=self.b_in[:li], w_o=self.w_o[:, :lo], **common)
-        self.right = right_cls(width, right_cfg, dtype=dtype, device=device, w_in=self.w_in[li:], w_o=self.w_o[:, lo:],
+        self.left = left_cls(width, left_cfg, dtype=dtype, device=device, w_in=self.w_in[:li], b_in=self.b_in[:li] if bias else None,
+                             w_o=self.w_o[:, :lo], **common)
+        self.right = right_cls(width, right_cfg, dtype=dtype, device=device, w_in=self.w_in[start:start + ri], w_o=self.w_o[:, lo:],
                                **{k: v for k, v in common.items() if k == "eps"})
-        self.split_in, self.split_out = li, lo
+        self.split_in, self.split_out = (li, start, start + ri), lo
 
     def load(self, leaf: str, w: torch.Tensor) -> bool:
         side, _, rest = leaf.partition(".")
@@ -58,9 +62,14 @@ class ParallelMixer:
         self.left.unbind()
         self.right.unbind()
 
+    def rotations(self):
+        """Sub-mixers whose rotation tables may be shared with other layers' (``rot_key``)."""
+        return [m for m in (self.left, self.right) if getattr(m, "cos_sin", None) is not None]
+
     def forward(self, h: torch.Tensor, positions, ctx, spans: mixops.StepSpans, inst: int = 0) -> torch.Tensor:
         proj = F.linear(h, self.w_in, self.b_in)
         both = torch.empty(h.shape[0], self.w_o.shape[1], dtype=self.dtype, device=self.device)
-        self.left.mix(proj[:, :self.split_in], h, positions, ctx, spans, inst, out=both[:, :self.split_out], out_scale=self.left_scale)
-        self.right.mix(proj[:, self.split_in:], h, positions, ctx, spans, inst, out=both[:, self.split_out:], out_scale=self.right_scale)
+        li, start, stop = self.split_in
+        self.left.mix(proj[:, :li], h, positions, ctx, spans, inst, out=both[:, :self.split_out], out_scale=self.left_scale)
+        self.right.mix(proj[:, start:stop], h, positions, ctx, spans, inst, out=both[:, self.split_out:], out_scale=self.right_scale)
         return F.linear(both, self.w_o)

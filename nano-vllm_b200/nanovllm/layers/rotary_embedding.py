@@ -64,6 +64,15 @@ def banded_frequencies(dims: int, base: float, scaling: dict | None = None) -> t
     return freq
 
 
+def build_scaled_cos_sin(dims: int, max_position: int, base: float, scaling: dict | None = None, device=None) -> torch.Tensor:
+    """The table for whichever frequency scaling the configuration names: {factor, original, fast, slow} is a ramp over the pair number
+    (``build_interleaved_cos_sin``), {factor, original, low, high} rescales by wavelength bands (``build_banded_cos_sin``).  The table does not
+    depend on which two elements form pair i."""
+    if scaling and "fast" in scaling:
+        return build_interleaved_cos_sin(dims, max_position, base, scaling, device)
+    return build_banded_cos_sin(dims, max_position, base, scaling, device)
+
+
 def build_banded_cos_sin(dims: int, max_position: int, base: float, scaling: dict | None = None, device=None) -> torch.Tensor:
     """fp32 ``[max_position, dims] = cat(cos, sin)`` of position * banded_frequencies: pair i of a rotated vector turns by column i
     (which two elements form pair i is the consuming kernel's layout).  Angles are formed in float64 and rounded once."""

@@ -398,3 +398,131 @@ class ChunkedSinkAttention:
 
     def forward(self, h: torch.Tensor, positions, ctx, spans: mixops.StepSpans, inst: int = 0) -> torch.Tensor:
         return F.linear(self.mix(h, positions, ctx, spans, inst), self.w_o)
+
+
+class HalfRotaryAttention:
+    """Causal grouped-query attention over all earlier tokens with a half-split partial rotation; what else it has is named by the subclass:
+
+        q = W_q h (+ b_q),  k = W_k h (+ b_k),  v = W_v h (+ b_v)                                               (``bias``)
+        q[h] <- rotate(q[h], p),  k[g] <- rotate(k[g], p)      (the first rot.dims elements turn, pair (i, i + dims / 2), frequencies by rot.scaling)
+        q[h] <- q[h] / rms(q[h]),  k[g] <- k[g] / rms(k[g])                                                     (``unit_norm``, after the rotation)
+        s[h, i, j] = (q_i[h] . k_j[h // (H / G)]) * scale;  s <- softcap * tanh(s / softcap) when the configuration has one
+        p_j = exp(s_j) / (exp(sink[h]) + sum_j exp(s_j))                                                        (``sink``: learned; else an ordinary softmax)
+        out = W_o (sigmoid(W_g h) * concat_h sum_j p_ij v_j)                                                    (``gate``, element by element)
+
+    One row ``[k (G * dim) | v (G * vdim)]`` per token, layer instance and page slot, keys after rotation and norm.  Cap, sink, gate and a
+    constant factor are applied inside the attention kernel.  Input projection ``[W_q ; W_k ; W_v ; W_g]``, bias and output projection may be
+    views into the merged weights of a block that runs this mixer beside another one (``ParallelMixer``).
+    """
+    kind = "attention"
+    bias = unit_norm = gate = sink = False
+
+    def __init__(self, width: int, m: dict, eps: float, dtype, device, max_position: int, w_in=None, b_in=None, w_o=None):
+        from .rotary_embedding import build_scaled_cos_sin
+        self.width, self.eps, self.dtype, self.device = width, eps, dtype, device
+        self.heads, self.kv_heads = int(m["heads"]), int(m["kv_heads"])
+        self.dim, self.vdim = int(m["dim"]), int(m["vdim"])
+        self.scale, self.softcap = float(m["scale"]), float(m.get("softcap") or 0.0)
+        if self.heads % self.kv_heads:
+            raise ValueError("heads must be a multiple of kv_heads")
+        if self.vdim > 512:
+            raise ValueError(f"vdim {self.vdim}: the attention kernels hold at most 512 output columns per query row")
+        H, G, d, vd = self.heads, self.kv_heads, self.dim, self.vdim
+        self.q_cols, self.k_cols, self.v_cols = H * d, G * d, G * vd
+        self.g_off = self.q_cols + self.k_cols + self.v_cols
+        self.in_cols, self.out_cols = self.projection_cols(m)
+        rot = m.get("rot")
+        self.cos_sin, self.rot_key = None, None
+        if rot and int(rot.get("dims") or 0) > 0:
+            dims, base = int(rot["dims"]), float(rot["base"])
+            if dims > d or dims % 2:
+                raise ValueError("rot.dims must be even and at most dim")
+            self.rot_key = ("halves", dims, base, repr(sorted((rot.get("scaling") or {}).items())), max_position)
+            self.cos_sin = build_scaled_cos_sin(dims, max_position, base, rot.get("scaling"), device)
+        if w_in is None:
+            w_in = torch.zeros(-(-self.in_cols // 8) * 8, width, dtype=dtype, device=device)          # whole 16-byte rows of the result
+            b_in = torch.zeros(w_in.shape[0], dtype=dtype, device=device) if self.bias else None
+        self.w_in, self.b_in = w_in, b_in
+        self.w_o = w_o if w_o is not None else torch.empty(width, self.out_cols, dtype=dtype, device=device)
+        assert self.w_in.shape[0] >= self.in_cols and self.w_o.shape == (width, self.out_cols) and (b_in is not None or not self.bias)
+        self.sinks = torch.zeros(H, dtype=torch.float32, device=device) if self.sink else None
+        self.cache: list = []                                              # per instance [num_blocks * block_size, G * (dim + vdim)]
+        self.block_size = 0
+
+    @classmethod
+    def projection_cols(cls, m: dict) -> tuple[int, int]:
+        """(rows of the wide input projection, columns of the output projection) for a mixer configuration."""
+        H, G, d, vd = int(m["heads"]), int(m["kv_heads"]), int(m["dim"]), int(m["vdim"])
+        return H * d + G * d + G * vd + (H * vd if cls.gate else 0), H * vd
+
+    def _spans(self) -> dict:
+        q, k, v = self.q_cols, self.k_cols, self.v_cols
+        spans = {"q": (0, q), "k": (q, q + k), "v": (q + k, q + k + v)}
+        if self.gate:
+            spans["g"] = (self.g_off, self.in_cols)
+        return spans
+
+    def load(self, leaf: str, w: torch.Tensor) -> bool:
+        spans = self._spans()
+        if leaf in spans:
+            self.w_in[spans[leaf][0]:spans[leaf][1]].copy_(w)
+        elif self.bias and leaf in ("q.b", "k.b", "v.b"):
+            self.b_in[spans[leaf[0]][0]:spans[leaf[0]][1]].copy_(w)
+        elif self.sink and leaf == "sink":
+            self.sinks.copy_(w.float())
+        elif leaf == "o":
+            self.w_o.copy_(w)
+        else:
+            return False
+        return True
+
+    def weight_shapes(self, width: int) -> dict:
+        out = {leaf: (b - a, width) for leaf, (a, b) in self._spans().items()}
+        if self.bias:
+            out.update({"q.b": (self.q_cols,), "k.b": (self.k_cols,), "v.b": (self.v_cols,)})
+        if self.sink:
+            out["sink"] = (self.heads,)
+        return dict(out, o=(width, self.out_cols))
+
+    def cache_row_elems(self) -> int:
+        return self.k_cols + self.v_cols
+
+    def state_slot_bytes(self) -> int:
+        return 0
+
+    def bind(self, num_blocks: int, block_size: int, num_slots: int, copies: int = 1) -> None:
+        self.block_size = block_size
+        self.cache = [torch.zeros(num_blocks * block_size, self.cache_row_elems(), dtype=self.dtype, device=self.device) for _ in range(copies)]
+
+    def unbind(self) -> None:
+        self.cache = []
+
+    def rotations(self):
+        """Layers that can share rotation tables (``rot_key``)."""
+        return [self]
+
+    def mix(self, proj: torch.Tensor, h: torch.Tensor, positions, ctx, spans: mixops.StepSpans, inst: int, out: torch.Tensor | None = None,
+            out_scale: float = 1.0) -> torch.Tensor:
+        """proj [n, >= in_cols] = h W_in^T + b_in (a row-strided view) -> the output projection's operand [n, heads * vdim]."""
+        q, k = self.q_cols, self.k_cols
+        cache = self.cache[inst]
+        mixops.headnorm_rope_store(proj, 0, q, q + k, self.heads, self.kv_heads, self.dim, self.vdim, None, None, False, self.cos_sin, positions,
+                                   ctx.slot_mapping, cache, self.eps, layout=mixops.ROT_HALVES, unit_after=self.unit_norm)
+        return mixops.window_attention(proj, cache, ctx.block_tables, self.block_size, spans, self.heads, self.kv_heads, self.dim, self.vdim,
+                                       self.scale, None, 0, sinks=self.sinks, softcap=self.softcap,
+                                       gate=proj[:, self.g_off:self.in_cols] if self.gate else None, out=out, out_scale=out_scale)
+
+    def forward(self, h: torch.Tensor, positions, ctx, spans: mixops.StepSpans, inst: int = 0) -> torch.Tensor:
+        return F.linear(self.mix(F.linear(h, self.w_in, self.b_in), h, positions, ctx, spans, inst), self.w_o)
+
+
+class CappedGatedAttention(HalfRotaryAttention):
+    """Biased projections, unit-RMS queries and keys after the rotation, soft-capped scores, an output gate per element."""
+    kind = "capped_attention"
+    bias = unit_norm = gate = True
+
+
+class LearnedSinkAttention(HalfRotaryAttention):
+    """A learned number per head joins the softmax's denominator."""
+    kind = "sink_attention"
+    sink = True

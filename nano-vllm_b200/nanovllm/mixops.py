@@ -191,6 +191,23 @@ def add_layernorm2(x: torch.Tensor, eps: float, y: torch.Tensor | None = None, m
     return tuple(outs)
 
 
+def add_rmsnorm(x: torch.Tensor, weight: torch.Tensor | None, eps: float, y: torch.Tensor | None = None, rows_idx: torch.Tensor | None = None,
+                out_scale: float = 1.0):
+    """x (fp32 [rows, cols], in place) += y; returns x / rms(x) * weight * out_scale in the weight's dtype (None without a weight).
+    ``rows_idx`` (int32): the norm of these rows only, nothing is added."""
+    assert x.dtype == torch.float32 and x.is_contiguous() and x.dim() == 2
+    rows, cols = x.shape
+    is32 = _is32(weight if weight is not None else y)
+    _same(is32, weight, y)
+    assert y is None or (y.is_contiguous() and y.shape == x.shape and rows_idx is None)
+    if rows_idx is not None:
+        assert rows_idx.dtype == torch.int32
+        rows = rows_idx.numel()
+    out = torch.empty(rows, cols, dtype=weight.dtype, device=x.device) if weight is not None else None
+    _call("b200m_add_rmsnorm", x.data_ptr(), _p(y), _p(weight), _p(out), _p(rows_idx), rows, cols, eps, float(out_scale), is32, _stream())
+    return out
+
+
 def rmsnorm(x: torch.Tensor, weight: torch.Tensor, eps: float, cols: int | None = None, out: torch.Tensor | None = None) -> torch.Tensor:
     """RMS norm over the first ``cols`` elements of each row of a 2-D, unit-inner-stride x."""
     assert x.dim() == 2 and x.stride(1) == 1
@@ -317,12 +334,14 @@ def window_attention(q: torch.Tensor, cache: torch.Tensor, block_tables: torch.T
                      heads: int, kv_heads: int, dim: int, vdim: int, scale: float, slopes: torch.Tensor | None = None,
                      window: int = 0, fma: bool = False, splits: int | None = None, keep_first: int = 0, all_values: bool = False,
                      out_f32: bool = False, chunk: int = 0, sinks: torch.Tensor | None = None, gate: torch.Tensor | None = None,
-                     out: torch.Tensor | None = None) -> torch.Tensor:
+                     out: torch.Tensor | None = None, softcap: float = 0.0, out_scale: float = 1.0) -> torch.Tensor:
     """q [n, >= heads * dim] (row-strided view), cache [slots, kv_heads * (dim + vdim)] -> [n, heads * vdim].
     ``keep_first``: the first tokens of a sequence that stay visible beyond the window.  ``all_values``: every head's weights
     meet the values of every value head, -> [n, heads, kv_heads, vdim] (``head_mix_gate`` mixes them).  ``out_f32``: fp32 result.
     ``chunk``: only keys of the query's own chunk of positions (instead of a window).  ``sinks`` (fp32 [heads]): scores of a valueless
-    extra term of each head's softmax.  ``gate`` ([n, heads], a row-strided view): head h times sigmoid(gate[:, h]).  ``out`` may be a row-strided view."""
+    extra term of each head's softmax.  ``softcap`` > 0: scores become softcap * tanh(score / softcap).  ``gate`` (a row-strided view):
+    [n, heads], head h times sigmoid(gate[:, h]), or [n, heads * vdim], element by element.  The result carries ``out_scale``; ``out`` may
+    be a row-strided view."""
     n = q.shape[0]
     assert q.dim() == 2 and q.stride(1) == 1 and cache.is_contiguous() and cache.shape[-1] == kv_heads * (dim + vdim)
     assert block_tables.dtype == torch.int32 and block_tables.stride(1) == 1
@@ -330,7 +349,8 @@ def window_attention(q: torch.Tensor, cache: torch.Tensor, block_tables: torch.T
     is32 = _is32(q)
     _same(is32, cache)
     assert sinks is None or (sinks.dtype == torch.float32 and sinks.is_contiguous() and sinks.numel() == heads)
-    assert gate is None or (gate.dtype == q.dtype and gate.shape == (n, heads) and gate.stride(1) == 1 and not all_values)
+    assert gate is None or (gate.dtype == q.dtype and gate.shape in ((n, heads), (n, heads * vdim)) and gate.stride(1) == 1 and not all_values)
+    gate_elems = gate is not None and gate.shape[1] == heads * vdim and vdim > 1
     vsets = kv_heads if all_values else 1
     if out is None:
         out = torch.empty(n, heads * vsets * vdim, dtype=torch.float32 if out_f32 else q.dtype, device=q.device)
@@ -345,7 +365,8 @@ def window_attention(q: torch.Tensor, cache: torch.Tensor, block_tables: torch.T
         ops.LAUNCHES[0] += 1
     _call("b200m_window_attention", q.data_ptr(), q.stride(0), cache.data_ptr(), cache.shape[-1], kv_heads * dim,
           block_tables.data_ptr(), block_tables.stride(0), block_size, _p(spans.cu_q), _p(spans.cu_k), _p(spans.ctx_lens),
-          _p(slopes), int(window), int(keep_first), int(chunk), _p(sinks), _p(gate), gate.stride(0) if gate is not None else 0, int(all_values),
+          _p(slopes), int(window), int(keep_first), int(chunk), _p(sinks), float(softcap), _p(gate), gate.stride(0) if gate is not None else 0,
+          int(gate_elems), float(out_scale), int(all_values),
           out.data_ptr(), out.stride(0), n, spans.num_seqs, spans.max_q, heads, kv_heads,
           dim, vdim, scale, is32, int(fma) | (2 if out_f32 else 0), nsplit, _p(part), _stream())
     return out.view(n, heads, vsets, vdim) if all_values else out
@@ -364,11 +385,12 @@ def window_attention_splits(spans: StepSpans, max_keys: int, window: int, kv_hea
 def headnorm_rope_store(x: torch.Tensor, q_off: int, k_off: int, v_off: int, heads: int, kv_heads: int, dim: int, vdim: int,
                         q_norm: torch.Tensor | None, k_norm: torch.Tensor | None, v_unit_norm: bool, cos_sin: torch.Tensor | None,
                         positions: torch.Tensor | None, slots: torch.Tensor | None, cache: torch.Tensor | None, eps: float,
-                        v_cos_sin: torch.Tensor | None = None, layout: int = ROT_PAIRS) -> None:
+                        v_cos_sin: torch.Tensor | None = None, layout: int = ROT_PAIRS, unit_after: bool = False) -> None:
     """x [n, cols] (q heads at q_off, key heads at k_off, value heads at v_off): per-head RMS norm of q and k with one weight of
     ``dim`` elements shared by the heads, pair rotation by cos_sin [positions, rope_dims] (fp32), q in place; normed, rotated keys
     and (unit-RMS) values into cache rows [k (kv_heads * dim) | v (kv_heads * vdim)] at ``slots``.  ``v_cos_sin`` (fp32
-    [positions, v_dims]): the value pairs are turned by the token's position before the store.  ``layout``: which query / key elements pair."""
+    [positions, v_dims]): the value pairs are turned by the token's position before the store.  ``layout``: which query / key elements pair.
+    ``unit_after`` (without norm weights): q and k are divided by their root mean square per head after the rotation."""
     assert x.dim() == 2 and x.stride(1) == 1
     is32 = _is32(x)
     _same(is32, q_norm, k_norm, cache)
@@ -383,7 +405,7 @@ def headnorm_rope_store(x: torch.Tensor, q_off: int, k_off: int, v_off: int, hea
     if cache is not None:
         assert cache.is_contiguous() and cache.shape[-1] == kv_heads * (dim + vdim) and slots.dtype == torch.int32 and slots.numel() == x.shape[0]
     _call("b200m_headnorm_rope_store", x.data_ptr(), x.stride(0), q_off, k_off, v_off, heads, kv_heads, dim, vdim, _p(q_norm), _p(k_norm),
-          int(v_unit_norm), _p(cos_sin), int(layout), rope_dims, _p(v_cos_sin), v_dims, _p(positions), _p(slots), _p(cache), x.shape[0], eps, is32,
+          int(v_unit_norm), int(unit_after), _p(cos_sin), int(layout), rope_dims, _p(v_cos_sin), v_dims, _p(positions), _p(slots), _p(cache), x.shape[0], eps, is32,
           _stream())
 
 
@@ -486,18 +508,77 @@ def channel_state(x: torch.Tensor, q_off: int, k_off: int, v_off: int, write: to
     return out
 
 
+def linear_state(x: torch.Tensor, q_off: int, k_off: int, v_off: int, state: torch.Tensor, state_slots: torch.Tensor, spans: StepSpans, heads: int,
+                 kv_heads: int, dim: int, vdim: int, q_scale: float = 1.0, step: torch.Tensor | None = None, rate: torch.Tensor | None = None,
+                 bias: torch.Tensor | None = None, log_decay: torch.Tensor | None = None, write: torch.Tensor | None = None,
+                 ones: bool = False) -> torch.Tensor:
+    """Matrix state with one decay and one write weight per token and head, S <- g S + w k v^T, out = q_scale * S^T q.  x [n, cols]: q, k ([kv_heads,
+    dim] at q_off / k_off), v ([heads, vdim] at v_off).  ``step`` [n, heads] (x's dtype, a row-strided view) with fp32 ``rate`` and ``bias``: w =
+    softplus(step + bias), g = exp(rate * w); else fp32 ``log_decay`` and ``write`` [n, heads].  ``ones``: an extra state column whose value is
+    always 1.  state fp32 [slots, heads, vdim + ones, dim] -> fp32 [n, heads, vdim + ones]."""
+    n, cols = x.shape[0], vdim + int(ones)
+    is32 = _is32(x)
+    assert x.dim() == 2 and x.stride(1) == 1 and state_slots.dtype == torch.int32
+    assert state.dtype == torch.float32 and state.is_contiguous() and state.shape[1:] == (heads, cols, dim)
+    if step is not None:
+        _same(is32, step)
+        assert step.shape == (n, heads) and step.stride(1) == 1 and rate.dtype == bias.dtype == torch.float32 and rate.numel() == bias.numel() == heads
+        gate_stride = step.stride(0)
+    else:
+        assert log_decay.dtype == write.dtype == torch.float32 and log_decay.shape == write.shape == (n, heads)
+        assert log_decay.is_contiguous() and write.is_contiguous()
+        gate_stride = heads
+    out = torch.empty(n, heads, cols, dtype=torch.float32, device=x.device)
+    _call("b200m_linear_state", x.data_ptr(), x.stride(0), q_off, k_off, v_off, _p(step), _p(log_decay), _p(write), gate_stride, _p(rate), _p(bias),
+          state.data_ptr(), state_slots.data_ptr(), _p(spans.cu_q), _p(spans.cu_k), _p(spans.ctx_lens), out.data_ptr(), spans.num_seqs, spans.max_q,
+          heads, kv_heads, dim, vdim, int(ones), float(q_scale), is32, _stream())
+    return out
+
+
+def mlstm_gates(pre: torch.Tensor, bias: torch.Tensor, cap: float, m_state: torch.Tensor, state_slots: torch.Tensor, spans: StepSpans, heads: int):
+    """pre fp32 [n, 2 heads] = [i | f] pre-activations, bias fp32 [2 heads], m_state fp32 [slots, heads] (the running maximum) -> fp32 [n, heads]
+    (log decay, write weight, exp(-m))."""
+    n = pre.shape[0]
+    assert pre.dtype == torch.float32 and pre.shape == (n, 2 * heads) and pre.stride(1) == 1 and bias.dtype == torch.float32 and bias.numel() == 2 * heads
+    assert m_state.dtype == torch.float32 and m_state.is_contiguous() and m_state.shape[1] == heads and state_slots.dtype == torch.int32
+    out = torch.empty(3, n, heads, dtype=torch.float32, device=pre.device)
+    _call("b200m_mlstm_gates", pre.data_ptr(), pre.stride(0), bias.data_ptr(), float(cap), m_state.data_ptr(), state_slots.data_ptr(), _p(spans.cu_q),
+          _p(spans.cu_k), _p(spans.ctx_lens), out[0].data_ptr(), out[1].data_ptr(), out[2].data_ptr(), spans.num_seqs, heads, _stream())
+    return out[0], out[1], out[2]
+
+
+def skip_gate_groupnorm(y: torch.Tensor, x: torch.Tensor, D: torch.Tensor, z: torch.Tensor, weight: torch.Tensor, groups: int, eps: float,
+                        out: torch.Tensor | None = None) -> torch.Tensor:
+    """y fp32 [n, H, vdim], x and z [n, H * vdim] (row-strided views), D fp32 [H] -> [n, H * vdim]: (y + D x) * silu(z), then each of ``groups`` equal
+    parts of the row divided by its own root mean square, times ``weight`` [H * vdim]."""
+    n, H, vdim = y.shape
+    dtype = weight.dtype
+    assert y.dtype == torch.float32 and y.is_contiguous() and D.dtype == torch.float32 and D.numel() == H and weight.numel() == H * vdim
+    assert x.shape == z.shape == (n, H * vdim) and x.stride(1) == z.stride(1) == 1 and x.dtype == z.dtype == dtype
+    if out is None:
+        out = torch.empty(n, H * vdim, dtype=dtype, device=y.device)
+    assert out.dtype == dtype and out.shape == (n, H * vdim) and out.stride(1) == 1
+    _call("b200m_skip_gate_groupnorm", y.data_ptr(), x.data_ptr(), x.stride(0), D.data_ptr(), z.data_ptr(), z.stride(0), weight.data_ptr(), out.data_ptr(),
+          out.stride(0), n, H, vdim, groups, eps, int(dtype == torch.float32), _stream())
+    return out
+
+
 def head_rmsnorm_gate(x: torch.Tensor, weight: torch.Tensor | None, gate: torch.Tensor | None, eps: float, dtype, silu: bool = True,
-                      out: torch.Tensor | None = None, out_scale: float = 1.0) -> torch.Tensor:
-    """x fp32 [n, H, vdim] -> [n, H * vdim] = out_scale * x / rms(x) * weight * act(gate), per head; act = silu or sigmoid;
-    ``out`` may be a row-strided view."""
+                      out: torch.Tensor | None = None, out_scale: float = 1.0, floor: torch.Tensor | None = None) -> torch.Tensor:
+    """x fp32 [n, H, vdim] -> [n, H * vdim] = out_scale * x / rms(x) * weight * act(gate), per head; act = silu or sigmoid; weight [vdim] shared by the
+    heads or [H * vdim]; ``out`` may be a row-strided view.  ``floor`` (fp32 [n, H]): x is [n, H, vdim + 1] and is first divided by
+    max(|x[..., vdim]|, floor) + 1e-6."""
     n, H, vdim = x.shape
+    vdim -= floor is not None
     assert x.dtype == torch.float32 and x.is_contiguous()
+    assert floor is None or (floor.dtype == torch.float32 and floor.is_contiguous() and floor.shape == (n, H))
     assert gate is None or (gate.stride(1) == 1 and gate.shape == (n, H * vdim) and gate.dtype == dtype)
-    assert weight is None or (weight.dtype == dtype and weight.numel() == vdim)
+    assert weight is None or (weight.dtype == dtype and weight.numel() in (vdim, H * vdim))
+    w_heads = weight is not None and weight.numel() == H * vdim and H > 1
     if out is None:
         out = torch.empty(n, H * vdim, dtype=dtype, device=x.device)
     assert out.dtype == dtype and out.shape == (n, H * vdim) and out.stride(1) == 1
-    _call("b200m_head_rmsnorm_gate", x.data_ptr(), _p(weight), _p(gate), gate.stride(0) if gate is not None else 0, int(silu), out.data_ptr(),
+    _call("b200m_head_rmsnorm_gate", x.data_ptr(), _p(floor), _p(weight), int(w_heads), _p(gate), gate.stride(0) if gate is not None else 0, int(silu), out.data_ptr(),
           out.stride(0), out_scale, n, H, vdim, eps, int(dtype == torch.float32), _stream())
     return out
 

@@ -63,10 +63,20 @@ def _zuvepel_config(raw: dict):
     return ZuvepelConfig(raw)
 
 
+def _pekunex():
+    from .pekunex import PekunexForCausalLM
+    return PekunexForCausalLM
+
+
+def _pekunex_config(raw: dict):
+    from .pekunex import PekunexConfig
+    return PekunexConfig(raw)
+
+
 MODELS = {"Qwen3ForCausalLM": _qwen3, "Qwen2ForCausalLM": _qwen3, "Tafopel": _tafopel, "Tipetar": _tipetar, "Musavik": _musavik, "Fegolorn": _fegolorn,
-          "Zuvepel": _zuvepel}
+          "Zuvepel": _zuvepel, "Pekunex": _pekunex}
 CONFIG_READERS = {"Tafopel": _tafopel_config, "Tipetar": _tipetar_config, "Musavik": _musavik_config, "Fegolorn": _fegolorn_config,
-                  "Zuvepel": _zuvepel_config}
+                  "Zuvepel": _zuvepel_config, "Pekunex": _pekunex_config}
 
 
 def architecture_of(hf_config) -> str:
