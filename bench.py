@@ -560,6 +560,11 @@ def main():
                          "a sink, delta rule with channel decays, gated linear attention) beside Musavik, Tafopel, Tipetar and Qwen3 at equal size, "
                          "with a per-kernel roofline table (profiles/channel_bench.py); one GPU")
     ap.add_argument("--channel-sizes", default="w1024,w2048")
+    ap.add_argument("--state-space", action="store_true",
+                    help="instead of the headline workload: prefill / decode throughput of the Pekunex decoder (soft-capped gated attention, sink "
+                         "attention beside a matrix memory, state-space recurrence) beside Zuvepel, Tafopel, Tipetar and Qwen3 at equal size, with a "
+                         "per-kernel roofline table (profiles/state_space_bench.py); one GPU")
+    ap.add_argument("--state-space-sizes", default="w1024,w2048")
     args = ap.parse_args()
     if args.windowed:
         sys.path.insert(0, os.path.join(os.path.dirname(os.path.abspath(__file__)), "profiles"))
@@ -575,6 +580,11 @@ def main():
         sys.path.insert(0, os.path.join(os.path.dirname(os.path.abspath(__file__)), "profiles"))
         import channel_bench
         channel_bench.main(["--sizes", args.channel_sizes])
+        return
+    if args.state_space:
+        sys.path.insert(0, os.path.join(os.path.dirname(os.path.abspath(__file__)), "profiles"))
+        import state_space_bench
+        state_space_bench.main(["--sizes", args.state_space_sizes])
         return
     if args.recurrent:
         sys.path.insert(0, os.path.join(os.path.dirname(os.path.abspath(__file__)), "profiles"))

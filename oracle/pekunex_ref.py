@@ -132,19 +132,26 @@ def sink_attention(W: dict, p: str, m: dict, h: torch.Tensor) -> torch.Tensor:
     return torch.cat(o, -1) @ w("o").T
 
 
-def memory_cell(q, k, v, i, f):
-    """One head's matrix memory, token by token.  q, k [n, d], v [n, vd], log input gate i [n], log forget gate f [n] -> o [n, vd]."""
+def memory_parts(q, k, v, i, f):
+    """One head's matrix memory, token by token.  q, k [n, d], v [n, vd], log input gate i [n], log forget gate f [n] -> (read-out before its
+    division [n, vd], normaliser n . q [n], running maximum [n])."""
     n, d, vd = q.shape[0], q.shape[1], v.shape[1]
     S, z, m = torch.zeros(d, vd, dtype=F64), torch.zeros(d, dtype=F64), 0.0
-    out = torch.empty(n, vd, dtype=F64)
+    num, nq, top = torch.empty(n, vd, dtype=F64), torch.empty(n, dtype=F64), torch.empty(n, dtype=F64)
     for t in range(n):
         new = max(float(f[t]) + m, float(i[t]))
         keep, write = math.exp(float(f[t]) + m - new), math.exp(float(i[t]) - new)
         S = keep * S + write * torch.outer(k[t], v[t])
         z = keep * z + write * k[t]
         m = new
-        out[t] = (S.T @ q[t]) / (max(abs(float(z @ q[t])), math.exp(-m)) + 1e-6)
-    return out
+        num[t], nq[t], top[t] = S.T @ q[t], z @ q[t], m
+    return num, nq, top
+
+
+def memory_cell(q, k, v, i, f):
+    """-> the read-out [n, vd]: divided by the larger of |n . q| and exp(-m), plus 1e-6."""
+    num, nq, top = memory_parts(q, k, v, i, f)
+    return num / (torch.maximum(nq.abs(), torch.exp(-top)) + 1e-6)[:, None]
 
 
 def matrix_memory(W: dict, p: str, m: dict, h: torch.Tensor, eps: float) -> torch.Tensor:
