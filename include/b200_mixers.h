@@ -245,12 +245,13 @@ int b200m_channel_state(const void* x, int64_t stride, int q_off, int k_off, int
  * stride gate_stride): w = softplus(step_in + bias[h]), g = exp(rate[h] * w), a state-space step with q = C, k = B, v = x.  step_in NULL:
  * log_decay = log g and write = w, fp32 [n, num_heads] with row stride gate_stride (b200m_mlstm_gates makes them).  ones = 1: the
  * state has one more column whose value is always 1; state fp32 [slots, num_heads, vdim + ones, dim], out fp32 [n, num_heads, vdim + ones].
- * dim <= 256. */
+ * dim <= 256.  bf16 prompt portions with dim up to 128 and 16-byte aligned parts (dim, vdim, offsets and stride multiples of eight) run on the
+ * tensor cores unless flags & 1; everything else on the fp32 FMA pipe. */
 int b200m_linear_state(const void* x, int64_t stride, int q_off, int k_off, int v_off, const void* step_in, const float* log_decay,
                        const float* write, int64_t gate_stride, const float* rate, const float* bias, float* state,
                        const int32_t* state_slots, const int32_t* cu_q, const int32_t* cu_k, const int32_t* ctx_lens, float* out,
                        int num_seqs, int max_q, int num_heads, int num_kv_heads, int dim, int vdim, int ones, float q_scale, int is32,
-                       void* stream);
+                       int flags, void* stream);
 
 /* Exponential gates of a matrix memory with a running maximum.  in fp32 [n, >= 2 num_heads] = [i | f] pre-activations, bias fp32 [2 num_heads]:
  *     i = cap * tanh((in_i + bias_i) / cap);  f = logsigmoid(cap * tanh((in_f + bias_f) / cap));  m_t = max(f_t + m_(t-1), i_t)

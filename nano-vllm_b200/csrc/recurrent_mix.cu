@@ -26,11 +26,10 @@
 //                               value is always 1, the running sum of weighted keys that normalises the read-out
 //   Channel decays are g = exp(rate_h softplus(sign (a + bias))): sign 1 is the softplus form; sigmoid(z)^(1 / tau) is rate
 //   -1 / tau with sign -1.  Columns of S are independent: a lane group owns one or two of them and walks the tokens.
-#include "mix_common.cuh"
+#include "state_common.cuh"
 
 namespace {
 
-__device__ __forceinline__ float softplus_(float x) { return x > 20.f ? x : log1pf(expf(x)); }
 __device__ __forceinline__ float gelu_tanh1_(float z) { return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z))); }
 
 // gates: fp32 [blocks, rows, 2 * cb]: for block b and token row t the cb pre-activations of r, then those of i.
@@ -121,6 +120,7 @@ __global__ void __launch_bounds__(128) diag_carry_kernel(float* __restrict__ ws,
 // lands, MS_THREADS / TB threads per token form its unit-norm factors and k . q once for the CTA.  The delta rule reads out
 // before it writes, o = (g S)^T q + u (k . q), so that both column sums of a token are reduced together.
 constexpr int MS_THREADS = 128;
+constexpr int MS_CHUNK_MIN = 16;       // longest portion up to which a step of scalar linear attention stays off the tensor cores
 
 struct DecayIn {
     const float* in;          // pre-activations, CH: [n, >= H * dim], else one per head.  (The token-at-a-time kernel reads CH decays ready-made.)
@@ -130,24 +130,6 @@ struct DecayIn {
     float sign;               // g = exp(rate_h * softplus(sign * (in + bias)))
 };
 __device__ __forceinline__ float decay_of(float a, float rate, float bias, float sign) { return expf(rate * softplus_(sign * (a + bias))); }
-
-// What scalar linear attention (neither CH nor DELTA) does with a token: raw fp32 (or T) inputs -> (log decay, write weight).
-template <typename T>
-struct ScalarGate {
-    const T* raw;             // step-size pre-activations (n, >= H), or NULL: `log_decay` and `write` are given
-    const float *log_decay, *write;
-    int64_t stride;           // of whichever is read
-    const float *rate, *bias;
-    __device__ __forceinline__ float2 fetch(int64_t row, int h) const {      // loads only
-        if (raw) return make_float2(ldf(raw + row * stride + h), 0.f);
-        return make_float2(log_decay[row * stride + h], write[row * stride + h]);
-    }
-    __device__ __forceinline__ float2 gates(float2 f, float rt, float b) const {
-        if (!raw) return f;
-        const float dt = softplus_(f.x + b);
-        return make_float2(rt * dt, dt);
-    }
-};
 
 template <typename T, int DPL, int LANES, int COLS, bool CH, bool DELTA>
 __global__ void __launch_bounds__(MS_THREADS) matrix_state_kernel(
@@ -1177,11 +1159,18 @@ extern "C" int b200m_linear_state(const void* x, int64_t stride, int q_off, int 
                                   const float* write, int64_t gate_stride, const float* rate, const float* bias, float* state,
                                   const int32_t* state_slots, const int32_t* cu_q, const int32_t* cu_k, const int32_t* ctx_lens, float* out,
                                   int num_seqs, int max_q, int num_heads, int num_kv_heads, int dim, int vdim, int ones, float q_scale,
-                                  int is32, void* stream) {
+                                  int is32, int flags, void* stream) {
     if (!x || !state || !state_slots || !out || (step_in ? (!rate || !bias) : (!log_decay || !write))) return B200_EINVAL;
     if ((cu_q == nullptr) != (cu_k == nullptr) || (cu_q == nullptr && ctx_lens == nullptr)) return B200_EINVAL;
     if (num_heads <= 0 || num_kv_heads <= 0 || num_heads % num_kv_heads || dim <= 0 || vdim <= 0 || ones < 0 || ones > 1) return B200_EINVAL;
     if (num_seqs <= 0) return B200_OK;
+    if (!is32 && max_q > MS_CHUNK_MIN && !(flags & 1)) {                    // prompt portions on the tensor cores
+        using bf = __nv_bfloat16;
+        const ScalarGate<bf> sg{static_cast<const bf*>(step_in), log_decay, write, gate_stride, step_in ? rate : nullptr, bias};
+        const int rc = chunk_state_launch(static_cast<const bf*>(x), stride, q_off, k_off, v_off, sg, state, state_slots, cu_q, cu_k, out, num_seqs,
+                                          num_heads, num_kv_heads, dim, vdim, ones, q_scale, static_cast<cudaStream_t>(stream));
+        if (rc != B200_EUNSUPPORTED) return rc;
+    }
     B200M_DISPATCH(is32, const ScalarGate<T> sg = (ScalarGate<T>{static_cast<const T*>(step_in), log_decay, write, gate_stride, step_in ? rate : nullptr, bias});
                    return (launch_matrix_state<T, false, false>(x, stride, q_off, k_off, v_off, nullptr, nullptr, 0, DecayIn{}, state, state_slots,
                                                                 cu_q, cu_k, ctx_lens, out, 0, num_seqs, max_q, num_heads, num_kv_heads, dim, vdim,

@@ -511,11 +511,12 @@ def channel_state(x: torch.Tensor, q_off: int, k_off: int, v_off: int, write: to
 def linear_state(x: torch.Tensor, q_off: int, k_off: int, v_off: int, state: torch.Tensor, state_slots: torch.Tensor, spans: StepSpans, heads: int,
                  kv_heads: int, dim: int, vdim: int, q_scale: float = 1.0, step: torch.Tensor | None = None, rate: torch.Tensor | None = None,
                  bias: torch.Tensor | None = None, log_decay: torch.Tensor | None = None, write: torch.Tensor | None = None,
-                 ones: bool = False) -> torch.Tensor:
+                 ones: bool = False, fma: bool = False) -> torch.Tensor:
     """Matrix state with one decay and one write weight per token and head, S <- g S + w k v^T, out = q_scale * S^T q.  x [n, cols]: q, k ([kv_heads,
     dim] at q_off / k_off), v ([heads, vdim] at v_off).  ``step`` [n, heads] (x's dtype, a row-strided view) with fp32 ``rate`` and ``bias``: w =
     softplus(step + bias), g = exp(rate * w); else fp32 ``log_decay`` and ``write`` [n, heads].  ``ones``: an extra state column whose value is
-    always 1.  state fp32 [slots, heads, vdim + ones, dim] -> fp32 [n, heads, vdim + ones]."""
+    always 1.  state fp32 [slots, heads, vdim + ones, dim] -> fp32 [n, heads, vdim + ones].  bf16 prompt portions run on the tensor cores unless
+    ``fma``."""
     n, cols = x.shape[0], vdim + int(ones)
     is32 = _is32(x)
     assert x.dim() == 2 and x.stride(1) == 1 and state_slots.dtype == torch.int32
@@ -531,7 +532,7 @@ def linear_state(x: torch.Tensor, q_off: int, k_off: int, v_off: int, state: tor
     out = torch.empty(n, heads, cols, dtype=torch.float32, device=x.device)
     _call("b200m_linear_state", x.data_ptr(), x.stride(0), q_off, k_off, v_off, _p(step), _p(log_decay), _p(write), gate_stride, _p(rate), _p(bias),
           state.data_ptr(), state_slots.data_ptr(), _p(spans.cu_q), _p(spans.cu_k), _p(spans.ctx_lens), out.data_ptr(), spans.num_seqs, spans.max_q,
-          heads, kv_heads, dim, vdim, int(ones), float(q_scale), is32, _stream())
+          heads, kv_heads, dim, vdim, int(ones), float(q_scale), is32, int(fma), _stream())
     return out
 
 

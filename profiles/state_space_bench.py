@@ -104,6 +104,9 @@ def kernel_table(size: str, peaks: dict):
         rate, bias = -torch.rand(sh, device=dev), torch.zeros(sh, device=dev)
         add(f"linear_state, state space {label}", lambda: mixops.linear_state(x, sh * 64 + gr * d, sh * 64, 0, st, slots, spn, sh, gr, d, 64, step=step, rate=rate,
             bias=bias), n * (C * 2 + sh * 2 + sh * 64 * 4) + 2 * st.numel() * 4, n * sh * 64 * d * 5, "fma")
+        if q > 1:
+            add(f"linear_state, state space, fp32-pipe form {label}", lambda: mixops.linear_state(x, sh * 64 + gr * d, sh * 64, 0, st, slots, spn, sh, gr, d, 64,
+                step=step, rate=rate, bias=bias, fma=True), n * (C * 2 + sh * 2 + sh * 64 * 4) + 2 * st.numel() * 4, n * sh * 64 * d * 5, "fma")
         y, z, wn, D = torch.randn(n, sh, 64, device=dev), rn(n, sh * 64), rn(sh * 64), torch.ones(sh, device=dev)
         if q != 1024:
             add(f"skip_gate_groupnorm {label}", lambda: mixops.skip_gate_groupnorm(y, x[:, :sh * 64], D, z, wn, gr, 1e-6), n * sh * 64 * 10, 0)
@@ -114,6 +117,10 @@ def kernel_table(size: str, peaks: dict):
         sm = torch.zeros(S, mh, d + 1, d, device=dev)
         add(f"linear_state, matrix memory {label}", lambda: mixops.linear_state(xg, 0, mh * d, 2 * mh * d, sm, slots, spn, mh, mh, d, d, d ** -0.5, log_decay=ld,
             write=wr, ones=True), n * (3 * mh * d * 2 + mh * (d + 1) * 4 + mh * 8) + 2 * sm.numel() * 4, n * mh * d * (d + 1) * 5, "fma")
+        if q > 1:
+            add(f"linear_state, matrix memory, fp32-pipe form {label}", lambda: mixops.linear_state(xg, 0, mh * d, 2 * mh * d, sm, slots, spn, mh, mh, d, d,
+                d ** -0.5, log_decay=ld, write=wr, ones=True, fma=True), n * (3 * mh * d * 2 + mh * (d + 1) * 4 + mh * 8) + 2 * sm.numel() * 4,
+                n * mh * d * (d + 1) * 5, "fma")
         zz, db, sg = torch.randn(n, mh * d, device=dev), torch.zeros(mh * d, device=dev), torch.zeros(S, mh, d, d, device=dev)
         add(f"channel_state, linear attention (zuvepel form) {label}", lambda: mixops.channel_state(xg, 0, mh * d, 2 * mh * d, None, zz, rate[:mh], db, -1.0, sg,
             slots, spn, mh, mh, d, d, d ** -0.5), n * (3 * mh * d * 2 + mh * d * 8) + 2 * sg.numel() * 4, n * mh * d * d * 5, "fma")

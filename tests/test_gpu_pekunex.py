@@ -288,11 +288,11 @@ def test_state_space_states_on_long_sequences(dtype, dim, vdim, H, G):
     S = torch.stack([sum(torch.exp(rate[h].double() * dt[t + 1:, h].sum()) * dt[t, h] * torch.outer(v[t, h], k[t, h // (H // G)]) for t in range(n)) for h in range(H)])
     slot = torch.zeros(1, dtype=torch.int32, device="cuda")
     xd, sd = x.cuda(), step.cuda()
-    for cuts in CUTS:
+    for cuts, fma in ((c, f) for c in CUTS for f in (False, True)):
         state = torch.full((1, H, vdim, dim), 9.0, device="cuda")            # a new sequence ignores what the slot holds
         out = walk(n, cuts, slot, lambda r, sp: mixops.linear_state(xd[r], H * vdim + G * dim, H * vdim, 0, state, slot, sp, H, G, dim, vdim, step=sd[r],
-                                                                   rate=rate.cuda(), bias=bias.cuda()))
-        assert rel_err(out, want) < 3e-5 and rel_err(state[0], S) < 3e-5, cuts
+                                                                   rate=rate.cuda(), bias=bias.cuda(), fma=fma))
+        assert rel_err(out, want) < 3e-5 and rel_err(state[0], S) < 3e-5, (cuts, fma)
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
@@ -315,16 +315,17 @@ def test_memory_cells_on_long_sequences(dtype, dim, vdim, H, mood):
     assert bool((nq.abs() < floor).any()) and (mood == "shut" or bool((nq.abs() > floor).any()))
     slot = torch.zeros(1, dtype=torch.int32, device="cuda")
     xd, pd = x.cuda(), pre.cuda()
-    for cuts in CUTS:
+    for cuts, fma in ((c, f) for c in CUTS for f in (False, True)):
         state, m = torch.full((1, H, vdim + 1, dim), 9.0, device="cuda"), torch.full((1, H), 5.0, device="cuda")
 
         def call(r, sp):
             ld, w, fl = mixops.mlstm_gates(pd[r], bias.cuda(), cap, m, slot, sp, H)
-            o = mixops.linear_state(xd[r], 0, H * dim, 2 * H * dim, state, slot, sp, H, H, dim, vdim, dim ** -0.5, log_decay=ld, write=w, ones=True)
+            o = mixops.linear_state(xd[r], 0, H * dim, 2 * H * dim, state, slot, sp, H, H, dim, vdim, dim ** -0.5, log_decay=ld, write=w, ones=True,
+                                    fma=fma)
             return torch.cat([o, fl[..., None]], -1)
         o = walk(n, cuts, slot, call)                        # before the division, which amplifies the rounding of a small n . q
-        assert rel_err(o[..., :vdim], want) < 5e-5 and rel_err(o[..., vdim], nq) < 5e-5 and rel_err(o[..., vdim + 1], floor) < 5e-5, cuts
-        assert rel_err(m[0], top[-1]) < 1e-5, cuts
+        assert rel_err(o[..., :vdim], want) < 5e-5 and rel_err(o[..., vdim], nq) < 5e-5 and rel_err(o[..., vdim + 1], floor) < 5e-5, (cuts, fma)
+        assert rel_err(m[0], top[-1]) < 1e-5, (cuts, fma)
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
