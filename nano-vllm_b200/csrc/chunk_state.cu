@@ -11,7 +11,7 @@
 //
 // A CTA (four warps) owns 64 value columns of one (sequence, head).  A warp holds 16 rows of S^T [vdim, dim] as product accumulators in
 // registers for the whole portion; read as the next product's left operand they need no shuffle (S^T Q^T).  Per chunk:
-//     P          : each warp 16 tokens against the keys up to them, split into terms in shared memory
+//     P          : 16 x 16 blocks of the lower triangle, two or three per warp, split into terms in shared memory
 //     O^T = S^T Q^T, scaled by e^(b_t), += V^T P^T over the lower triangle        (V^T by transposing loads)
 //     S^T <- e^(b_L) S^T + (V scaled)^T K
 // The next chunk's q, k, v arrive by asynchronous copies into a second buffer meanwhile; warp 0 forms the next chunk's gates.
@@ -34,9 +34,9 @@ __device__ __forceinline__ uint32_t swz(int row, int piece) {
 template <int D>
 struct ChunkSmem {
     static constexpr int Q = 0, QB = CS_L * D * 2, K = 2 * QB, V = K + 2 * QB, VB = CS_L * CS_VC * 2, P = V + 2 * VB, PB = CS_L * CS_L * 2,
-                         GATE = P + CS_TERMS * PB, GB = 5 * CS_L * 4 + 16, NV = GATE + 2 * GB, RS = NV + D * 4, BYTES = RS + CS_L * 4;
+                         GATE = P + CS_TERMS * PB, GB = 5 * CS_L * 4 + 16, NV = GATE + 2 * GB, RS = NV + D * 4, BYTES = RS + 4 * CS_L * 4;
 };
-// a chunk's gates: b as (high, low), write weight, q_scale e^b, e^(b_L - b) w, then e^(b_L)
+// a chunk's gates: b * log2(e) as (high, low), write weight * q_scale, q_scale e^b, e^(b_L - b) w, then e^(b_L)
 constexpr int CG_BH = 0, CG_BL = CS_L, CG_W = 2 * CS_L, CG_IN = 3 * CS_L, CG_OUT = 4 * CS_L, CG_ALL = 5 * CS_L;
 
 // (a, b) -> packed bf16 pair of their roundings; a and b become what the rounding left
@@ -105,7 +105,8 @@ __global__ void __launch_bounds__(CS_THREADS, 2) chunk_state_kernel(
         float2 g[2];
 #pragma unroll
         for (int j = 0; j < 2; ++j) g[j] = c * CS_L + 2 * lane + j < sp.qlen ? sg.gates(graw[j], rt, gb) : make_float2(0.f, 0.f);
-        double b0 = g[0].x, b1 = b0 + (double)g[1].x, run = b1;
+        constexpr double LOG2E = 1.4426950408889634;
+        double b0 = LOG2E * (double)g[0].x, b1 = b0 + LOG2E * (double)g[1].x, run = b1;
 #pragma unroll
         for (int o = 1; o < 32; o <<= 1) {
             const double up = __shfl_up_sync(0xffffffffu, run, o);
@@ -122,10 +123,10 @@ __global__ void __launch_bounds__(CS_THREADS, 2) chunk_state_kernel(
             gs[CG_BH + t] = hi;
             gs[CG_BL + t] = (float)(bb[j] - (double)hi);
             gs[CG_W + t] = g[j].y * q_scale;
-            gs[CG_IN + t] = expf(hi) * q_scale;
-            gs[CG_OUT + t] = expf((float)(all - bb[j])) * g[j].y;
+            gs[CG_IN + t] = fast_exp2(hi) * q_scale;
+            gs[CG_OUT + t] = fast_exp2((float)(all - bb[j])) * g[j].y;
         }
-        if (lane == 0) gs[CG_ALL] = expf((float)all);
+        if (lane == 0) gs[CG_ALL] = fast_exp2((float)all);
     };
 
     load_chunk(0, 0);
@@ -158,34 +159,44 @@ __global__ void __launch_bounds__(CS_THREADS, 2) chunk_state_kernel(
         }
         if (with_n && tid < D) nvec[tid] = nn;
 
-        // ---- P: tokens warp * 16 .. + 15 against keys 0 .. warp * 16 + 15 ----
+        // ---- P: ten blocks of 16 tokens x 16 keys (keys up to the tokens), shared out over the warps ----
         {
-            const int ar = warp * 16 + (lane & 15), br = (lane & 7) + ((lane >> 4) << 3);
-            uint32_t a[KT][4];
+            const int ar = lane & 15, br = (lane & 7) + ((lane >> 4) << 3);
+            // warp 0: (0,0) (3,0)   1: (1,0) (1,1) (3,1)   2: (2,0) (2,1) (2,2)   3: (3,2) (3,3)      as (token block, key block)
+            const int nblk = warp == 0 || warp == 3 ? 2 : 3;
+            for (int i = 0; i < nblk; ++i) {
+                const int tb = warp == 3 ? 3 : i == (warp == 0 ? 1 : 2) && warp < 2 ? 3 : warp;
+                const int np = warp == 3 ? 2 + i : tb == warp ? i : warp;
+                float sc[2][4], sd[2][4];                   // two sums each, over even and odd steps: more products in flight
 #pragma unroll
-            for (int kk = 0; kk < KT; ++kk) wm_ldsm(qb + swz<D>(ar, kk * 2 + (lane >> 4)), a[kk][0], a[kk][1], a[kk][2], a[kk][3]);
-            const int t0 = warp * 16 + gq;
-            const float bh0 = gs[CG_BH + t0], bl0 = gs[CG_BL + t0], bh1 = gs[CG_BH + t0 + 8], bl1 = gs[CG_BL + t0 + 8];
-            float row0 = 0.f, row1 = 0.f;
-            for (int np = 0; np <= warp; ++np) {            // 16 keys at a time
-                float sc[2][4];
+                for (int j = 0; j < 2; ++j)
 #pragma unroll
-                for (int j = 0; j < 2; ++j) sc[j][0] = sc[j][1] = sc[j][2] = sc[j][3] = 0.f;
+                    for (int e = 0; e < 4; ++e) sc[j][e] = sd[j][e] = 0.f;
 #pragma unroll
-                for (int kk = 0; kk < KT; ++kk) {
-                    uint32_t b[4];
+                for (int kk = 0; kk < KT; kk += 2) {
+                    uint32_t a[4], b[4], a2[4], b2[4];
+                    wm_ldsm(qb + swz<D>(tb * 16 + ar, kk * 2 + (lane >> 4)), a[0], a[1], a[2], a[3]);
                     wm_ldsm(kb + swz<D>(np * 16 + br, kk * 2 + ((lane >> 3) & 1)), b[0], b[1], b[2], b[3]);
-                    wm_mma(sc[0], a[kk][0], a[kk][1], a[kk][2], a[kk][3], b[0], b[1]);
-                    wm_mma(sc[1], a[kk][0], a[kk][1], a[kk][2], a[kk][3], b[2], b[3]);
+                    wm_ldsm(qb + swz<D>(tb * 16 + ar, kk * 2 + 2 + (lane >> 4)), a2[0], a2[1], a2[2], a2[3]);
+                    wm_ldsm(kb + swz<D>(np * 16 + br, kk * 2 + 2 + ((lane >> 3) & 1)), b2[0], b2[1], b2[2], b2[3]);
+                    wm_mma(sc[0], a[0], a[1], a[2], a[3], b[0], b[1]);
+                    wm_mma(sc[1], a[0], a[1], a[2], a[3], b[2], b[3]);
+                    wm_mma(sd[0], a2[0], a2[1], a2[2], a2[3], b2[0], b2[1]);
+                    wm_mma(sd[1], a2[0], a2[1], a2[2], a2[3], b2[2], b2[3]);
                 }
+                const int t0 = tb * 16 + gq;
+                const float bh0 = gs[CG_BH + t0], bl0 = gs[CG_BL + t0], bh1 = gs[CG_BH + t0 + 8], bl1 = gs[CG_BL + t0 + 8];
+                float row0 = 0.f, row1 = 0.f;
 #pragma unroll
                 for (int j = 0; j < 2; ++j) {
                     const int s0 = np * 16 + j * 8 + 2 * t4;
+                    const float2 bh = *reinterpret_cast<const float2*>(gs + CG_BH + s0), bl = *reinterpret_cast<const float2*>(gs + CG_BL + s0),
+                                 w = *reinterpret_cast<const float2*>(gs + CG_W + s0);
 #pragma unroll
                     for (int e = 0; e < 2; ++e) {
-                        const float bh = gs[CG_BH + s0 + e], bl = gs[CG_BL + s0 + e], w = gs[CG_W + s0 + e];
-                        sc[j][e] = s0 + e <= t0 ? sc[j][e] * (expf((bh0 - bh) + (bl0 - bl)) * w) : 0.f;
-                        sc[j][2 + e] = s0 + e <= t0 + 8 ? sc[j][2 + e] * (expf((bh1 - bh) + (bl1 - bl)) * w) : 0.f;
+                        const float h_ = e ? bh.y : bh.x, l_ = e ? bl.y : bl.x, w_ = e ? w.y : w.x;
+                        sc[j][e] = s0 + e <= t0 ? (sc[j][e] + sd[j][e]) * (fast_exp2((bh0 - h_) + (bl0 - l_)) * w_) : 0.f;
+                        sc[j][2 + e] = s0 + e <= t0 + 8 ? (sc[j][2 + e] + sd[j][2 + e]) * (fast_exp2((bh1 - h_) + (bl1 - l_)) * w_) : 0.f;
                     }
                     row0 += sc[j][0] + sc[j][1];
                     row1 += sc[j][2] + sc[j][3];
@@ -196,11 +207,11 @@ __global__ void __launch_bounds__(CS_THREADS, 2) chunk_state_kernel(
                         *reinterpret_cast<uint32_t*>(dst + swz<CS_L>(t0 + 8, np * 2 + j)) = take_term(sc[j][2], sc[j][3]);
                     }
                 }
-            }
-            if (with_n) {
-                row0 += __shfl_xor_sync(0xffffffffu, row0, 1), row1 += __shfl_xor_sync(0xffffffffu, row1, 1);
-                row0 += __shfl_xor_sync(0xffffffffu, row0, 2), row1 += __shfl_xor_sync(0xffffffffu, row1, 2);
-                if (t4 == 0) rsum[t0] = row0, rsum[t0 + 8] = row1;
+                if (with_n) {
+                    row0 += __shfl_xor_sync(0xffffffffu, row0, 1), row1 += __shfl_xor_sync(0xffffffffu, row1, 1);
+                    row0 += __shfl_xor_sync(0xffffffffu, row0, 2), row1 += __shfl_xor_sync(0xffffffffu, row1, 2);
+                    if (t4 == 0) rsum[np * CS_L + t0] = row0, rsum[np * CS_L + t0 + 8] = row1;
+                }
             }
         }
         // ---- O^T = S^T Q^T ----
@@ -313,8 +324,11 @@ __global__ void __launch_bounds__(CS_THREADS, 2) chunk_state_kernel(
                 for (int e = 0; e < 8; ++e) a = fmaf(nvec[piece * 8 + e], f[e], a);
             }
             a += __shfl_xor_sync(0xffffffffu, a, 1);
-            if ((tid & 1) == 0 && c * CS_L + t < sp.qlen)
-                out[((int64_t)(sp.q0 + c * CS_L + t) * H + h) * vcols + vdim] = fmaf(a, gs[CG_IN + t], rsum[t]);
+            if ((tid & 1) == 0 && c * CS_L + t < sp.qlen) {
+                float r = 0.f;                              // sums of P over the key blocks up to the token's own
+                for (int np = 0; np <= t >> 4; ++np) r += rsum[np * CS_L + t];
+                out[((int64_t)(sp.q0 + c * CS_L + t) * H + h) * vcols + vdim] = fmaf(a, gs[CG_IN + t], r);
+            }
             if (tid < D) {
                 float b = 0.f;
 #pragma unroll 8
