@@ -175,7 +175,7 @@ int b200m_head_mix_gate(const void* acc, int acc_f32, const float* mix, const vo
  * values of EVERY value head, out [total_q, num_heads, num_kv_heads, vdim] (for b200m_head_mix_gate).  flags & 2: out is fp32.  A cache row is row_elems long: key head g at g * dim, value head g at
  * v_off + g * vdim.  q [total_q, >= num_heads * dim] with row stride q_stride; out [total_q, >= num_heads * vdim] with row stride out_stride.
  * bf16 with dim and vdim multiples of eight up to 128 runs on the tensor cores unless flags & 1 (32, 64 and 128 as they are, other sizes
- * with zero columns up to 64 or 128); everything else on the fp32 FMA pipe.
+ * with zero columns up to 64, 96 or 128); everything else on the fp32 FMA pipe.
  * splits > 1 (bf16 tensor-core decode steps only): the visible keys of every row are shared out over `splits` CTAs whose
  * partials, fp32 [num_seqs, splits, num_heads (x num_kv_heads with all_values), vdim + 2] in `part`, a second launch merges. */
 int b200m_window_attention(const void* q, int64_t q_stride, const void* cache, int row_elems, int v_off,

@@ -915,7 +915,8 @@ int launch_matrix_state(const void* x, int64_t stride, int q_off, int k_off, int
 // Exponential gates of a matrix memory: from pre-activations (i | f) of H heads each, i <- cap tanh((i + b) / cap), f <- logsigmoid(cap
 // tanh((f + b) / cap)), the running maximum m_t = max(f_t + m_(t-1), i_t) (from 0 for a new sequence), and with it
 //     log_decay = f_t + m_(t-1) - m_t,   write = exp(i_t - m_t),   floor = exp(-m_t)                        (all fp32)
-// One warp per (sequence, head), 32 tokens per step: (f, i) pairs compose as (f1 + f2, max(i1 + f2, i2)), a scan over the lanes.
+// One warp per (sequence, head), 32 x MG_T tokens per step: (f, i) pairs compose as (f1 + f2, max(i1 + f2, i2)), a scan over the lanes.
+constexpr int MG_T = 4;
 __global__ void __launch_bounds__(128) mlstm_gates_kernel(const float* __restrict__ in, int64_t stride, const float* __restrict__ bias, float cap,
                                                           float* __restrict__ mstate, const int32_t* __restrict__ state_slots,
                                                           const int32_t* __restrict__ cu_q, const int32_t* __restrict__ cu_k,
@@ -928,19 +929,28 @@ __global__ void __launch_bounds__(128) mlstm_gates_kernel(const float* __restric
     float* mp = mstate + (int64_t)state_slots[s] * H + h;
     float m = sp.klen - sp.qlen > 0 ? *mp : 0.f;
     const float bi = bias[h], bf = bias[H + h];
-    float ri = 0.f, rf = 0.f;
+    float ri[MG_T], rf[MG_T];
     auto fetch = [&](int i0) {
-        if (i0 + lane < sp.qlen) {
-            const float* row = in + (int64_t)(sp.q0 + i0 + lane) * stride + h;
-            ri = row[0], rf = row[H];
+#pragma unroll
+        for (int j = 0; j < MG_T; ++j) {
+            const int i = i0 + lane * MG_T + j;
+            const float* row = in + (int64_t)(sp.q0 + i) * stride + h;
+            ri[j] = i < sp.qlen ? row[0] : 0.f;
+            rf[j] = i < sp.qlen ? row[H] : 0.f;
         }
     };
     fetch(0);
-    for (int i0 = 0; i0 < sp.qlen; i0 += 32) {
-        const bool ok = i0 + lane < sp.qlen;
-        const float gi = cap * tanhf((ri + bi) / cap), gf = -softplus_(-cap * tanhf((rf + bf) / cap));
-        fetch(i0 + 32);
-        float F = ok ? gf : 0.f, I = ok ? gi : -INFINITY;
+    for (int i0 = 0; i0 < sp.qlen; i0 += 32 * MG_T) {
+        float gi[MG_T], gf[MG_T], F = 0.f, I = -INFINITY;      // (F, I): the lane's tokens composed; nothing past the end
+#pragma unroll
+        for (int j = 0; j < MG_T; ++j) {
+            const bool ok = i0 + lane * MG_T + j < sp.qlen;
+            gi[j] = ok ? cap * tanhf((ri[j] + bi) / cap) : -INFINITY;
+            gf[j] = ok ? -softplus_(-cap * tanhf((rf[j] + bf) / cap)) : 0.f;
+            I = fmaxf(I + gf[j], gi[j]);
+            F += gf[j];
+        }
+        fetch(i0 + 32 * MG_T);
 #pragma unroll
         for (int o = 1; o < 32; o <<= 1) {
             const float pf = __shfl_up_sync(0xffffffffu, F, o), pi = __shfl_up_sync(0xffffffffu, I, o);
@@ -949,16 +959,21 @@ __global__ void __launch_bounds__(128) mlstm_gates_kernel(const float* __restric
                 F += pf;
             }
         }
-        const float mt = fmaxf(F + m, I);
-        float prev = __shfl_up_sync(0xffffffffu, mt, 1);
+        const float end = fmaxf(F + m, I);                     // maximum after the lane's last token
+        float prev = __shfl_up_sync(0xffffffffu, end, 1);
         if (lane == 0) prev = m;
-        if (ok) {
-            const int64_t at = (int64_t)(sp.q0 + i0 + lane) * H + h;
-            log_decay[at] = gf + prev - mt;
-            write[at] = expf(gi - mt);
+        m = __shfl_sync(0xffffffffu, end, 31);                 // lanes past the end carry the last token's maximum on
+#pragma unroll
+        for (int j = 0; j < MG_T; ++j) {
+            const int i = i0 + lane * MG_T + j;
+            if (i >= sp.qlen) break;
+            const float mt = fmaxf(gf[j] + prev, gi[j]);
+            const int64_t at = (int64_t)(sp.q0 + i) * H + h;
+            log_decay[at] = gf[j] + prev - mt;
+            write[at] = expf(gi[j] - mt);
             flr[at] = expf(-mt);
+            prev = mt;
         }
-        m = __shfl_sync(0xffffffffu, mt, 31);                // lanes past the end carry the last token's maximum on
     }
     if (lane == 0) *mp = m;
 }
@@ -966,7 +981,7 @@ __global__ void __launch_bounds__(128) mlstm_gates_kernel(const float* __restric
 // out[t, h, :] = c * o / sqrt(mean(o^2) + eps) * w * act(gate[t, h, :]) for o = x[t, h, :] (fp32), one warp per (token, head).
 // act 0: sigmoid, 1: silu.  w (optional): [vdim], shared by the heads, or (w_heads) [H * vdim].  flr (optional, [n, H]): rows of x have one
 // more element z, and o is first divided by max(|z|, flr) + 1e-6.
-template <typename T>
+template <typename T, int PER>
 __global__ void __launch_bounds__(128) head_rmsnorm_gate_kernel(const float* __restrict__ x, const float* __restrict__ flr, const T* __restrict__ w,
                                                                 int w_heads, const T* __restrict__ gate, int64_t gate_stride, int act,
                                                                 T* __restrict__ out, int64_t out_stride, float out_scale, int64_t rows, int H,
@@ -980,6 +995,32 @@ __global__ void __launch_bounds__(128) head_rmsnorm_gate_kernel(const float* __r
     const float* o = x + r * (vdim + (flr ? 1 : 0));
     const float inv = flr ? 1.0f / (fmaxf(fabsf(o[vdim]), flr[r]) + 1e-6f) : 1.0f;
     if (w && w_heads) w += (int64_t)h * vdim;
+    const T* gr = gate ? gate + t * gate_stride + (int64_t)h * vdim : nullptr;
+    T* dst = out + t * out_stride + (int64_t)h * vdim;
+    if constexpr (PER > 0) {                                // the whole head in registers, every operand in flight at once
+        float v[PER], g[PER], wv[PER];
+#pragma unroll
+        for (int k = 0; k < PER; ++k) {
+            const int c = lane + 32 * k;
+            const bool in = c < vdim;
+            v[k] = in ? o[c] : 0.f;
+            g[k] = in && gr ? ldf(gr + c) : 0.f;
+            wv[k] = in && w ? ldf(w + c) : 1.f;
+        }
+        float ss = 0.f;
+#pragma unroll
+        for (int k = 0; k < PER; ++k) {
+            v[k] *= inv;
+            ss = fmaf(v[k], v[k], ss);
+        }
+        const float rstd = out_scale / sqrtf(warp_sum(ss) / (float)vdim + eps);
+#pragma unroll
+        for (int k = 0; k < PER; ++k) {
+            const int c = lane + 32 * k;
+            if (c < vdim) stf(dst + c, v[k] * rstd * wv[k] * (gr ? (act ? siluf_(g[k]) : sigmoidf_(g[k])) : 1.f));
+        }
+        return;
+    }
     float ss = 0.f;
     for (int c = lane; c < vdim; c += 32) {
         const float v = o[c] * inv;
@@ -989,11 +1030,11 @@ __global__ void __launch_bounds__(128) head_rmsnorm_gate_kernel(const float* __r
     for (int c = lane; c < vdim; c += 32) {
         float v = o[c] * rstd;
         if (w) v *= ldf(w + c);
-        if (gate) {
-            const float z = ldf(gate + t * gate_stride + (int64_t)h * vdim + c);
+        if (gr) {
+            const float z = ldf(gr + c);
             v *= act ? siluf_(z) : sigmoidf_(z);
         }
-        stf(out + t * out_stride + (int64_t)h * vdim + c, v * out_scale);
+        stf(dst + c, v * out_scale);
     }
 }
 
@@ -1205,8 +1246,14 @@ extern "C" int b200m_head_rmsnorm_gate(const float* x, const float* floor, const
     if (!x || !out || n < 0 || num_heads <= 0 || vdim <= 0) return B200_EINVAL;
     if (n == 0) return B200_OK;
     const int64_t rows = (int64_t)n * num_heads;
-    B200M_DISPATCH(is32, B200_LAUNCH((head_rmsnorm_gate_kernel<T>), (unsigned)((rows + 3) / 4), 128, 0, static_cast<cudaStream_t>(stream), x, floor,
-                                     static_cast<const T*>(w), w_heads, static_cast<const T*>(gate), gate_stride, act, static_cast<T*>(out),
-                                     out_stride, out_scale, rows, num_heads, vdim, eps));
+#define HRG_GO(PER)                                                                                                                \
+    B200M_DISPATCH(is32, B200_LAUNCH((head_rmsnorm_gate_kernel<T, PER>), (unsigned)((rows + 3) / 4), 128, 0, static_cast<cudaStream_t>(stream), x, floor, \
+                                     static_cast<const T*>(w), w_heads, static_cast<const T*>(gate), gate_stride, act, static_cast<T*>(out), \
+                                     out_stride, out_scale, rows, num_heads, vdim, eps))
+    if (vdim <= 64) HRG_GO(2);
+    else if (vdim <= 128) HRG_GO(4);
+    else if (vdim <= 256) HRG_GO(8);
+    else HRG_GO(0);
+#undef HRG_GO
     return b200_launch_status(nullptr);
 }

@@ -7,6 +7,7 @@
 // when it changes hands.
 //
 //   causal_conv_kernel      : depthwise causal convolution + bias (+ SiLU) over a varlen batch, history taken from the slot
+//                             (causal_conv_vec_kernel: the same for bf16 rows in 8-byte steps)
 //   conv_state_update_kernel: the slot's history after the step (run after the convolution: it overwrites what that reads)
 //   selective_scan_kernel   : the recurrence, serial over a sequence's tokens, 4 lanes per channel holding the state in
 //                             registers; one token per sequence is the decode case of the same kernel.  Long portions run
@@ -64,6 +65,65 @@ __global__ void __launch_bounds__(256) causal_conv_kernel(const T* __restrict__ 
         float a = b;
         for (int k = 0; k < taps; ++k) a = fmaf(ldf(w + (int64_t)c * taps + k), input(i - (taps - 1 - k)), a);
         stf(out + (int64_t)(sp.q0 + i) * channels + c, act ? siluf_(a) : a);
+    }
+}
+
+// The same for bf16 rows in 8-byte steps: four channels per thread, TB tokens' inputs in flight at once, at most four taps.
+constexpr int CONV_TB = 8;
+__global__ void __launch_bounds__(128) causal_conv_vec_kernel(const __nv_bfloat16* __restrict__ x, int64_t x_stride, const __nv_bfloat16* __restrict__ w,
+                                                              const __nv_bfloat16* __restrict__ bias, const float* __restrict__ conv_state,
+                                                              const int32_t* __restrict__ state_slots, const int32_t* __restrict__ cu_q,
+                                                              const int32_t* __restrict__ cu_k, const int32_t* __restrict__ ctx_lens,
+                                                              __nv_bfloat16* __restrict__ out, int channels, int taps, int tok_tile, int act) {
+    B200_PDL_SYNC();
+    const int s = blockIdx.z;
+    const SeqSpan sp = seq_span(cu_q, cu_k, ctx_lens, s);
+    const int i0 = blockIdx.y * tok_tile;
+    if (i0 >= sp.qlen) return;
+    const int c = (blockIdx.x * 128 + threadIdx.x) * 4;
+    if (c >= channels) return;
+    const float* hist = conv_state + (int64_t)state_slots[s] * (taps - 1) * channels + c;
+    const __nv_bfloat16* xs = x + (int64_t)sp.q0 * x_stride + c;
+    __nv_bfloat16* os = out + (int64_t)sp.q0 * channels + c;
+    const int i1 = min(sp.qlen, i0 + tok_tile);
+    auto widen = [](const uint2& v, float (&f)[4]) { f[0] = bf16lo(v.x), f[1] = bf16hi(v.x), f[2] = bf16lo(v.y), f[3] = bf16hi(v.y); };
+    float wr[4][4], win[4][4], b[4] = {0.f, 0.f, 0.f, 0.f};        // [taps back][channel]; win[0] is the token's own input
+    if (bias) widen(*reinterpret_cast<const uint2*>(bias + c), b);
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+            wr[k][e] = k < taps ? ldf(w + (int64_t)(c + e) * taps + (taps - 1 - k)) : 0.f;
+            win[k][e] = 0.f;
+        }
+        if (k == 0 || k >= taps) continue;
+        if (i0 - k >= 0) {
+            widen(*reinterpret_cast<const uint2*>(xs + (int64_t)(i0 - k) * x_stride), win[k]);
+        } else if (sp.klen - sp.qlen > 0) {
+            const float4 f = *reinterpret_cast<const float4*>(hist + (int64_t)(taps - 1 + i0 - k) * channels);
+            win[k][0] = f.x, win[k][1] = f.y, win[k][2] = f.z, win[k][3] = f.w;
+        }
+    }
+    for (int i = i0; i < i1; i += CONV_TB) {
+        uint2 in[CONV_TB];
+#pragma unroll
+        for (int j = 0; j < CONV_TB; ++j) in[j] = i + j < i1 ? *reinterpret_cast<const uint2*>(xs + (int64_t)(i + j) * x_stride) : make_uint2(0, 0);
+#pragma unroll
+        for (int j = 0; j < CONV_TB; ++j) {
+            if (i + j >= i1) break;
+            widen(in[j], win[0]);
+            float a[4];
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                a[e] = b[e];
+#pragma unroll
+                for (int k = 0; k < 4; ++k) a[e] = fmaf(wr[k][e], win[k][e], a[e]);
+                if (act) a[e] = __fdividef(a[e], 1.0f + __expf(-a[e]));     // a bf16 result: the fast forms' error is far below its rounding
+#pragma unroll
+                for (int k = 3; k >= 1; --k) win[k][e] = win[k - 1][e];
+            }
+            *reinterpret_cast<uint2*>(os + (int64_t)(i + j) * channels) = make_uint2(pack_bf16x2(a[0], a[1]), pack_bf16x2(a[2], a[3]));
+        }
     }
 }
 
@@ -315,9 +375,16 @@ extern "C" int b200m_causal_conv(const void* x, int64_t x_stride, const void* w,
     if ((cu_q == nullptr) != (cu_k == nullptr) || (cu_q == nullptr && ctx_lens == nullptr)) return B200_EINVAL;
     if (num_seqs <= 0 || max_q <= 0) return B200_OK;
     cudaStream_t st = static_cast<cudaStream_t>(stream);
-    const int tok_tile = 64;
+    const uintptr_t bits = reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(bias) | reinterpret_cast<uintptr_t>(out);
+    const bool vec = !is32 && taps <= 4 && channels % 4 == 0 && x_stride % 4 == 0 && bits % 8 == 0 && reinterpret_cast<uintptr_t>(conv_state) % 16 == 0;
+    const int tok_tile = vec ? 32 : 64;
     dim3 grid((channels + 255) / 256, (max_q + tok_tile - 1) / tok_tile, num_seqs);
-    B200M_DISPATCH(is32, B200_LAUNCH((causal_conv_kernel<T>), grid, 256, 0, st, static_cast<const T*>(x), x_stride,
+    if (vec) {
+        using bf = __nv_bfloat16;
+        grid.x = (channels / 4 + 127) / 128;
+        B200_LAUNCH((causal_conv_vec_kernel), grid, 128, 0, st, static_cast<const bf*>(x), x_stride, static_cast<const bf*>(w), static_cast<const bf*>(bias),
+                    conv_state, state_slots, cu_q, cu_k, ctx_lens, static_cast<bf*>(out), channels, taps, tok_tile, act);
+    } else B200M_DISPATCH(is32, B200_LAUNCH((causal_conv_kernel<T>), grid, 256, 0, st, static_cast<const T*>(x), x_stride,
                                      static_cast<const T*>(w), static_cast<const T*>(bias), conv_state, state_slots, cu_q, cu_k,
                                      ctx_lens, static_cast<T*>(out), channels, taps, tok_tile, act));
     int rc = b200_launch_status(nullptr);

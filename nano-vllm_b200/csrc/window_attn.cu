@@ -17,7 +17,7 @@
 //                          key/value tiles shared by the warps of a CTA through shared memory)
 //   window_attn_mma_kernel (bf16): the same on the tensor cores, 64 (token, head) rows x 64-key tiles, double-buffered
 //                          asynchronous copies; single-token steps may split a long window over several CTAs.  Head sizes other
-//                          than 32 / 64 / 128 (multiples of eight up to 128) run as 64 or 128 with zero columns
+//                          than 32 / 64 / 128 (multiples of eight up to 128) run as 64, 96 or 128 with zero columns
 #include "mma_common.cuh"
 
 namespace {
@@ -786,6 +786,7 @@ extern "C" int b200m_window_attention(const void* q, int64_t q_stride, const voi
         WA_MMA(128, 64);
         WA_MMA(128, 128);
         if (dim <= 64 && vdim <= 64) WA_MMA_AS(64, 64, true);            // other head sizes: zero columns up to the next tile
+        if (dim <= 96 && vdim <= 96) WA_MMA_AS(96, 96, true);
         WA_MMA_AS(128, 128, true);
 #undef WA_MMA
 #undef WA_MMA_AS
@@ -885,6 +886,72 @@ __global__ void __launch_bounds__(128) headnorm_rope_store_kernel(T* __restrict_
             if (c1 < d) stf(dst + c1, b);
         }
     }
+}
+
+// The same for bf16 rows with half-split pairs, no norm weights and values as they are: a group of GS lanes per query or key head, sixteen
+// elements per lane (two 16-byte pieces: eight first and their eight second partners, or sixteen behind the rotated part), the rest of
+// the CTA copies values.  rope_dims and dim multiples of sixteen, vdim of eight, everything 16-byte aligned.
+template <int GS>
+__global__ void __launch_bounds__(256) rope_store_vec_kernel(__nv_bfloat16* __restrict__ x, int64_t stride, int q_off, int k_off, int v_off, int H, int G,
+                                                             int dim, int vdim, int unit_after, const float* __restrict__ cos_sin, int rope_dims,
+                                                             const int64_t* __restrict__ positions, const int32_t* __restrict__ slots,
+                                                             __nv_bfloat16* __restrict__ cache, float eps) {
+    B200_PDL_SYNC();
+    const int t = blockIdx.x, half = rope_dims / 2, units = dim / 16, heads = H + G;
+    __nv_bfloat16* row = x + (int64_t)t * stride;
+    const int slot = cache ? slots[t] : -1;
+    __nv_bfloat16* crow = slot >= 0 ? cache + (int64_t)slot * ((int64_t)G * (dim + vdim)) : nullptr;
+    const float* cs = rope_dims ? cos_sin + positions[t] * rope_dims : nullptr;
+    const int head_work = (heads * GS + 255) / 256 * 256;          // whole CTA strides: every lane of a group takes part in its sums
+    for (int e = threadIdx.x; e < head_work; e += 256) {
+        const int r = e / GS, u = e % GS;
+        const bool ok = r < heads && u < units && (r < H || crow != nullptr);
+        __nv_bfloat16* src = row + (r < H ? q_off + r * dim : k_off + (r - H) * dim);
+        __nv_bfloat16* dst = r < H ? src : crow + (int64_t)(r - H) * dim;
+        const bool turn = u * 8 < half;
+        const int c0 = turn ? u * 8 : 16 * u, c1 = turn ? c0 + half : c0 + 8;
+        float a[8], b[8];
+#pragma unroll
+        for (int i = 0; i < 8; ++i) a[i] = b[i] = 0.f;
+        if (ok) {
+            unpack8(*reinterpret_cast<const uint4*>(src + c0), a);
+            unpack8(*reinterpret_cast<const uint4*>(src + c1), b);
+            if (turn) {
+                float co[8], si[8];
+#pragma unroll
+                for (int i = 0; i < 8; i += 4) {
+                    *reinterpret_cast<float4*>(co + i) = *reinterpret_cast<const float4*>(cs + c0 + i);
+                    *reinterpret_cast<float4*>(si + i) = *reinterpret_cast<const float4*>(cs + half + c0 + i);
+                }
+#pragma unroll
+                for (int i = 0; i < 8; ++i) {
+                    const float ra = a[i] * co[i] - b[i] * si[i], rb = b[i] * co[i] + a[i] * si[i];
+                    a[i] = ra;
+                    b[i] = rb;
+                }
+            }
+        }
+        if (unit_after) {
+            float ss = 0.f;
+#pragma unroll
+            for (int i = 0; i < 8; ++i) ss = fmaf(a[i], a[i], fmaf(b[i], b[i], ss));
+#pragma unroll
+            for (int o = 1; o < GS; o <<= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+            const float rstd = 1.0f / sqrtf(ss / (float)dim + eps);
+#pragma unroll
+            for (int i = 0; i < 8; ++i) {
+                a[i] *= rstd;
+                b[i] *= rstd;
+            }
+        }
+        if (ok) {
+            *reinterpret_cast<uint4*>(dst + c0) = pack8(a);
+            *reinterpret_cast<uint4*>(dst + c1) = pack8(b);
+        }
+    }
+    if (crow == nullptr) return;
+    for (int e = threadIdx.x; e < G * vdim / 8; e += 256)
+        *reinterpret_cast<uint4*>(crow + (int64_t)G * dim + e * 8) = *reinterpret_cast<const uint4*>(row + v_off + e * 8);
 }
 
 // out[t, h, :] = rotate(acc[t, h, :], sign * position) * sigmoid(gate[t, h, :]): a thread per pair of elements of a head.
@@ -1022,6 +1089,23 @@ extern "C" int b200m_headnorm_rope_store(void* x, int64_t stride, int q_off, int
     if (v_rope_dims == 0) v_cos_sin = nullptr;
     if (n == 0) return B200_OK;
     if (rope_dims == 0) cos_sin = nullptr;
+    const uintptr_t bits = reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(cache) | reinterpret_cast<uintptr_t>(cos_sin);
+    if (!is32 && layout == 1 && !q_norm_w && !k_norm_w && !v_unit_norm && !v_cos_sin && dim <= 256 && dim % 16 == 0 && rope_dims % 16 == 0 && vdim % 8 == 0 &&
+        (stride | q_off | k_off | v_off) % 8 == 0 && bits % 16 == 0) {
+        using bf = __nv_bfloat16;
+#define ROPE_VEC(GS)                                                                                                               \
+    do {                                                                                                                           \
+        B200_LAUNCH((rope_store_vec_kernel<GS>), n, 256, 0, static_cast<cudaStream_t>(stream), static_cast<bf*>(x), stride, q_off, k_off, v_off, \
+                    num_heads, num_kv_heads, dim, vdim, unit_after, cos_sin, cos_sin ? rope_dims : 0, positions, slots, static_cast<bf*>(cache), eps); \
+        return b200_launch_status(nullptr);                                                                                        \
+    } while (0)
+        if (dim <= 16) ROPE_VEC(1);
+        if (dim <= 32) ROPE_VEC(2);
+        if (dim <= 64) ROPE_VEC(4);
+        if (dim <= 128) ROPE_VEC(8);
+        ROPE_VEC(16);
+#undef ROPE_VEC
+    }
     B200M_DISPATCH(is32, B200_LAUNCH((headnorm_rope_store_kernel<T>), n, 128, 0, static_cast<cudaStream_t>(stream), static_cast<T*>(x), stride,
                                      q_off, k_off, v_off, num_heads, num_kv_heads, dim, vdim, static_cast<const T*>(q_norm_w),
                                      static_cast<const T*>(k_norm_w), v_unit_norm, unit_after, cos_sin, layout, rope_dims, v_cos_sin, v_rope_dims, positions, slots,

@@ -64,8 +64,10 @@ def test_silu_gated_feed_forward(dtype, ff):
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
-@pytest.mark.parametrize("shape", [(3, 1, 16, 24, 8), (4, 2, 64, 32, 64), (2, 2, 9, 7, 4), (5, 5, 32, 128, 0), (2, 1, 96, 16, 48), (1, 1, 200, 8, 66)])
-def test_unit_norm_after_the_rotation(dtype, shape):
+@pytest.mark.parametrize("pad", [5, 8])
+@pytest.mark.parametrize("shape", [(3, 1, 16, 24, 8), (4, 2, 64, 32, 64), (2, 2, 9, 7, 4), (5, 5, 32, 128, 0), (2, 1, 96, 16, 48), (1, 1, 200, 8, 66),
+                                   (40, 4, 128, 64, 64), (3, 3, 16, 8, 16), (2, 1, 256, 24, 32), (1, 1, 48, 40, 16)])
+def test_unit_norm_after_the_rotation(dtype, shape, pad):
     """Rotated part scaled by the table's magnitude, the rest not, then one root mean square over both (with an eps that counts for small
     heads); positions up to the thousands; keys cached so, values as they are; a token with slot -1 stores nothing."""
     from nanovllm import mixops
@@ -73,7 +75,7 @@ def test_unit_norm_after_the_rotation(dtype, shape):
     H, G, d, vd, dims = shape
     g = torch.Generator().manual_seed(sum(shape))
     n, base, eps = 9, 777.0, 1e-2
-    cols = H * d + G * d + G * vd + 5
+    cols = H * d + G * d + G * vd + pad                       # 5: rows that are not 16-byte aligned
     x = (torch.randn(n, cols, generator=g) * torch.tensor([1.0, 0.05, 3.0, 1.0, 0.2, 1.0, 1.0, 10.0, 1.0])[:, None]).to(DT[dtype])
     pos = torch.tensor([0, 1, 2, 63, 64, 500, 1999, 3, 1000], dtype=torch.int64)
     slots = torch.tensor([4, 0, 17, -1, 3, 9, 8, 30, 1], dtype=torch.int32)
