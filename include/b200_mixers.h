@@ -259,7 +259,7 @@ int b200m_linear_state(const void* x, int64_t stride, int q_off, int k_off, int 
  * m_state fp32 [slots, num_heads], 0 for a new sequence. */
 int b200m_mlstm_gates(const float* in, int64_t stride, const float* bias, float cap, float* m_state, const int32_t* state_slots,
                       const int32_t* cu_q, const int32_t* cu_k, const int32_t* ctx_lens, float* log_decay, float* write, float* floor,
-                      int num_seqs, int num_heads, void* stream);
+                      int num_seqs, int max_q, int num_heads, void* stream);
 
 /* t = (y[r, h, :] + D[h] x[r, h, :]) * silu(z[r, h, :]) over rows of num_heads * vdim columns, then every one of `groups` equal parts of the
  * row divided by its own root mean square (sqrt(mean(t^2) + eps)), times w [num_heads * vdim].  y, D fp32; x, z, w, out in the activation

@@ -915,42 +915,36 @@ int launch_matrix_state(const void* x, int64_t stride, int q_off, int k_off, int
 // Exponential gates of a matrix memory: from pre-activations (i | f) of H heads each, i <- cap tanh((i + b) / cap), f <- logsigmoid(cap
 // tanh((f + b) / cap)), the running maximum m_t = max(f_t + m_(t-1), i_t) (from 0 for a new sequence), and with it
 //     log_decay = f_t + m_(t-1) - m_t,   write = exp(i_t - m_t),   floor = exp(-m_t)                        (all fp32)
-// One warp per (sequence, head), 32 x MG_T tokens per step: (f, i) pairs compose as (f1 + f2, max(i1 + f2, i2)), a scan over the lanes.
-constexpr int MG_T = 4;
-__global__ void __launch_bounds__(128) mlstm_gates_kernel(const float* __restrict__ in, int64_t stride, const float* __restrict__ bias, float cap,
-                                                          float* __restrict__ mstate, const int32_t* __restrict__ state_slots,
-                                                          const int32_t* __restrict__ cu_q, const int32_t* __restrict__ cu_k,
-                                                          const int32_t* __restrict__ ctx_lens, float* __restrict__ log_decay,
-                                                          float* __restrict__ write, float* __restrict__ flr, int H) {
+// One CTA of NW warps per (sequence, head), a token per thread and step: (f, i) pairs compose as (f1 + f2, max(i1 + f2, i2)), a scan over
+// the lanes and then over the warps.
+template <int NW>
+__global__ void __launch_bounds__(NW * 32) mlstm_gates_kernel(const float* __restrict__ in, int64_t stride, const float* __restrict__ bias, float cap,
+                                                              float* __restrict__ mstate, const int32_t* __restrict__ state_slots,
+                                                              const int32_t* __restrict__ cu_q, const int32_t* __restrict__ cu_k,
+                                                              const int32_t* __restrict__ ctx_lens, float* __restrict__ log_decay,
+                                                              float* __restrict__ write, float* __restrict__ flr, int H) {
     B200_PDL_SYNC();
-    const int s = blockIdx.y, h = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+    __shared__ float2 part[2][NW];                          // (F, I) of every warp's tokens, double-buffered over the steps
+    const int s = blockIdx.y, h = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const SeqSpan sp = seq_span(cu_q, cu_k, ctx_lens, s);
-    if (sp.qlen <= 0 || h >= H) return;
+    if (sp.qlen <= 0) return;
     float* mp = mstate + (int64_t)state_slots[s] * H + h;
     float m = sp.klen - sp.qlen > 0 ? *mp : 0.f;
     const float bi = bias[h], bf = bias[H + h];
-    float ri[MG_T], rf[MG_T];
-    auto fetch = [&](int i0) {
-#pragma unroll
-        for (int j = 0; j < MG_T; ++j) {
-            const int i = i0 + lane * MG_T + j;
+    float ri = 0.f, rf = 0.f;
+    auto fetch = [&](int i) {
+        if (i < sp.qlen) {
             const float* row = in + (int64_t)(sp.q0 + i) * stride + h;
-            ri[j] = i < sp.qlen ? row[0] : 0.f;
-            rf[j] = i < sp.qlen ? row[H] : 0.f;
+            ri = row[0], rf = row[H];
         }
     };
-    fetch(0);
-    for (int i0 = 0; i0 < sp.qlen; i0 += 32 * MG_T) {
-        float gi[MG_T], gf[MG_T], F = 0.f, I = -INFINITY;      // (F, I): the lane's tokens composed; nothing past the end
-#pragma unroll
-        for (int j = 0; j < MG_T; ++j) {
-            const bool ok = i0 + lane * MG_T + j < sp.qlen;
-            gi[j] = ok ? cap * tanhf((ri[j] + bi) / cap) : -INFINITY;
-            gf[j] = ok ? -softplus_(-cap * tanhf((rf[j] + bf) / cap)) : 0.f;
-            I = fmaxf(I + gf[j], gi[j]);
-            F += gf[j];
-        }
-        fetch(i0 + 32 * MG_T);
+    fetch(threadIdx.x);
+    for (int i0 = 0, buf = 0; i0 < sp.qlen; i0 += NW * 32, buf ^= 1) {
+        const int i = i0 + threadIdx.x;
+        const bool ok = i < sp.qlen;                         // past the end: nothing is added and the maximum stays
+        const float gi = ok ? cap * tanhf((ri + bi) / cap) : -INFINITY, gf = ok ? -softplus_(-cap * tanhf((rf + bf) / cap)) : 0.f;
+        fetch(i + NW * 32);
+        float F = gf, I = gi;
 #pragma unroll
         for (int o = 1; o < 32; o <<= 1) {
             const float pf = __shfl_up_sync(0xffffffffu, F, o), pi = __shfl_up_sync(0xffffffffu, I, o);
@@ -959,23 +953,31 @@ __global__ void __launch_bounds__(128) mlstm_gates_kernel(const float* __restric
                 F += pf;
             }
         }
-        const float end = fmaxf(F + m, I);                     // maximum after the lane's last token
-        float prev = __shfl_up_sync(0xffffffffu, end, 1);
-        if (lane == 0) prev = m;
-        m = __shfl_sync(0xffffffffu, end, 31);                 // lanes past the end carry the last token's maximum on
+        if constexpr (NW > 1) {
+            if (lane == 31) part[buf][warp] = make_float2(F, I);
+            __syncthreads();
+        }
+        float prev = m;                                      // maximum before this warp's tokens
+        if constexpr (NW > 1) {
 #pragma unroll
-        for (int j = 0; j < MG_T; ++j) {
-            const int i = i0 + lane * MG_T + j;
-            if (i >= sp.qlen) break;
-            const float mt = fmaxf(gf[j] + prev, gi[j]);
+            for (int w = 0; w < NW; ++w) {
+                const float2 p = part[buf][w];
+                m = fmaxf(p.x + m, p.y);
+                if (w + 1 == warp) prev = m;
+            }
+        }
+        const float mt = fmaxf(F + prev, I);
+        const float up = __shfl_up_sync(0xffffffffu, mt, 1);
+        if (lane > 0) prev = up;
+        if constexpr (NW == 1) m = __shfl_sync(0xffffffffu, mt, 31);
+        if (ok) {
             const int64_t at = (int64_t)(sp.q0 + i) * H + h;
-            log_decay[at] = gf[j] + prev - mt;
-            write[at] = expf(gi[j] - mt);
+            log_decay[at] = gf + prev - mt;
+            write[at] = expf(gi - mt);
             flr[at] = expf(-mt);
-            prev = mt;
         }
     }
-    if (lane == 0) *mp = m;
+    if (threadIdx.x == 0) *mp = m;
 }
 
 // out[t, h, :] = c * o / sqrt(mean(o^2) + eps) * w * act(gate[t, h, :]) for o = x[t, h, :] (fp32), one warp per (token, head).
@@ -1186,13 +1188,17 @@ extern "C" int b200m_channel_state(const void* x, int64_t stride, int q_off, int
 
 extern "C" int b200m_mlstm_gates(const float* in, int64_t stride, const float* bias, float cap, float* m_state, const int32_t* state_slots,
                                  const int32_t* cu_q, const int32_t* cu_k, const int32_t* ctx_lens, float* log_decay, float* write, float* floor,
-                                 int num_seqs, int num_heads, void* stream) {
+                                 int num_seqs, int max_q, int num_heads, void* stream) {
     if (!in || !bias || !m_state || !state_slots || !log_decay || !write || !floor || num_heads <= 0 || !(cap > 0.f) || stride < 2 * num_heads)
         return B200_EINVAL;
     if ((cu_q == nullptr) != (cu_k == nullptr) || (cu_q == nullptr && ctx_lens == nullptr)) return B200_EINVAL;
     if (num_seqs <= 0) return B200_OK;
-    B200_LAUNCH((mlstm_gates_kernel), dim3((num_heads + 3) / 4, num_seqs), 128, 0, static_cast<cudaStream_t>(stream), in, stride, bias, cap, m_state,
-                state_slots, cu_q, cu_k, ctx_lens, log_decay, write, floor, num_heads);
+#define MG_GO(NW)                                                                                                                  \
+    B200_LAUNCH((mlstm_gates_kernel<NW>), dim3(num_heads, num_seqs), NW * 32, 0, static_cast<cudaStream_t>(stream), in, stride, bias, cap, m_state, \
+                state_slots, cu_q, cu_k, ctx_lens, log_decay, write, floor, num_heads)
+    if (cu_q == nullptr || max_q <= 32) MG_GO(1);
+    else MG_GO(8);
+#undef MG_GO
     return b200_launch_status(nullptr);
 }
 

@@ -69,7 +69,7 @@ MIX_SIGNATURES = {
                                  _i, _f, _i, _vp]),
     "b200m_linear_state": (_i, [_vp, _i64, _i, _i, _i, _vp, _vp, _vp, _i64, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _f,
                                 _i, _i, _vp]),
-    "b200m_mlstm_gates": (_i, [_vp, _i64, _vp, _f, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _vp]),
+    "b200m_mlstm_gates": (_i, [_vp, _i64, _vp, _f, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _vp]),
     "b200m_skip_gate_groupnorm": (_i, [_vp, _vp, _i64, _vp, _vp, _i64, _vp, _vp, _i64, _i, _i, _i, _i, _f, _i, _vp]),
     "b200m_head_rmsnorm_gate": (_i, [_vp, _vp, _vp, _i, _vp, _i64, _i, _vp, _i64, _f, _i, _i, _i, _f, _i, _vp]),
     "b200m_moe_route_grouped": (_i, [_vp, _i64, _i, _i, _i, _vp, _i, _i, _i, _i, _i, _f, _vp, _vp, _vp]),

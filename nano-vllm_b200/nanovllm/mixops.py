@@ -544,7 +544,7 @@ def mlstm_gates(pre: torch.Tensor, bias: torch.Tensor, cap: float, m_state: torc
     assert m_state.dtype == torch.float32 and m_state.is_contiguous() and m_state.shape[1] == heads and state_slots.dtype == torch.int32
     out = torch.empty(3, n, heads, dtype=torch.float32, device=pre.device)
     _call("b200m_mlstm_gates", pre.data_ptr(), pre.stride(0), bias.data_ptr(), float(cap), m_state.data_ptr(), state_slots.data_ptr(), _p(spans.cu_q),
-          _p(spans.cu_k), _p(spans.ctx_lens), out[0].data_ptr(), out[1].data_ptr(), out[2].data_ptr(), spans.num_seqs, heads, _stream())
+          _p(spans.cu_k), _p(spans.ctx_lens), out[0].data_ptr(), out[1].data_ptr(), out[2].data_ptr(), spans.num_seqs, spans.max_q, heads, _stream())
     return out[0], out[1], out[2]
 
 
