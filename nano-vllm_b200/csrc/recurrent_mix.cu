@@ -859,6 +859,83 @@ __global__ void __launch_bounds__(MB_THREADS, DPL <= 16 ? 2 : 1) matrix_state_bl
     }
 }
 
+// Scalar linear attention, single-token steps: the state streams through registers once.  LPC lanes share a column (VPL float4s of its dim
+// rows each), a warp works on eight columns per lane group at a time, all of whose loads are in flight together; no shared memory.
+constexpr int LD_COLS = 8;
+template <typename T, int LPC, int VPL>
+__global__ void __launch_bounds__(128) linear_state_token_kernel(const T* __restrict__ x, int64_t stride, int q_off, int k_off, int v_off, ScalarGate<T> sg,
+                                                                 float* __restrict__ state, const int32_t* __restrict__ state_slots,
+                                                                 const int32_t* __restrict__ ctx_lens, float* __restrict__ out, int H, int G, int dim,
+                                                                 int vdim, int ones, float q_scale, int vec_x) {
+    B200_PDL_SYNC();
+    constexpr int GROUPS = 32 / LPC;
+    const int h = blockIdx.x, s = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, sub = lane % LPC;
+    const int klen = ctx_lens[s];
+    if (klen <= 0) return;                                  // padding row
+    const int vcols = vdim + ones, col0 = (blockIdx.z * 4 + warp) * LD_COLS * GROUPS + lane / LPC;
+    if ((blockIdx.z * 4 + warp) * LD_COLS * GROUPS >= vcols) return;
+    float* st = state + ((int64_t)state_slots[s] * H + h) * vcols * dim;
+    float4 S[LD_COLS][VPL];
+#pragma unroll
+    for (int i = 0; i < LD_COLS; ++i)
+#pragma unroll
+        for (int j = 0; j < VPL; ++j) {
+            const int col = col0 + i * GROUPS, d = (j * LPC + sub) * 4;
+            S[i][j] = klen > 1 && col < vcols && d < dim ? *reinterpret_cast<const float4*>(st + (int64_t)col * dim + d) : make_float4(0.f, 0.f, 0.f, 0.f);
+        }
+    const T* xr = x + (int64_t)s * stride;
+    const float2 f = sg.gates(sg.fetch(s, h), sg.rate ? sg.rate[h] : 0.f, sg.rate ? sg.bias[h] : 0.f);
+    const float g = expf(f.x), w = f.y;
+    float k[VPL][4], q[VPL][4], v[LD_COLS], o[LD_COLS];
+#pragma unroll
+    for (int j = 0; j < VPL; ++j) {
+        const int d = (j * LPC + sub) * 4;
+        RawCols<T, 4> rk, rq;
+        rk.load(xr + k_off + (int64_t)(h / (H / G)) * dim + d, dim - d, vec_x);
+        rq.load(xr + q_off + (int64_t)(h / (H / G)) * dim + d, dim - d, vec_x);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+            k[j][e] = rk.at(e);
+            q[j][e] = rq.at(e) * q_scale;
+        }
+    }
+#pragma unroll
+    for (int i = 0; i < LD_COLS; ++i) {
+        const int col = col0 + i * GROUPS;
+        v[i] = w * (col < vdim ? ldf(xr + v_off + (int64_t)h * vdim + col) : 1.0f);        // the column behind the values holds ones
+        o[i] = 0.f;
+    }
+#pragma unroll
+    for (int i = 0; i < LD_COLS; ++i)
+#pragma unroll
+        for (int j = 0; j < VPL; ++j) {
+            const int col = col0 + i * GROUPS, d = (j * LPC + sub) * 4;
+            float4& t = S[i][j];
+            t.x = fmaf(k[j][0], v[i], g * t.x), t.y = fmaf(k[j][1], v[i], g * t.y), t.z = fmaf(k[j][2], v[i], g * t.z), t.w = fmaf(k[j][3], v[i], g * t.w);
+            o[i] = fmaf(t.x, q[j][0], fmaf(t.y, q[j][1], fmaf(t.z, q[j][2], fmaf(t.w, q[j][3], o[i]))));
+            if (col < vcols && d < dim) *reinterpret_cast<float4*>(st + (int64_t)col * dim + d) = t;
+        }
+    // eight sums over LPC lanes: three steps halve the sums a lane carries, the rest add up the one that is left
+    int own = 0;
+#pragma unroll
+    for (int n = LD_COLS / 2, off = LPC / 2; off > 0; n >>= 1, off >>= 1) {
+        if (n > 0) {
+            const bool hi = sub & off;
+            own += hi ? n : 0;
+#pragma unroll
+            for (int i = 0; i < LD_COLS / 2; ++i)
+                if (i < n) {
+                    const float send = hi ? o[i] : o[i + n], keep = hi ? o[i + n] : o[i];
+                    o[i] = keep + __shfl_xor_sync(0xffffffffu, send, off);
+                }
+        } else {
+            o[0] += __shfl_xor_sync(0xffffffffu, o[0], off);
+        }
+    }
+    const int col = col0 + own * GROUPS;
+    if ((sub & (LPC / LD_COLS - 1)) == 0 && col < vcols) out[((int64_t)s * H + h) * vcols + col] = o[0];
+}
+
 template <typename T, bool CH, bool DELTA>
 int launch_matrix_state(const void* x, int64_t stride, int q_off, int k_off, int v_off, const float* write_in, const void* write_t,
                         int64_t write_stride, const DecayIn& dec, float* state, const int32_t* state_slots, const int32_t* cu_q,
@@ -888,6 +965,23 @@ int launch_matrix_state(const void* x, int64_t stride, int q_off, int k_off, int
         MB_GO(32, 2);
     }
 #undef MB_GO
+    if constexpr (!CH && !DELTA) {
+        if (cu_q == nullptr && dim % 4 == 0) {
+            const int vx = (stride | q_off | k_off) % 4 == 0 && reinterpret_cast<uintptr_t>(x) % 16 == 0;
+#define LS_GO(LPC, VPL)                                                                                                            \
+    do {                                                                                                                           \
+        constexpr int CC = 4 * LD_COLS * (32 / LPC);                                                                               \
+        B200_LAUNCH((linear_state_token_kernel<T, LPC, VPL>), dim3(H, num_seqs, (vcols + CC - 1) / CC), 128, 0, st, static_cast<const T*>(x), stride, \
+                    q_off, k_off, v_off, sg, state, state_slots, ctx_lens, out, H, G, dim, vdim, ones, q_scale, vx);                \
+        return b200_launch_status(nullptr);                                                                                        \
+    } while (0)
+            if (dim <= 32) LS_GO(8, 1);
+            if (dim <= 64) LS_GO(16, 1);
+            if (dim <= 128) LS_GO(32, 1);
+            LS_GO(32, 2);
+#undef LS_GO
+        }
+    }
     if constexpr (CH) {
         const int cols = H * dim, rows = cu_q ? total_rows : num_seqs;
         B200_LAUNCH((channel_decay_kernel), dim3(rows, (unsigned)((cols + 1023) / 1024)), 256, 0, st, const_cast<float*>(dec.in), dec.stride,
