@@ -8,7 +8,8 @@
 //
 //   causal_conv_kernel      : depthwise causal convolution + bias (+ SiLU) over a varlen batch, history taken from the slot
 //                             (causal_conv_vec_kernel: the same for bf16 rows in 8-byte steps)
-//   conv_state_update_kernel: the slot's history after the step (run after the convolution: it overwrites what that reads)
+//   conv_state_update_kernel: the slot's history after the step (run after the convolution: it overwrites what that reads; single-token
+//                             steps with at most eight taps leave it to the convolution, whose threads own their channels then)
 //   selective_scan_kernel   : the recurrence, serial over a sequence's tokens, 4 lanes per channel holding the state in
 //                             registers; one token per sequence is the decode case of the same kernel.  Long portions run
 //                             it three times over chunks of tokens: (1) every chunk from a zero state, keeping its end state
@@ -23,7 +24,7 @@ constexpr int CONV_MAX_TAPS = 8;
 // conv_state: [slots, taps - 1, channels] fp32, row taps-2 is the newest input.
 template <typename T>
 __global__ void __launch_bounds__(256) causal_conv_kernel(const T* __restrict__ x, int64_t x_stride, const T* __restrict__ w,
-                                                          const T* __restrict__ bias, const float* __restrict__ conv_state,
+                                                          const T* __restrict__ bias, float* conv_state,
                                                           const int32_t* __restrict__ state_slots, const int32_t* __restrict__ cu_q,
                                                           const int32_t* __restrict__ cu_k, const int32_t* __restrict__ ctx_lens,
                                                           T* __restrict__ out, int channels, int taps, int tok_tile, int act) {
@@ -35,7 +36,7 @@ __global__ void __launch_bounds__(256) causal_conv_kernel(const T* __restrict__ 
     const int c = blockIdx.x * blockDim.x + threadIdx.x;
     if (c >= channels) return;
     const bool has_hist = sp.klen - sp.qlen > 0;
-    const float* hist = conv_state + (int64_t)state_slots[s] * (taps - 1) * channels;
+    float* hist = conv_state + (int64_t)state_slots[s] * (taps - 1) * channels;
     const float b = bias ? ldf(bias + c) : 0.f;
     const int i1 = min(sp.qlen, i0 + tok_tile);
     auto input = [&](int m) -> float {                     // input at local index m of the portion (negative: before it)
@@ -59,6 +60,11 @@ __global__ void __launch_bounds__(256) causal_conv_kernel(const T* __restrict__ 
 #pragma unroll
             for (int k = CONV_MAX_TAPS - 1; k >= 1; --k) win[k] = win[k - 1];
         }
+        if (cu_q == nullptr) {                              // single-token step: this thread alone knows the channel, the history moves on here
+#pragma unroll
+            for (int k = 1; k < CONV_MAX_TAPS; ++k)
+                if (k < taps) hist[(int64_t)(taps - 1 - k) * channels + c] = win[k];
+        }
         return;
     }
     for (int i = i0; i < i1; ++i) {
@@ -71,7 +77,7 @@ __global__ void __launch_bounds__(256) causal_conv_kernel(const T* __restrict__ 
 // The same for bf16 rows in 8-byte steps: four channels per thread, TB tokens' inputs in flight at once, at most four taps.
 constexpr int CONV_TB = 8;
 __global__ void __launch_bounds__(128) causal_conv_vec_kernel(const __nv_bfloat16* __restrict__ x, int64_t x_stride, const __nv_bfloat16* __restrict__ w,
-                                                              const __nv_bfloat16* __restrict__ bias, const float* __restrict__ conv_state,
+                                                              const __nv_bfloat16* __restrict__ bias, float* conv_state,
                                                               const int32_t* __restrict__ state_slots, const int32_t* __restrict__ cu_q,
                                                               const int32_t* __restrict__ cu_k, const int32_t* __restrict__ ctx_lens,
                                                               __nv_bfloat16* __restrict__ out, int channels, int taps, int tok_tile, int act) {
@@ -82,7 +88,7 @@ __global__ void __launch_bounds__(128) causal_conv_vec_kernel(const __nv_bfloat1
     if (i0 >= sp.qlen) return;
     const int c = (blockIdx.x * 128 + threadIdx.x) * 4;
     if (c >= channels) return;
-    const float* hist = conv_state + (int64_t)state_slots[s] * (taps - 1) * channels + c;
+    float* hist = conv_state + (int64_t)state_slots[s] * (taps - 1) * channels + c;
     const __nv_bfloat16* xs = x + (int64_t)sp.q0 * x_stride + c;
     __nv_bfloat16* os = out + (int64_t)sp.q0 * channels + c;
     const int i1 = min(sp.qlen, i0 + tok_tile);
@@ -124,6 +130,11 @@ __global__ void __launch_bounds__(128) causal_conv_vec_kernel(const __nv_bfloat1
             }
             *reinterpret_cast<uint2*>(os + (int64_t)(i + j) * channels) = make_uint2(pack_bf16x2(a[0], a[1]), pack_bf16x2(a[2], a[3]));
         }
+    }
+    if (cu_q == nullptr) {                                  // single-token step: the history moves on here
+#pragma unroll
+        for (int k = 1; k < 4; ++k)
+            if (k < taps) *reinterpret_cast<float4*>(hist + (int64_t)(taps - 1 - k) * channels) = make_float4(win[k][0], win[k][1], win[k][2], win[k][3]);
     }
 }
 
@@ -388,7 +399,7 @@ extern "C" int b200m_causal_conv(const void* x, int64_t x_stride, const void* w,
                                      static_cast<const T*>(w), static_cast<const T*>(bias), conv_state, state_slots, cu_q, cu_k,
                                      ctx_lens, static_cast<T*>(out), channels, taps, tok_tile, act));
     int rc = b200_launch_status(nullptr);
-    if (rc != B200_OK || taps == 1) return rc;
+    if (rc != B200_OK || taps == 1 || (cu_q == nullptr && taps <= CONV_MAX_TAPS)) return rc;
     dim3 grid2((channels + 255) / 256, num_seqs);
     B200M_DISPATCH(is32, B200_LAUNCH((conv_state_update_kernel<T>), grid2, 256, 0, st, static_cast<const T*>(x), x_stride,
                                      conv_state, state_slots, cu_q, cu_k, ctx_lens, channels, taps));
